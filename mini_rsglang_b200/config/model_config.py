@@ -746,3 +746,171 @@ class MigenexConfig(ModelConfig):
         if self.eos_token_id is not None:
             out["eos_token_id"] = self.eos_token_id
         return out
+
+
+@dataclass
+class PisatarConfig(ModelConfig):
+    """Pisatar: a decoder of layers whose two branches, a mixer and a dense gated feed-forward, each read an RMS norm of their own
+    (weights stored around zero) of the same stream.  The mixer is a retention (linear attention with rotated heads and a
+    constant decay a head), a gated delta rule with one decay a key channel ("channel_delta"), or two mixers side by side
+    ("parallel"): an attention with partly rotated heads and an exponentially gated matrix memory, each times a constant.  The
+    embeddings pass a norm.  A layer may use another layer's weights, with a cache or state of its own.  config.json names the
+    design under `architecture`; its keys are read as they stand there:
+
+      vocab, width, norm.eps
+      layers[i].type = "retention":     mixer.{heads, dim, vdim, decay[heads], rot.{base, dims}}
+      layers[i].type = "channel_delta": mixer.{heads, kv_heads, dim, vdim, conv}
+      layers[i].type = "parallel":      mixer.{left.{heads, kv_heads, dim, vdim, scale, rot.{base, dims, scaling.{factor, low, high, original}}},
+                                               right.{heads, dim, vdim, gate_cap}, left_scale, right_scale}
+      layers[i].mlp = null | {kind: "dense", ff};  layers[i].weights_of = j (the rest of the entry equals layer j's)
+
+    `mlp`, `weights_of` and `rot.scaling` may be absent.  The inner sizes of a channel_delta's thin products stand in the
+    checkpoint; `mixer.decay_rank` and `mixer.gate_rank` give them for a model that is drawn at random.  The design states no
+    longest context and no end-of-sequence token; `max_position_embeddings` and `eos_token_id` are read if a file has them."""
+
+    width: int = 0
+    norm_eps: float = 0.0
+    layers: list = None
+
+    MODEL_TYPES: ClassVar[tuple[str, ...]] = ("pisatar",)
+    NO_CONTEXT_LIMIT: ClassVar[int] = 1 << 22
+    MIXERS: ClassVar[tuple[str, ...]] = ("retention", "channel_delta", "parallel")
+
+    @staticmethod
+    def _object(raw: dict, key: str, where: str) -> dict:
+        value = raw.get(key)
+        if not isinstance(value, dict):
+            raise InvalidRequest(f"config.json: {where}.{key} must be an object")
+        return value
+
+    @classmethod
+    def _rotation(cls, mixer: dict, where: str, scaled: bool) -> dict:
+        rot = cls._object(mixer, "rot", where)
+        out = {"base": _require(rot, "base", float, "rotary base"), "dims": _require(rot, "dims", int, "rotated elements")}
+        if scaled and rot.get("scaling") is not None:
+            scaling = cls._object(rot, "scaling", f"{where}.rot")
+            out["scaling"] = {key: _require(scaling, key, float, f"{where}.rot.scaling") for key in ("factor", "low", "high", "original")}
+        return out
+
+    @classmethod
+    def _mixer(cls, i: int, kind: str, mixer: dict) -> dict:
+        where = f"layers[{i}].mixer"
+        if kind == "retention":
+            out = {key: _require(mixer, key, int, where) for key in ("heads", "dim", "vdim")}
+            decay = mixer.get("decay")
+            if not isinstance(decay, list) or any(isinstance(x, bool) or not isinstance(x, (int, float)) for x in decay):
+                raise InvalidRequest(f"config.json: {where}.decay must be a list of numbers")
+            out["decay"] = [float(x) for x in decay]
+            out["rot"] = cls._rotation(mixer, where, False)
+            return out
+        if kind == "channel_delta":
+            out = {key: _require(mixer, key, int, where) for key in ("heads", "kv_heads", "dim", "vdim", "conv")}
+            for key in ("decay_rank", "gate_rank"):          # not keys of the design: for models without a checkpoint
+                if mixer.get(key) is not None:
+                    out[key] = _require(mixer, key, int, "inner size of a thin product")
+            return out
+        left, right = cls._object(mixer, "left", where), cls._object(mixer, "right", where)
+        out = {"left": {key: _require(left, key, int, f"{where}.left") for key in ("heads", "kv_heads", "dim", "vdim")},
+               "right": {key: _require(right, key, int, f"{where}.right") for key in ("heads", "dim", "vdim")}}
+        out["left"]["scale"] = _require(left, "scale", float, f"{where}.left")
+        out["left"]["rot"] = cls._rotation(left, f"{where}.left", True)
+        out["right"]["gate_cap"] = _require(right, "gate_cap", float, f"{where}.right")
+        for key in ("left_scale", "right_scale"):
+            out[key] = _require(mixer, key, float, where)
+        return out
+
+    @classmethod
+    def from_dict(cls, raw: dict) -> "PisatarConfig":
+        norm = cls._object(raw, "norm", "config")
+        layers = raw.get("layers")
+        if not isinstance(layers, list) or not layers:
+            raise InvalidRequest("config.json: `layers` must be a list of layers")
+        read = []
+        for i, layer in enumerate(layers):
+            if not isinstance(layer, dict):
+                raise InvalidRequest(f"config.json: layers[{i}] must be an object")
+            kind = _require(layer, "type", str, f"mixer of layer {i}")
+            if kind not in cls.MIXERS:
+                raise InvalidRequest(f"config.json: layers[{i}].type {kind!r}; known: {', '.join(cls.MIXERS)}")
+            entry = {"type": kind, "mixer": cls._mixer(i, kind, cls._object(layer, "mixer", f"layers[{i}]")), "mlp": None}
+            if layer.get("mlp") is not None:
+                mlp = cls._object(layer, "mlp", f"layers[{i}]")
+                entry["mlp"] = {"kind": _require(mlp, "kind", str, "feed-forward kind"), "ff": _require(mlp, "ff", int, "feed-forward width")}
+            if layer.get("weights_of") is not None:
+                entry["weights_of"] = _require(layer, "weights_of", int, "the layer whose weights are used")
+            read.append(entry)
+        cfg = cls(model_type="pisatar", architectures=["Pisatar"], vocab_size=_require(raw, "vocab", int, "vocabulary"),
+                  max_position_embeddings=int(raw.get("max_position_embeddings") or cls.NO_CONTEXT_LIMIT),
+                  eos_token_id=raw.get("eos_token_id"), width=_require(raw, "width", int, "model width"),
+                  norm_eps=_require(norm, "eps", float, "norm epsilon"), layers=read)
+        cfg.validate()
+        return cfg
+
+    def weights_layer(self, i: int) -> int:
+        """The layer that owns the tensors layer i runs with."""
+        seen = [i]
+        while self.layers[seen[-1]].get("weights_of") is not None:
+            j = self.layers[seen[-1]]["weights_of"]
+            if not 0 <= j < len(self.layers) or j in seen:
+                raise InvalidRequest(f"layers[{i}].weights_of must lead to a layer with weights of its own")
+            seen.append(j)
+        return seen[-1]
+
+    @staticmethod
+    def _check_rotation(rot: dict, dim: int, where: str) -> None:
+        if rot["dims"] < 0 or rot["dims"] % 2 or rot["dims"] > dim or not rot["base"] > 0:
+            raise InvalidRequest(f"{where}.rot: an even number of elements, at most dim, and a positive base")
+        scaling = rot.get("scaling")
+        if scaling is not None and (min(scaling.values()) <= 0 or scaling["high"] < scaling["low"]):
+            raise InvalidRequest(f"{where}.rot.scaling: positive numbers, low at most high")
+
+    def validate(self) -> None:
+        if self.vocab_size <= 0 or self.width <= 0 or self.max_position_embeddings <= 0:
+            raise InvalidRequest("invalid Pisatar dimensions: every size must be a positive integer")
+        if not math.isfinite(self.norm_eps) or self.norm_eps <= 0:
+            raise InvalidRequest("invalid normalization parameters")
+        for i, layer in enumerate(self.layers):
+            m, where = layer["mixer"], f"layers[{i}].mixer"
+            parts = [(where, m)] if layer["type"] != "parallel" else [(f"{where}.left", m["left"]), (f"{where}.right", m["right"])]
+            for at, part in parts:
+                for key in ("heads", "kv_heads", "dim", "vdim", "conv", "decay_rank", "gate_rank"):
+                    if key in part and part[key] <= 0:
+                        raise InvalidRequest(f"{at}.{key} must be positive")
+                if "kv_heads" in part and part["heads"] % part["kv_heads"]:
+                    raise InvalidRequest(f"{at}: heads must be a multiple of kv_heads")
+                if "rot" in part:
+                    self._check_rotation(part["rot"], part["dim"], at)
+            if layer["type"] == "retention":
+                if len(m["decay"]) != m["heads"] or not all(math.isfinite(x) and 0 <= x <= 1 for x in m["decay"]):
+                    raise InvalidRequest(f"{where}.decay: one number from 0 to 1 a head")
+            elif layer["type"] == "parallel":
+                if max(m["left"]["dim"], m["left"]["vdim"]) > 256:
+                    raise InvalidRequest(f"{where}.left: heads have at most 256 elements")
+                if not m["left"]["scale"] > 0 or not m["right"]["gate_cap"] > 0:
+                    raise InvalidRequest(f"{where}: the scores' scale and the gates' cap must be positive")
+                if not math.isfinite(m["left_scale"]) or not math.isfinite(m["right_scale"]):
+                    raise InvalidRequest(f"{where}: left_scale and right_scale must be finite")
+            elif ("decay_rank" in m) != ("gate_rank" in m):
+                raise InvalidRequest(f"{where}: decay_rank and gate_rank are given together")
+            mlp = layer["mlp"]
+            if mlp is not None and (mlp["kind"] != "dense" or mlp["ff"] <= 0):
+                raise InvalidRequest(f"layers[{i}].mlp: only kind `dense` with a positive `ff` is built")
+            owner = self.layers[self.weights_layer(i)]
+            if any(owner[key] != layer[key] for key in ("type", "mixer", "mlp")):
+                raise InvalidRequest(f"layers[{i}]: a layer with another one's weights has that layer's type, mixer and feed-forward")
+        if self.eos_token_id is not None:
+            self.eos_ids()
+
+    def eos_ids(self, folder: str | None = None) -> list[int]:
+        if self.eos_token_id is None and (folder is None or not os.path.exists(os.path.join(folder, "generation_config.json"))):
+            return []                # the design names no end-of-sequence token: generation ends by length
+        return super().eos_ids(folder)
+
+    def to_dict(self) -> dict:
+        out = {"architecture": "Pisatar", "vocab": self.vocab_size, "width": self.width, "norm": {"eps": self.norm_eps},
+               "layers": self.layers}
+        if self.max_position_embeddings != self.NO_CONTEXT_LIMIT:
+            out["max_position_embeddings"] = self.max_position_embeddings
+        if self.eos_token_id is not None:
+            out["eos_token_id"] = self.eos_token_id
+        return out

@@ -188,6 +188,7 @@ LATENT_KERNEL_SOURCES = ("latent_elementwise.cu",)
 EXPERT_KERNEL_SOURCES = ("experts.cu", "experts_mma.cu")
 PARALLEL_KERNEL_SOURCES = ("parallel_elementwise.cu",)
 DELTA_KERNEL_SOURCES = ("delta_rule.cu",)
+LINEAR_SCAN_KERNEL_SOURCES = ("linear_scan.cu",)
 ROTARY_KERNEL_SOURCES = ("rotary_store.cu", "stream_entry.cu")
 
 
@@ -229,6 +230,12 @@ def delta_kernel_library() -> ctypes.CDLL:
     return _kernel_group("delta", "mrs_delta", DELTA_KERNEL_SOURCES)
 
 
+def linear_scan_kernel_library() -> ctypes.CDLL:
+    """The kernels of recurrences that are linear in their state (every size at run time); compiled when a model first needs
+    them."""
+    return _kernel_group("linear_scan", "mrs_linear_scan", LINEAR_SCAN_KERNEL_SOURCES)
+
+
 def rotary_kernel_library() -> ctypes.CDLL:
     """The kernels of rotated and normed heads on their way into the cache, of embeddings with a table of token pairs and
     of a stream that is joined with another before a product (every size at run time); compiled when a model first needs
@@ -266,7 +273,7 @@ SPECIALISED_BUILDS = tuple((lambda d=d: specialised_kernel_library("attention_mm
     tuple((lambda d=d: specialised_kernel_library("attention_prefill_tc.cu", {"MRS_HEAD_DIM": d})) for d in (64, 128)) + \
     (lambda: specialised_kernel_library("gemm_tc.cu", {}), lambda: specialised_kernel_library("gemm_many_rows.cu", {}),
      hybrid_kernel_library, latent_kernel_library, expert_kernel_library, parallel_kernel_library, delta_kernel_library,
-     rotary_kernel_library,
+     linear_scan_kernel_library, rotary_kernel_library,
      biased_attention_library,
      lambda: specialised_kernel_library("attention_biased_mma.cu", {"MRS_HEAD_DIM": 128, "MRS_VALUE_DIM": 128}),
      lambda: specialised_kernel_library("attention_biased_mma.cu", {"MRS_HEAD_DIM": 64, "MRS_VALUE_DIM": 32}),

@@ -4,18 +4,20 @@
 //     S <- g_t S;   u_t = beta_t (v_t - S^T k_t);   S <- S + k_t u_t^T;   o_t = S^T q_t
 //
 // with q_t, k_t [d] (shared by the query heads of a group) made unit vectors, x / sqrt(sum x^2 + unit_eps), q also times
-// a constant; beta_t = sigmoid(b_t); g_t = exp(-exp(A_log_h) softplus(a_t + dt_bias_h)).  Afterwards every head's o_t is
-// divided by its root mean square, multiplied by a weight and by silu of a gate.
+// a constant; beta_t = sigmoid(b_t); g_t = exp(-exp(A_log_h) softplus(a_t + dt_bias_h)), one a head, or one a head and key
+// channel (g_t [d] then acts on the rows of S).  Afterwards every head's o_t is divided by its root mean square, multiplied
+// by a weight and by silu or sigmoid of a gate.
 //
 // Everything here is float32: unit norms, step sizes, decays, the state and the read-out.  S lives in the request's
 // state slot between steps [slots, heads, d, e]; where a sequence starts at position 0 its state counts as zero, whatever
 // the slot held (slots are used again).  State slot -1: a padding sequence, nothing is read or written.  The step's
 // facts come from device arrays only, so a step can be recorded.
 //
-//   delta_prepare     per token: q and k of every group to unit length in place; beta and g of every head
+//   delta_prepare     per token: q and k of every group to unit length in place; beta and g of every head (or beta, and in
+//                     place the g of every head and channel)
 //   delta_scan        the recurrence token by token; one block a (sequence, head, slice of S's columns), the tokens'
 //                     inputs staged through shared memory ahead of their use
-//   head_norm_gate    o / rms(o) * weight * silu(gate) per (token, head)
+//   head_norm_gate    o / rms(o) * weight * act(gate) per (token, head), o first divided by a normaliser where there is one
 #include "common.cuh"
 
 namespace {
@@ -24,10 +26,12 @@ __device__ __forceinline__ float softplus_f(float x) { return fmaxf(x, 0.0f) + l
 
 // qkv [tokens, 2 * groups * d + heads * e] float32: q of every group, k of every group, v of every head.
 // raw [tokens, raw_stride] float32: at column b_offset one b a head, at a_offset one a a head.
-// coef [tokens, 2 * heads]: beta, then g.
+// coef [tokens, 2 * heads]: beta, then g.  With `channels` (rows of `channels_stride` floats, heads * d columns of raw decays,
+// dt_bias one a column) the decays are made there in place and coef is [tokens, heads]: beta.
 __global__ void delta_prepare_kernel(float* __restrict__ qkv, int qkv_width, const float* __restrict__ raw, int raw_stride,
                                      int b_offset, int a_offset, const float* __restrict__ a_log, const float* __restrict__ dt_bias,
-                                     float* __restrict__ coef, int groups, int d, int heads, float unit_eps, float q_factor) {
+                                     float* __restrict__ coef, float* __restrict__ channels, int channels_stride, int groups, int d,
+                                     int heads, float unit_eps, float q_factor) {
     pdl_launch_dependents();
     pdl_wait();
     const size_t t = blockIdx.x;
@@ -41,6 +45,15 @@ __global__ void delta_prepare_kernel(float* __restrict__ qkv, int qkv_width, con
         for (int i = lane; i < d; i += 32) x[i] *= factor;
     }
     const float* r = raw + t * raw_stride;
+    if (channels) {
+        for (int h = threadIdx.x; h < heads; h += blockDim.x) coef[t * heads + h] = 1.0f / (1.0f + expf(-r[b_offset + h]));
+        float* z = channels + t * channels_stride;
+        for (int h = warp; h < heads; h += warps) {
+            const float rate = -expf(a_log[h]);
+            for (int i = h * d + lane; i < (h + 1) * d; i += 32) z[i] = expf(rate * softplus_f(z[i] + dt_bias[i]));
+        }
+        return;
+    }
     for (int h = threadIdx.x; h < heads; h += blockDim.x) {
         coef[t * 2 * heads + h] = 1.0f / (1.0f + expf(-r[b_offset + h]));
         coef[t * 2 * heads + heads + h] = expf(-expf(a_log[h]) * softplus_f(r[a_offset + h] + dt_bias[h]));
@@ -60,9 +73,9 @@ template <int N> __device__ __forceinline__ void copy_async_wait() { asm volatil
 // Thread (column c of the block's slice, part p): rows p * PER .. p * PER + PER - 1 of column c of S in registers (PER is
 // 16 or 8, the launcher's choice); the
 // PARTS lanes of one column are neighbours, so that the two sums over d are log2(PARTS) shuffles.  The tokens' inputs (k and
-// q of the head's group, the slice of v, beta and g) come in batches of `batch_tokens` through two stages of shared memory:
+// q of the head's group, the slice of v, beta and g; CHANNEL: also the head's d decays) come in batches of `batch_tokens` through two stages of shared memory:
 // the next batch is copied while this one is computed, and the threads of a block share what they read.  A token in shared
-// memory: k [PARTS * PITCH] | q [PARTS * PITCH] | v [cols rounded up to 4] | beta, g, 0, 0, with PITCH = PER + 4, so that
+// memory: k [PARTS * PITCH] | q [PARTS * PITCH] (| decays [PARTS * PITCH]) | v [cols rounded up to 4] | beta, g, 0, 0, with PITCH = PER + 4, so that
 // the 16-byte reads of the parts fall on different banks; the rows beyond d stay zero.
 //
 // One warp a scheduler is all that a single sequence offers, so every instruction's latency shows.  What a thread copies is
@@ -74,18 +87,20 @@ struct Copies {
     int src[N], dst[N], token[N];      // offsets in floats from the batch's first row and from the stage; a huge token: none
 };
 
-template <int PER, int PARTS>
+template <int PER, int PARTS, bool CHANNEL>
 __global__ void __launch_bounds__(128) delta_scan_kernel(const float* __restrict__ qkv, int qkv_width, const float* __restrict__ coef,
+                                  const float* __restrict__ channels, int channels_stride,
                                   float* __restrict__ state, long long state_stride, const int* __restrict__ positions,
                                   const int* __restrict__ q_start, const int* __restrict__ state_slots, float* __restrict__ out,
                                   int heads, int groups, int d, int e, int cols, int batch_tokens, int wide_copies,
                                   int write_state) {
     extern __shared__ __align__(16) float stage[];
-    constexpr int PITCH = PER + 4, ROWS = PARTS * PITCH;
+    constexpr int PITCH = PER + 4, ROWS = PARTS * PITCH, VECTORS = CHANNEL ? 3 : 2;
+    constexpr int FACTS = CHANNEL ? 1 : 2;                 // beta, and the decay of the head
     constexpr int WIDE = 8, NARROW = 3;                    // copies a thread and batch that are worked out ahead
     pdl_launch_dependents();
     const int cols_pad = (cols + 3) & ~3;
-    const int token_floats = 2 * ROWS + cols_pad + 4, stage_floats = batch_tokens * token_floats;
+    const int token_floats = VECTORS * ROWS + cols_pad + 4, stage_floats = batch_tokens * token_floats;
     for (int i = threadIdx.x; i < 2 * stage_floats; i += blockDim.x) stage[i] = 0.0f;
     __syncthreads();
     pdl_wait();
@@ -106,24 +121,25 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(const float* __restrict
 
     const int q_at = group * d, k_at = (groups + group) * d, v_at = 2 * groups * d + head * e + (int)blockIdx.z * cols;
     const int live_cols = min(cols, e - (int)blockIdx.z * cols);
-    // copy number i of a batch's keys and queries: token j, k or q, elements el .. of the vector
-    const int width = wide_copies ? d >> 2 : d, vector_copies = batch_tokens * 2 * width;
+    // copy number i of a batch's keys and queries (and decays): token j, k, q or decays, elements el .. of the vector
+    const int width = wide_copies ? d >> 2 : d, vector_copies = batch_tokens * VECTORS * width;
     auto vector_copy = [&](int i, int& src, int& dst) {
-        const int j = i / (2 * width), r = i % (2 * width), which = r / width, el = (r % width) * (wide_copies ? 4 : 1);
-        src = j * qkv_width + (which ? q_at : k_at) + el;
+        const int j = i / (VECTORS * width), r = i % (VECTORS * width), which = r / width, el = (r % width) * (wide_copies ? 4 : 1);
+        if (CHANNEL && which == 2) src = -1 - (j * channels_stride + head * d + el);          // below zero: from the decays
+        else src = j * qkv_width + (which ? q_at : k_at) + el;
         dst = j * token_floats + which * ROWS + (el / PER) * PITCH + el % PER;
         return j;
     };
     // copy number i of a batch's values and coefficients: token j, a column of v, beta or g
-    const int scalar_copies = batch_tokens * (live_cols + 2);
+    const int scalar_copies = batch_tokens * (live_cols + FACTS);
     auto scalar_copy = [&](int i, long long& src, int& dst) {
-        const int j = i / (live_cols + 2), r = i % (live_cols + 2);
+        const int j = i / (live_cols + FACTS), r = i % (live_cols + FACTS);
         if (r < live_cols) {
             src = (long long)j * qkv_width + v_at + r;
-            dst = j * token_floats + 2 * ROWS + r;
+            dst = j * token_floats + VECTORS * ROWS + r;
         } else {
-            src = -1 - ((long long)j * 2 * heads + (r == live_cols ? head : heads + head));      // below zero: from coef
-            dst = j * token_floats + 2 * ROWS + cols_pad + (r - live_cols);
+            src = -1 - ((long long)j * FACTS * heads + (r == live_cols ? head : heads + head));      // below zero: from coef
+            dst = j * token_floats + VECTORS * ROWS + cols_pad + (r - live_cols);
         }
         return j;
     };
@@ -134,28 +150,31 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(const float* __restrict
 #pragma unroll
     for (int i = 0; i < WIDE; ++i) {
         const int at = threadIdx.x + i * blockDim.x;
-        wide.token[i] = at < longest * 2 * width ? vector_copy(at, wide.src[i], wide.dst[i]) : (1 << 30);
+        wide.token[i] = at < longest * VECTORS * width ? vector_copy(at, wide.src[i], wide.dst[i]) : (1 << 30);
     }
 #pragma unroll
     for (int i = 0; i < NARROW; ++i) {
         const int at = threadIdx.x + i * blockDim.x;
-        narrow.token[i] = at < longest * (live_cols + 2) ? scalar_copy(at, narrow_src[i], narrow.dst[i]) : (1 << 30);
+        narrow.token[i] = at < longest * (live_cols + FACTS) ? scalar_copy(at, narrow_src[i], narrow.dst[i]) : (1 << 30);
     }
     auto issue = [&](int t0, int n, int buffer) {
         float* base = stage + buffer * stage_floats;
         const float* rows = qkv + (size_t)t0 * qkv_width;
-        const float* facts = coef + (size_t)t0 * 2 * heads;
+        const float* facts = coef + (size_t)t0 * FACTS * heads;
+        const float* fades = CHANNEL ? channels + (size_t)t0 * channels_stride : nullptr;
 #pragma unroll
         for (int i = 0; i < WIDE; ++i)
             if (wide.token[i] < n) {
-                if (wide_copies) copy_async16(base + wide.dst[i], rows + wide.src[i]);
-                else copy_async4(base + wide.dst[i], rows + wide.src[i]);
+                const float* from = CHANNEL && wide.src[i] < 0 ? fades + (-1 - wide.src[i]) : rows + wide.src[i];
+                if (wide_copies) copy_async16(base + wide.dst[i], from);
+                else copy_async4(base + wide.dst[i], from);
             }
         for (int at = threadIdx.x + WIDE * blockDim.x; at < vector_copies; at += blockDim.x) {      // sizes beyond the usual
             int src, dst;
             if (vector_copy(at, src, dst) < n) {
-                if (wide_copies) copy_async16(base + dst, rows + src);
-                else copy_async4(base + dst, rows + src);
+                const float* from = CHANNEL && src < 0 ? fades + (-1 - src) : rows + src;
+                if (wide_copies) copy_async16(base + dst, from);
+                else copy_async4(base + dst, from);
             }
         }
 #pragma unroll
@@ -169,7 +188,7 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(const float* __restrict
         copy_async_commit();
     };
     const int batches = (last - first + batch_tokens - 1) / batch_tokens;
-    const int token_tail = 2 * ROWS + cols_pad;
+    const int token_tail = VECTORS * ROWS + cols_pad;
     float* out_at = out + (size_t)first * heads * e + (size_t)head * e + c;
     const size_t out_step = (size_t)heads * e;
     const bool writes = live && part == 0;
@@ -186,16 +205,24 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(const float* __restrict
         const float* token = stage + (b & 1) * stage_floats + part * PITCH;
 #pragma unroll 2
         for (int j = 0; j < n; ++j, token += token_floats, out_at += out_step) {
-            float k[PER], q[PER];
+            float k[PER], q[PER], fade[CHANNEL ? PER : 1];
 #pragma unroll
             for (int i = 0; i < PER; i += 4) {
+                if (CHANNEL) {
+                    const float4 ff = *reinterpret_cast<const float4*>(token + 2 * ROWS + i);
+                    fade[i] = ff.x, fade[i + 1] = ff.y, fade[i + 2] = ff.z, fade[i + 3] = ff.w;
+                }
                 const float4 kk = *reinterpret_cast<const float4*>(token + i);
                 const float4 qq = *reinterpret_cast<const float4*>(token + ROWS + i);
                 k[i] = kk.x, k[i + 1] = kk.y, k[i + 2] = kk.z, k[i + 3] = kk.w;
                 q[i] = qq.x, q[i + 1] = qq.y, q[i + 2] = qq.z, q[i + 3] = qq.w;
             }
             const float* tail = token - part * PITCH + token_tail;
-            const float v = (tail - cols_pad)[col_in_slice], beta = tail[0], decay = tail[1];
+            const float v = (tail - cols_pad)[col_in_slice], beta = tail[0], decay = CHANNEL ? 1.0f : tail[1];
+            if (CHANNEL) {                                               // S forgets before the correction reads it
+#pragma unroll
+                for (int i = 0; i < PER; ++i) s[i] *= fade[i];
+            }
             float r4[4] = {0.0f, 0.0f, 0.0f, 0.0f};
 #pragma unroll
             for (int i = 0; i < PER; ++i) r4[i & 3] = fmaf(s[i], k[i], r4[i & 3]);
@@ -203,7 +230,8 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(const float* __restrict
 #pragma unroll
             for (int o = PARTS >> 1; o > 0; o >>= 1) r += __shfl_xor_sync(0xffffffffu, r, o);
 #pragma unroll
-            for (int i = 0; i < PER; ++i) s[i] *= decay;                 // beside the shuffles, off the chain
+            for (int i = 0; i < PER; ++i)
+                if (!CHANNEL) s[i] *= decay;                             // beside the shuffles, off the chain
             const float u = beta * (v - decay * r);
             float y4[4] = {0.0f, 0.0f, 0.0f, 0.0f};
 #pragma unroll
@@ -225,43 +253,121 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(const float* __restrict
     }
 }
 
-// One warp a (token, head): out = o / sqrt(mean(o^2) + eps) * weight * silu(gate).  o [tokens, heads * e] float32; gate a
-// column range of wider float32 rows; weight [e], shared by the heads.
-template <typename T>
-__global__ void head_norm_gate_kernel(const float* __restrict__ o, const float* __restrict__ gate, int gate_stride,
-                                      const float* __restrict__ weight, float eps, T* __restrict__ out, int tokens, int heads, int e) {
+// One warp a (token, head): x = o * factor (/ (max(|c * factor|, floor) + floor_eps) where there is a normaliser c), then
+// out = x / sqrt(mean(x^2) + eps) * weight * act(gate), act = silu or (SIGMOID) the sigmoid.  o [tokens, heads * e] float32;
+// gate a column range of wider float32 rows; weight [e] shared by the heads (weight_stride 0), [heads, e] (weight_stride e) or
+// null; c [tokens, heads], floor [tokens, floor_stride] from its first column on.
+struct HeadNorm {
+    const float *o, *gate, *weight, *c, *floor;
+    int gate_stride, weight_stride, floor_stride, tokens, heads, e;
+    float eps, factor, floor_eps;
+};
+
+template <bool SIGMOID> __device__ __forceinline__ float gate_of(float g) {
+    const float s = 1.0f / (1.0f + expf(-g));
+    return SIGMOID ? s : g * s;
+}
+
+__device__ __forceinline__ float head_factor(const HeadNorm& A, size_t t, int h) {
+    if (!A.c) return A.factor;
+    return A.factor / (fmaxf(fabsf(A.c[t * A.heads + h] * A.factor), A.floor[t * A.floor_stride + h]) + A.floor_eps);
+}
+
+template <typename T, bool SIGMOID>
+__global__ void head_norm_gate_kernel(const HeadNorm A, T* __restrict__ out) {
     pdl_launch_dependents();
     pdl_wait();
-    const int lane = threadIdx.x & 31;
+    const int lane = threadIdx.x & 31, e = A.e;
     const long long unit = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
-    if (unit >= (long long)tokens * heads) return;
-    const size_t t = (size_t)(unit / heads);
-    const int h = (int)(unit % heads);
-    const float* x = o + t * heads * e + (size_t)h * e;
-    const float* g = gate + t * gate_stride + (size_t)h * e;
+    if (unit >= (long long)A.tokens * A.heads) return;
+    const size_t t = (size_t)(unit / A.heads);
+    const int h = (int)(unit % A.heads);
+    const float* x = A.o + t * A.heads * e + (size_t)h * e;
+    const float* g = A.gate + t * A.gate_stride + (size_t)h * e;
+    const float* w = A.weight ? A.weight + (size_t)h * A.weight_stride : nullptr;
+    const float factor = head_factor(A, t, h);
     float sum = 0.0f;
-    for (int i = lane; i < e; i += 32) sum += x[i] * x[i];
-    const float scale = 1.0f / sqrtf(warp_sum(sum) / (float)e + eps);
-    T* dst = out + t * heads * e + (size_t)h * e;
-    for (int i = lane; i < e; i += 32) dst[i] = from_float<T>(x[i] * scale * weight[i] * (g[i] / (1.0f + expf(-g[i]))));
+    for (int i = lane; i < e; i += 32) sum += (x[i] * factor) * (x[i] * factor);
+    const float scale = 1.0f / sqrtf(warp_sum(sum) / (float)e + A.eps);
+    T* dst = out + t * A.heads * e + (size_t)h * e;
+    for (int i = lane; i < e; i += 32) {
+        const float y = x[i] * factor * scale;
+        dst[i] = from_float<T>((w ? y * w[i] : y) * gate_of<SIGMOID>(g[i]));
+    }
+}
+
+template <typename T> __device__ __forceinline__ void put_four(T* p, float4 v);
+template <> __device__ __forceinline__ void put_four<float>(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+template <> __device__ __forceinline__ void put_four<bf16>(bf16* p, float4 v) {
+    __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+    uint2 raw;
+    raw.x = *reinterpret_cast<uint32_t*>(&lo);
+    raw.y = *reinterpret_cast<uint32_t*>(&hi);
+    *reinterpret_cast<uint2*>(p) = raw;
+}
+
+// Heads of a multiple of four elements in rows on 16-byte boundaries, at most 128 * NV: four elements a lane and access, all of a
+// head's loads in flight together.  LANES lanes a head (32, or 16 for heads of up to 64 elements).
+template <typename T, bool SIGMOID, int NV, int LANES>
+__global__ void head_norm_gate_vec_kernel(const HeadNorm A, T* __restrict__ out) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int lane = threadIdx.x % LANES, e = A.e;
+    const long long units = (long long)A.tokens * A.heads;
+    long long unit = (long long)blockIdx.x * (blockDim.x / LANES) + threadIdx.x / LANES;
+    const bool live = unit < units;
+    if (!live) unit = units - 1;                             // its lanes still take part in the shuffles
+    const size_t t = (size_t)(unit / A.heads);
+    const int h = (int)(unit % A.heads);
+    const float* x = A.o + t * A.heads * e + (size_t)h * e;
+    const float* g = A.gate + t * A.gate_stride + (size_t)h * e;
+    float4 v[NV], gates[NV];
+#pragma unroll
+    for (int j = 0; j < NV; ++j) {
+        const int i = 4 * (lane + j * LANES);
+        v[j] = gates[j] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        if (i < e) v[j] = *reinterpret_cast<const float4*>(x + i), gates[j] = *reinterpret_cast<const float4*>(g + i);
+    }
+    const float factor = head_factor(A, t, h);
+    float sum = 0.0f;
+#pragma unroll
+    for (int j = 0; j < NV; ++j) {
+        v[j].x *= factor, v[j].y *= factor, v[j].z *= factor, v[j].w *= factor;
+        sum += v[j].x * v[j].x + v[j].y * v[j].y + v[j].z * v[j].z + v[j].w * v[j].w;
+    }
+#pragma unroll
+    for (int o = LANES / 2; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+    const float scale = 1.0f / sqrtf(sum / (float)e + A.eps);
+    if (!live) return;
+    T* dst = out + t * A.heads * e + (size_t)h * e;
+#pragma unroll
+    for (int j = 0; j < NV; ++j) {
+        const int i = 4 * (lane + j * LANES);
+        if (i >= e) continue;
+        float4 w = make_float4(1.0f, 1.0f, 1.0f, 1.0f);
+        if (A.weight) w = *reinterpret_cast<const float4*>(A.weight + (size_t)h * A.weight_stride + i);
+        put_four<T>(dst + i, make_float4(v[j].x * scale * w.x * gate_of<SIGMOID>(gates[j].x), v[j].y * scale * w.y * gate_of<SIGMOID>(gates[j].y),
+                                         v[j].z * scale * w.z * gate_of<SIGMOID>(gates[j].z), v[j].w * scale * w.w * gate_of<SIGMOID>(gates[j].w)));
+    }
 }
 
 }  // namespace
 
 MRS_EXPORT int mrs_delta_prepare(float* qkv, const float* raw, int raw_stride, int b_offset, int a_offset, const float* a_log,
-                                 const float* dt_bias, float* coef, int tokens, int groups, int d, int heads, int e, float unit_eps,
-                                 float q_factor, void* stream) {
+                                 const float* dt_bias, float* coef, float* channels, int channels_stride, int tokens, int groups, int d,
+                                 int heads, int e, float unit_eps, float q_factor, void* stream) {
     if (tokens <= 0) return 0;
     if (groups <= 0 || d <= 0 || heads <= 0 || e <= 0 || heads % groups) return MRS_BAD_ARGUMENT;
     const int units = 2 * groups;
     const int threads = units >= 8 ? 256 : (units >= 4 ? 128 : 64);
     MRS_LAUNCH(delta_prepare_kernel, tokens, threads, 0, stream, qkv, 2 * groups * d + heads * e, raw, raw_stride, b_offset, a_offset,
-               a_log, dt_bias, coef, groups, d, heads, unit_eps, q_factor);
+               a_log, dt_bias, coef, channels, channels_stride, groups, d, heads, unit_eps, q_factor);
     MRS_RETURN_LAUNCH_STATUS();
 }
 
 // state [slots, heads, d, e] float32 with `state_stride` floats from slot to slot; out [tokens, heads * e] float32.
-MRS_EXPORT int mrs_delta_scan(const float* qkv, const float* coef, float* state, long long state_stride, const int* positions,
+// `channels`: the decays of every head and channel, rows of `channels_stride` floats (null: one a head, in coef).
+MRS_EXPORT int mrs_delta_scan(const float* qkv, const float* coef, const float* channels, int channels_stride, float* state, long long state_stride, const int* positions,
                               const int* q_start, const int* state_slots, float* out, int tokens, int sequences, int heads,
                               int groups, int d, int e, int write_state, void* stream) {
     if (tokens <= 0 || sequences <= 0) return 0;
@@ -285,41 +391,60 @@ MRS_EXPORT int mrs_delta_scan(const float* qkv, const float* coef, float* state,
     if (d <= 256 && tokens >= 256LL * sequences && pairs * slices > mrs_sm_count()) plan(8);
     if (slices > 65535) return MRS_BAD_ARGUMENT;
     const int qkv_width = 2 * groups * d + heads * e;
-    const int token_floats = 2 * parts * (per + 4) + ((cols + 3) & ~3) + 4;
+    const int token_floats = (channels ? 3 : 2) * parts * (per + 4) + ((cols + 3) & ~3) + 4;
     int batch_tokens = (48 * 1024) / (2 * token_floats * (int)sizeof(float));
     if (batch_tokens > 8) batch_tokens = 8;
     if (batch_tokens < 1) return MRS_BAD_ARGUMENT;
-    const int wide_copies = d % 4 == 0 && qkv_width % 4 == 0 && ((uintptr_t)qkv & 15) == 0;
+    const int wide_copies = d % 4 == 0 && qkv_width % 4 == 0 && ((uintptr_t)qkv & 15) == 0 &&
+                            (!channels || (channels_stride % 4 == 0 && ((uintptr_t)channels & 15) == 0));
     const dim3 grid(sequences, heads, slices);
     const size_t shared = 2 * (size_t)batch_tokens * token_floats * sizeof(float);
-#define MRS_DELTA_SCAN(PER, PARTS)                                                                                                   \
-    MRS_LAUNCH((delta_scan_kernel<PER, PARTS>), grid, cols * PARTS, shared, stream, qkv, qkv_width, coef, state, state_stride,       \
-               positions, q_start, state_slots, out, heads, groups, d, e, cols, batch_tokens, wide_copies, write_state)
-#define MRS_DELTA_SCAN_ROWS(PER)                                                                                                     \
+#define MRS_DELTA_SCAN(PER, PARTS, CHANNEL)                                                                                          \
+    MRS_LAUNCH((delta_scan_kernel<PER, PARTS, CHANNEL>), grid, cols * PARTS, shared, stream, qkv, qkv_width, coef, channels,         \
+               channels_stride, state, state_stride, positions, q_start, state_slots, out, heads, groups, d, e, cols, batch_tokens,  \
+               wide_copies, write_state)
+#define MRS_DELTA_SCAN_ROWS(PER, CHANNEL)                                                                                            \
     switch (parts) {                                                                                                                 \
-        case 1: MRS_DELTA_SCAN(PER, 1); break;                                                                                       \
-        case 2: MRS_DELTA_SCAN(PER, 2); break;                                                                                       \
-        case 4: MRS_DELTA_SCAN(PER, 4); break;                                                                                       \
-        case 8: MRS_DELTA_SCAN(PER, 8); break;                                                                                       \
-        case 16: MRS_DELTA_SCAN(PER, 16); break;                                                                                     \
-        default: MRS_DELTA_SCAN(PER, 32); break;                                                                                     \
+        case 1: MRS_DELTA_SCAN(PER, 1, CHANNEL); break;                                                                              \
+        case 2: MRS_DELTA_SCAN(PER, 2, CHANNEL); break;                                                                              \
+        case 4: MRS_DELTA_SCAN(PER, 4, CHANNEL); break;                                                                              \
+        case 8: MRS_DELTA_SCAN(PER, 8, CHANNEL); break;                                                                              \
+        case 16: MRS_DELTA_SCAN(PER, 16, CHANNEL); break;                                                                            \
+        default: MRS_DELTA_SCAN(PER, 32, CHANNEL); break;                                                                            \
     }
-    if (per == 16) { MRS_DELTA_SCAN_ROWS(16) } else { MRS_DELTA_SCAN_ROWS(8) }
+    if (channels) {
+        if (per == 16) { MRS_DELTA_SCAN_ROWS(16, true) } else { MRS_DELTA_SCAN_ROWS(8, true) }
+    } else {
+        if (per == 16) { MRS_DELTA_SCAN_ROWS(16, false) } else { MRS_DELTA_SCAN_ROWS(8, false) }
+    }
 #undef MRS_DELTA_SCAN_ROWS
 #undef MRS_DELTA_SCAN
     MRS_RETURN_LAUNCH_STATUS();
 }
 
-MRS_EXPORT int mrs_head_norm_gate(int is_bf16, const float* o, const float* gate, int gate_stride, const float* weight, float eps,
-                                  void* out, int tokens, int heads, int e, void* stream) {
+MRS_EXPORT int mrs_head_norm_gate(int is_bf16, const float* o, const float* gate, int gate_stride, int sigmoid, const float* weight,
+                                  int weight_stride, float eps, float factor, const float* c, const float* floor, int floor_stride,
+                                  float floor_eps, void* out, int tokens, int heads, int e, void* stream) {
     if (tokens <= 0) return 0;
-    if (heads <= 0 || e <= 0) return MRS_BAD_ARGUMENT;
-    const int warps = 4;
+    if (heads <= 0 || e <= 0 || (c && !floor)) return MRS_BAD_ARGUMENT;
+    HeadNorm A = {o, gate, weight, c, floor, gate_stride, weight_stride, floor_stride, tokens, heads, e, eps, factor, floor_eps};
     const long long units = (long long)tokens * heads;
-    const unsigned blocks = (unsigned)((units + warps - 1) / warps);
-    if (is_bf16)
-        MRS_LAUNCH(head_norm_gate_kernel<bf16>, blocks, 32 * warps, 0, stream, o, gate, gate_stride, weight, eps, (bf16*)out, tokens, heads, e);
-    else
-        MRS_LAUNCH(head_norm_gate_kernel<float>, blocks, 32 * warps, 0, stream, o, gate, gate_stride, weight, eps, (float*)out, tokens, heads, e);
+    const bool vec = e % 4 == 0 && e <= 512 && gate_stride % 4 == 0 && (((uintptr_t)o | (uintptr_t)gate | (uintptr_t)weight | (uintptr_t)out) & 15) == 0;
+    const int per_block = vec && e <= 64 ? 8 : 4;
+    const unsigned blocks = (unsigned)((units + per_block - 1) / per_block);
+#define MRS_HEAD_NORM(T, SIGMOID)                                                                                                \
+    do {                                                                                                                         \
+        if (!vec) MRS_LAUNCH((head_norm_gate_kernel<T, SIGMOID>), blocks, 128, 0, stream, A, (T*)out);                            \
+        else if (e <= 64) MRS_LAUNCH((head_norm_gate_vec_kernel<T, SIGMOID, 1, 16>), blocks, 128, 0, stream, A, (T*)out);         \
+        else if (e <= 128) MRS_LAUNCH((head_norm_gate_vec_kernel<T, SIGMOID, 1, 32>), blocks, 128, 0, stream, A, (T*)out);        \
+        else if (e <= 256) MRS_LAUNCH((head_norm_gate_vec_kernel<T, SIGMOID, 2, 32>), blocks, 128, 0, stream, A, (T*)out);        \
+        else MRS_LAUNCH((head_norm_gate_vec_kernel<T, SIGMOID, 4, 32>), blocks, 128, 0, stream, A, (T*)out);                      \
+    } while (0)
+    if (is_bf16) {
+        if (sigmoid) MRS_HEAD_NORM(bf16, true); else MRS_HEAD_NORM(bf16, false);
+    } else {
+        if (sigmoid) MRS_HEAD_NORM(float, true); else MRS_HEAD_NORM(float, false);
+    }
+#undef MRS_HEAD_NORM
     MRS_RETURN_LAUNCH_STATUS();
 }

@@ -1,0 +1,511 @@
+// Recurrences that are linear in their state, a matrix S [d, e] per (request, head):
+//
+//     S_t = keep_t S_(t-1) + take_t k_t v_t^T,   o_t = S_t^T q_t          (and with a normaliser n_t likewise with k alone, c_t = n_t . q_t)
+//
+// keep is a constant a head (a retention: take = 1) or comes a token with take (gates of an exponential memory).  Everything
+// here is float32.  S (and n) live in the request's state slot between steps; where a sequence starts at position 0 its
+// state counts as zero, whatever the slot held (slots are used again).  State slot -1: a padding sequence, nothing is read or
+// written.  The step's facts come from device arrays only, so a step can be recorded.
+//
+//   rotate_heads       q and k heads inside the float32 projection turn by their token's position, in place
+//   memory_gates       keep, take and exp(-m) of every (token, head) from the raw gates of an exponential memory with a running
+//                      maximum m (which starts at 0)
+//   linear_scan        the recurrence
+//   narrow_columns     a range of float32 columns as rows of the engine's dtype
+#include "common.cuh"
+
+namespace {
+
+// ---------------------------------------------------------------------------------------------
+// rows [tokens, stride] float32; `heads` heads of d elements from column `offset` on; the first `rot` elements of a head turn:
+// element i with i + rot / 2 by the step's table [tokens, rot / 2, 2] of cosines and sines.  VEC: four pairs a thread.
+// ---------------------------------------------------------------------------------------------
+template <bool VEC>
+__global__ void rotate_heads_kernel(float* __restrict__ rows, int stride, int offset, const float* __restrict__ table, int tokens,
+                                    int heads, int d, int rot) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const size_t t = blockIdx.x;
+    const int half = rot / 2;
+    float* row = rows + t * stride + offset;
+    const float* turn = table + t * (size_t)rot;
+    if (VEC) {
+        const int quads = half >> 2;
+        for (int at = threadIdx.x; at < heads * quads; at += blockDim.x) {
+            const int i = (at % quads) * 4;
+            float* x = row + (size_t)(at / quads) * d + i;
+            const float4 c01 = *reinterpret_cast<const float4*>(turn + 2 * i), c23 = *reinterpret_cast<const float4*>(turn + 2 * i + 4);
+            const float4 u = *reinterpret_cast<const float4*>(x), v = *reinterpret_cast<const float4*>(x + half);
+            *reinterpret_cast<float4*>(x) = make_float4(u.x * c01.x - v.x * c01.y, u.y * c01.z - v.y * c01.w, u.z * c23.x - v.z * c23.y,
+                                                        u.w * c23.z - v.w * c23.w);
+            *reinterpret_cast<float4*>(x + half) = make_float4(v.x * c01.x + u.x * c01.y, v.y * c01.z + u.y * c01.w,
+                                                               v.z * c23.x + u.z * c23.y, v.w * c23.z + u.w * c23.w);
+        }
+    } else {
+        for (int at = threadIdx.x; at < heads * half; at += blockDim.x) {
+            const int i = at % half;
+            float* x = row + (size_t)(at / half) * d + i;
+            const float c = turn[2 * i], s = turn[2 * i + 1], u = x[0], v = x[half];
+            x[0] = u * c - v * s;
+            x[half] = v * c + u * s;
+        }
+    }
+}
+
+template <typename T>
+__global__ void narrow_columns_kernel(const float* __restrict__ rows, int stride, int offset, T* __restrict__ out, long long total, int columns,
+                                      int live) {
+    pdl_launch_dependents();
+    pdl_wait();
+    for (long long at = (long long)blockIdx.x * blockDim.x + threadIdx.x; at < total; at += (long long)gridDim.x * blockDim.x) {
+        const long long t = at / columns;
+        const int c = (int)(at % columns);
+        out[at] = from_float<T>(c < live ? rows[t * stride + offset + c] : 0.0f);
+    }
+}
+
+// ---------------------------------------------------------------------------------------------
+// Gates of an exponential memory.  Per head: i = cap tanh((raw_i + bias_i) / cap), f = logsigmoid(cap tanh((raw_f + bias_f) / cap)),
+// m_t = max(f_t + m_(t-1), i_t); keep_t = exp(f_t + m_(t-1) - m_t), take_t = exp(i_t - m_t), floor_t = exp(-m_t).
+// One block a (sequence, head); a block's worth of tokens at a time by a scan over the maps m -> max(A + m, B), whose
+// composition is (A1, B1) then (A2, B2) = (A1 + A2, max(B1 + A2, B2)).  coef [tokens, 3 heads]: keep | take | floor.
+// ---------------------------------------------------------------------------------------------
+__device__ __forceinline__ float log_sigmoid_f(float x) { return fminf(x, 0.0f) - log1pf(expf(-fabsf(x))); }
+
+__global__ void memory_gates_kernel(const float* __restrict__ raw, int raw_stride, int i_offset, int f_offset,
+                                    const float* __restrict__ i_bias, const float* __restrict__ f_bias, float cap,
+                                    float* __restrict__ m_state, long long state_stride, const int* __restrict__ positions,
+                                    const int* __restrict__ q_start, const int* __restrict__ state_slots, float* __restrict__ coef,
+                                    int heads, int write_state) {
+    pdl_launch_dependents();
+    pdl_wait();
+    __shared__ float total_a[32], total_b[32], carried;
+    const int seq = blockIdx.x, head = blockIdx.y;
+    const int first = q_start[seq], last = q_start[seq + 1];
+    const int slot = state_slots[seq];
+    if (slot < 0 || last <= first) return;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    float* mine = m_state + (long long)slot * state_stride + head;
+    float m0 = positions[first] == 0 ? 0.0f : *mine;
+    const float bi = i_bias[head], bf = f_bias[head];
+    for (int base = first; base < last; base += blockDim.x) {
+        const int t = base + threadIdx.x;
+        const bool live = t < last;
+        float in = 0.0f, keep = 0.0f;
+        if (live) {
+            const float* r = raw + (size_t)t * raw_stride;
+            in = cap * tanhf((r[i_offset + head] + bi) / cap);
+            keep = log_sigmoid_f(cap * tanhf((r[f_offset + head] + bf) / cap));
+        }
+        float a = live ? keep : 0.0f, b = live ? in : -CUDART_INF_F;
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+            const float a1 = __shfl_up_sync(0xffffffffu, a, o), b1 = __shfl_up_sync(0xffffffffu, b, o);
+            if (lane >= o) {
+                b = fmaxf(b1 + a, b);
+                a += a1;
+            }
+        }
+        if (lane == 31) total_a[warp] = a, total_b[warp] = b;
+        __syncthreads();
+        float before = m0;                                   // m ahead of this warp's first token
+        for (int w = 0; w < warp; ++w) before = fmaxf(total_a[w] + before, total_b[w]);
+        const float m = fmaxf(a + before, b);
+        float previous = __shfl_up_sync(0xffffffffu, m, 1);
+        if (lane == 0) previous = before;
+        if (live) {
+            float* c = coef + (size_t)t * 3 * heads + head;
+            c[0] = expf(keep + previous - m);
+            c[heads] = expf(in - m);
+            c[2 * heads] = expf(-m);
+            if (t == last - 1 || threadIdx.x == blockDim.x - 1) carried = m;
+        }
+        __syncthreads();
+        m0 = carried;
+    }
+    if (write_state && threadIdx.x == 0) *mine = m0;
+}
+
+// ---------------------------------------------------------------------------------------------
+// The recurrence.  A thread keeps SCAN_ROWS rows x 4 neighbouring columns of S in registers; the PARTS lanes that share four
+// columns cover the d rows, so what a thread reads of k and q from shared memory serves four columns, and a token's
+// read-out is a reduction that hands its columns out while it sums (2 + 1 + 1 ... shuffles).  The tokens' k, q, v and gates
+// come through two stages of shared memory, filled by cp.async a batch ahead.
+//
+// The decay costs no instruction an element: with P the product of the keeps since S was last rescaled, the registers hold
+// S / P, a token adds (take / P) k v^T and its read-out is P (S / P)^T q; where P falls below SCAN_LEAST the registers are
+// multiplied by it and P starts again at 1.
+//
+// SCAN_WHOLE: a sequence's rows in one go, from the slot's state to the slot's state.  Long portions of few sequences are cut
+// into chunks of `chunk_len` rows that run side by side: SCAN_LOCAL runs every chunk from zero and leaves its end state and
+// the product of its keeps in scratch, scan_chunk_states walks a sequence's chunks once and turns the end states into the
+// state at every chunk's start (and the slot's new state), SCAN_FINAL runs every chunk from there and writes o.
+// ---------------------------------------------------------------------------------------------
+#define SCAN_ROWS 16
+#define SCAN_PITCH (SCAN_ROWS + 4)       // 16-byte reads of the parts fall on different banks
+#define SCAN_LEAST 1e-8f
+enum { SCAN_WHOLE = 0, SCAN_LOCAL = 1, SCAN_FINAL = 2 };
+
+struct ScanArgs {
+    const float *q, *k, *v;              // columns of float32 rows of `stride` floats; heads of d, d and e elements
+    int stride;
+    const float* decay;                  // [heads], or null: the coefficients
+    const float* coef;                   // [tokens, coef_stride]: keep of every head, then take
+    int coef_stride;
+    float* state;                        // [slots][heads, d, e]
+    float* norm_state;                   // [slots][heads, d], or null: no normaliser
+    long long state_stride;
+    const int *positions, *q_start, *state_slots;
+    float* out;                          // [tokens, heads * e]
+    float* norm_out;                     // [tokens, heads]
+    int heads, d, e, cols, slices, batch, write_state, vec_qk, vec_v, vec_state, vec_out;
+    float *chunk_state, *chunk_decay;
+    int chunk_len, max_chunks, chunk_floats;
+};
+
+__device__ __forceinline__ void scan_copy16(float* to, const float* from) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"((uint32_t)__cvta_generic_to_shared(to)), "l"(from));
+}
+__device__ __forceinline__ void scan_copy4(float* to, const float* from) {
+    asm volatile("cp.async.ca.shared.global [%0], [%1], 4;\n" ::"r"((uint32_t)__cvta_generic_to_shared(to)), "l"(from));
+}
+
+template <int MODE, int PARTS>
+__global__ void __launch_bounds__(256) linear_scan_kernel(const ScanArgs A) {
+    extern __shared__ __align__(16) float stage[];
+    constexpr int GROUPS = 32 / PARTS;                       // groups of four columns a warp covers
+    constexpr int VECTOR = PARTS * SCAN_PITCH;               // floats of a k (or q) in shared memory
+    pdl_launch_dependents();
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
+    const int token_floats = 2 * VECTOR + A.cols + 4, stage_floats = A.batch * token_floats;
+    for (int i = threadIdx.x; i < 2 * stage_floats; i += blockDim.x) stage[i] = 0.0f;      // rows beyond d, columns beyond e
+    __syncthreads();
+    pdl_wait();
+    const int seq = blockIdx.x, head = blockIdx.y / A.slices, slice = blockIdx.y % A.slices, chunk = blockIdx.z;
+    const int seq_first = A.q_start[seq], seq_last = A.q_start[seq + 1];
+    const int slot = A.state_slots[seq];
+    if (slot < 0 || seq_last <= seq_first) return;
+    const int first = MODE == SCAN_WHOLE ? seq_first : seq_first + chunk * A.chunk_len;
+    const int last = MODE == SCAN_WHOLE ? seq_last : min(seq_last, first + A.chunk_len);
+    if (first >= last) return;
+    const int part = lane / GROUPS, place = (warp * GROUPS + lane % GROUPS) * 4, col = slice * A.cols + place;
+    const int row0 = part * SCAN_ROWS;
+    const bool owns_norm = A.norm_state != nullptr && slice == 0 && warp == 0;
+    const size_t chunk_at = (((size_t)seq * A.heads + head) * A.max_chunks + chunk);
+    float* mine = MODE == SCAN_WHOLE ? A.state + (long long)slot * A.state_stride + (size_t)head * A.d * A.e : A.chunk_state + chunk_at * A.chunk_floats;
+    float* norm_mine = MODE == SCAN_WHOLE ? A.norm_state + (long long)slot * A.state_stride + (size_t)head * A.d : mine + (size_t)A.d * A.e;
+    const bool zero = MODE == SCAN_LOCAL || (MODE == SCAN_WHOLE && A.positions[seq_first] == 0);
+
+    const int q_at = head * A.d, v_at = head * A.e + slice * A.cols, live_cols = min(A.cols, A.e - slice * A.cols);
+    auto issue = [&](int t0, int n, int buffer) {
+        float* base = stage + buffer * stage_floats;
+        for (int j = warp; j < n; j += warps) {              // a warp copies a token
+            float* to = base + j * token_floats;
+            const size_t row = (size_t)(t0 + j) * A.stride;
+            if (A.vec_qk) {
+                for (int i = 4 * lane; i < A.d; i += 128) {
+                    const int where = (i / SCAN_ROWS) * SCAN_PITCH + i % SCAN_ROWS;
+                    scan_copy16(to + where, A.k + row + q_at + i);
+                    if (MODE != SCAN_LOCAL) scan_copy16(to + VECTOR + where, A.q + row + q_at + i);
+                }
+            } else {
+                for (int i = lane; i < A.d; i += 32) {
+                    const int where = (i / SCAN_ROWS) * SCAN_PITCH + i % SCAN_ROWS;
+                    scan_copy4(to + where, A.k + row + q_at + i);
+                    if (MODE != SCAN_LOCAL) scan_copy4(to + VECTOR + where, A.q + row + q_at + i);
+                }
+            }
+            if (A.vec_v) {
+                for (int i = 4 * lane; i < live_cols; i += 128) scan_copy16(to + 2 * VECTOR + i, A.v + row + v_at + i);
+            } else {
+                for (int i = lane; i < live_cols; i += 32) scan_copy4(to + 2 * VECTOR + i, A.v + row + v_at + i);
+            }
+            if (A.coef && lane < 2) scan_copy4(to + 2 * VECTOR + A.cols + lane, A.coef + (size_t)(t0 + j) * A.coef_stride + lane * A.heads + head);
+        }
+        asm volatile("cp.async.commit_group;\n" ::);
+    };
+    issue(first, min(A.batch, last - first), 0);
+
+    float4 s[SCAN_ROWS];
+    float norm[SCAN_ROWS];
+#pragma unroll
+    for (int i = 0; i < SCAN_ROWS; ++i) {
+        s[i] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        norm[i] = 0.0f;
+        if (!zero && row0 + i < A.d) {
+            const float* from = mine + (size_t)(row0 + i) * A.e + col;
+            if (A.vec_state) {
+                if (col < A.e) s[i] = *reinterpret_cast<const float4*>(from);
+            } else {
+                if (col < A.e) s[i].x = from[0];
+                if (col + 1 < A.e) s[i].y = from[1];
+                if (col + 2 < A.e) s[i].z = from[2];
+                if (col + 3 < A.e) s[i].w = from[3];
+            }
+            if (owns_norm) norm[i] = norm_mine[row0 + i];
+        }
+    }
+    const float fixed = A.decay ? A.decay[head] : 1.0f;
+    float P = 1.0f, product = 1.0f;
+    const int batches = (last - first + A.batch - 1) / A.batch;
+    for (int b = 0; b < batches; ++b) {
+        const int t0 = first + b * A.batch, n = min(A.batch, last - t0);
+        if (b + 1 < batches) {
+            issue(t0 + A.batch, min(A.batch, last - t0 - A.batch), (b + 1) & 1);
+            asm volatile("cp.async.wait_group 1;\n" ::);
+        } else {
+            asm volatile("cp.async.wait_group 0;\n" ::);
+        }
+        __syncthreads();
+        const float* token = stage + (b & 1) * stage_floats;
+        for (int j = 0; j < n; ++j, token += token_floats) {
+            float keep = fixed, take = 1.0f;
+            if (A.coef) keep = token[2 * VECTOR + A.cols], take = token[2 * VECTOR + A.cols + 1];
+            P *= keep;
+            if (MODE == SCAN_LOCAL) product *= keep;
+            if (P < SCAN_LEAST) {                            // the same for every thread of the block
+#pragma unroll
+                for (int i = 0; i < SCAN_ROWS; ++i) {
+                    s[i].x *= P, s[i].y *= P, s[i].z *= P, s[i].w *= P;
+                    norm[i] *= P;
+                }
+                P = 1.0f;
+            }
+            const float weight = take / P;
+            const float4 vv = *reinterpret_cast<const float4*>(token + 2 * VECTOR + place);
+            const float4 tv = make_float4(vv.x * weight, vv.y * weight, vv.z * weight, vv.w * weight);
+            float4 y = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            const float* kp = token + part * SCAN_PITCH;
+#pragma unroll
+            for (int i4 = 0; i4 < SCAN_ROWS; i4 += 4) {
+                const float4 k4 = *reinterpret_cast<const float4*>(kp + i4);
+                const float kk[4] = {k4.x, k4.y, k4.z, k4.w};
+                float qq[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+                if (MODE != SCAN_LOCAL) {
+                    const float4 q4 = *reinterpret_cast<const float4*>(kp + VECTOR + i4);
+                    qq[0] = q4.x, qq[1] = q4.y, qq[2] = q4.z, qq[3] = q4.w;
+                }
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                    float4& r = s[i4 + i];
+                    r.x = fmaf(kk[i], tv.x, r.x), r.y = fmaf(kk[i], tv.y, r.y), r.z = fmaf(kk[i], tv.z, r.z), r.w = fmaf(kk[i], tv.w, r.w);
+                    if (MODE != SCAN_LOCAL)
+                        y.x = fmaf(r.x, qq[i], y.x), y.y = fmaf(r.y, qq[i], y.y), y.z = fmaf(r.z, qq[i], y.z), y.w = fmaf(r.w, qq[i], y.w);
+                }
+            }
+            if (owns_norm) {                                 // n takes k alone: a column whose value is always 1
+                float c = 0.0f;
+#pragma unroll
+                for (int i = 0; i < SCAN_ROWS; ++i) {
+                    norm[i] = fmaf(kp[i], weight, norm[i]);
+                    if (MODE != SCAN_LOCAL) c = fmaf(norm[i], kp[VECTOR + i], c);
+                }
+                if (MODE != SCAN_LOCAL) {
+#pragma unroll
+                    for (int o = GROUPS; o < 32; o <<= 1) c += __shfl_xor_sync(0xffffffffu, c, o);
+                    if (lane == 0) A.norm_out[(size_t)(t0 + j) * A.heads + head] = c * P;
+                }
+            }
+            if (MODE == SCAN_LOCAL) continue;
+            float* to = A.out + (size_t)(t0 + j) * A.heads * A.e + (size_t)head * A.e + col;
+            if (PARTS == 1) {
+                if (A.vec_out) {
+                    if (col < A.e) *reinterpret_cast<float4*>(to) = make_float4(y.x * P, y.y * P, y.z * P, y.w * P);
+                } else {
+                    if (col < A.e) to[0] = y.x * P;
+                    if (col + 1 < A.e) to[1] = y.y * P;
+                    if (col + 2 < A.e) to[2] = y.z * P;
+                    if (col + 3 < A.e) to[3] = y.w * P;
+                }
+            } else {
+                const bool upper = part & 1;                 // this lane goes on with the upper two of the four columns
+                float y0 = upper ? y.z : y.x, y1 = upper ? y.w : y.y;
+                y0 += __shfl_xor_sync(0xffffffffu, upper ? y.x : y.z, GROUPS);
+                y1 += __shfl_xor_sync(0xffffffffu, upper ? y.y : y.w, GROUPS);
+                if (PARTS == 2) {
+                    const int at = upper ? 2 : 0;
+                    if (col + at < A.e) to[at] = y0 * P;
+                    if (col + at + 1 < A.e) to[at + 1] = y1 * P;
+                } else {
+                    const bool second = part & 2;
+                    float z = second ? y1 : y0;
+                    z += __shfl_xor_sync(0xffffffffu, second ? y0 : y1, 2 * GROUPS);
+#pragma unroll
+                    for (int o = 4 * GROUPS; o < 32; o <<= 1) z += __shfl_xor_sync(0xffffffffu, z, o);
+                    const int at = (upper ? 2 : 0) + (second ? 1 : 0);
+                    if (part < 4 && col + at < A.e) to[at] = z * P;
+                }
+            }
+        }
+        __syncthreads();                                     // the stage is copied into again two batches on
+    }
+    if (MODE == SCAN_LOCAL && threadIdx.x == 0 && slice == 0) A.chunk_decay[chunk_at] = product;
+    if (MODE == SCAN_LOCAL || (MODE == SCAN_WHOLE && A.write_state)) {
+#pragma unroll
+        for (int i = 0; i < SCAN_ROWS; ++i) {
+            if (row0 + i >= A.d) continue;
+            float* to = mine + (size_t)(row0 + i) * A.e + col;
+            if (A.vec_state) {
+                if (col < A.e) *reinterpret_cast<float4*>(to) = make_float4(s[i].x * P, s[i].y * P, s[i].z * P, s[i].w * P);
+            } else {
+                if (col < A.e) to[0] = s[i].x * P;
+                if (col + 1 < A.e) to[1] = s[i].y * P;
+                if (col + 2 < A.e) to[2] = s[i].z * P;
+                if (col + 3 < A.e) to[3] = s[i].w * P;
+            }
+            if (owns_norm && lane % GROUPS == 0) norm_mine[row0 + i] = norm[i] * P;
+        }
+    }
+}
+
+// One thread an element of a (sequence, head)'s S (and n behind it): chunk c's entry goes from the chunk's end state from zero
+// to the state at its start, in[0] = the slot's state (zero at position 0), in[c + 1] = product_c in[c] + end_c.
+__global__ void scan_chunk_states_kernel(const ScanArgs A, int elements) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int seq = blockIdx.x, head = blockIdx.y;
+    const int first = A.q_start[seq], rows = A.q_start[seq + 1] - first;
+    const int slot = A.state_slots[seq];
+    if (slot < 0 || rows <= 0) return;
+    const int chunks = (rows + A.chunk_len - 1) / A.chunk_len, matrix = A.d * A.e;
+    const bool fresh = A.positions[first] == 0;
+    float* local = A.chunk_state + ((size_t)seq * A.heads + head) * A.max_chunks * A.chunk_floats;
+    const float* product = A.chunk_decay + ((size_t)seq * A.heads + head) * A.max_chunks;
+    for (int i = blockIdx.z * blockDim.x + threadIdx.x; i < elements; i += gridDim.z * blockDim.x) {
+        float* slot_at = (i < matrix ? A.state + (size_t)head * matrix + i : A.norm_state + (size_t)head * A.d + (i - matrix)) +
+                         (long long)slot * A.state_stride;
+        float value = fresh ? 0.0f : *slot_at;
+        for (int c = 0; c < chunks; ++c) {
+            const float end = local[(size_t)c * A.chunk_floats + i];
+            local[(size_t)c * A.chunk_floats + i] = value;
+            value = product[c] * value + end;
+        }
+        if (A.write_state) *slot_at = value;
+    }
+}
+
+}  // namespace
+
+MRS_EXPORT int mrs_rotate_heads(float* rows, int stride, int offset, const float* table, int tokens, int heads, int d, int rot, void* s) {
+    if (tokens <= 0 || rot == 0) return 0;
+    if (heads <= 0 || d <= 0 || rot < 0 || rot % 2 || rot > d || offset < 0 || offset + heads * d > stride || !table) return MRS_BAD_ARGUMENT;
+    const bool vec = rot % 8 == 0 && d % 4 == 0 && stride % 4 == 0 && offset % 4 == 0 && (((uintptr_t)rows | (uintptr_t)table) & 15) == 0;
+    const int work = heads * (vec ? rot / 8 : rot / 2);
+    const int threads = work >= 256 ? 256 : (work >= 128 ? 128 : 64);
+    if (vec)
+        MRS_LAUNCH(rotate_heads_kernel<true>, tokens, threads, 0, s, rows, stride, offset, table, tokens, heads, d, rot);
+    else
+        MRS_LAUNCH(rotate_heads_kernel<false>, tokens, threads, 0, s, rows, stride, offset, table, tokens, heads, d, rot);
+    MRS_RETURN_LAUNCH_STATUS();
+}
+
+MRS_EXPORT int mrs_narrow_columns(int is_bf16, const float* rows, int stride, int offset, void* out, int tokens, int columns, int live, void* s) {
+    if (tokens <= 0 || columns <= 0) return 0;
+    if (live < 0 || live > columns || offset < 0 || offset + live > stride) return MRS_BAD_ARGUMENT;
+    const long long total = (long long)tokens * columns;
+    long long blocks = (total + 255) / 256;
+    if (blocks > 8LL * mrs_sm_count()) blocks = 8LL * mrs_sm_count();
+    if (is_bf16)
+        MRS_LAUNCH(narrow_columns_kernel<bf16>, (unsigned)blocks, 256, 0, s, rows, stride, offset, (bf16*)out, total, columns, live);
+    else
+        MRS_LAUNCH(narrow_columns_kernel<float>, (unsigned)blocks, 256, 0, s, rows, stride, offset, (float*)out, total, columns, live);
+    MRS_RETURN_LAUNCH_STATUS();
+}
+
+MRS_EXPORT int mrs_memory_gates(const float* raw, int raw_stride, int i_offset, int f_offset, const float* i_bias, const float* f_bias,
+                                float cap, float* m_state, long long state_stride, const int* positions, const int* q_start,
+                                const int* state_slots, float* coef, int tokens, int sequences, int heads, int write_state, void* s) {
+    if (tokens <= 0 || sequences <= 0) return 0;
+    if (heads <= 0 || heads > 65535 || !(cap > 0.0f) || i_offset < 0 || f_offset < 0 || i_offset + heads > raw_stride ||
+        f_offset + heads > raw_stride)
+        return MRS_BAD_ARGUMENT;
+    const int average = tokens / sequences;
+    const int threads = average >= 256 ? 512 : (average >= 64 ? 128 : 32);
+    MRS_LAUNCH(memory_gates_kernel, dim3(sequences, heads), threads, 0, s, raw, raw_stride, i_offset, f_offset, i_bias, f_bias, cap, m_state,
+               state_stride, positions, q_start, state_slots, coef, heads, write_state);
+    MRS_RETURN_LAUNCH_STATUS();
+}
+
+// How the recurrence is cut: lanes that share a column group, columns a block, slices of the columns.  Returns the slices.
+static int scan_shape(int d, int e, int* parts_out, int* cols_out) {
+    int parts = 1;
+    while (parts * SCAN_ROWS < d) parts <<= 1;
+    const int per_warp = 4 * (32 / parts);
+    int warps = (e + per_warp - 1) / per_warp;
+    if (warps > 8) warps = 8;
+    *parts_out = parts;
+    *cols_out = warps * per_warp;
+    return (e + *cols_out - 1) / *cols_out;
+}
+
+MRS_EXPORT int mrs_linear_scan_slices(int d, int e) {
+    int parts, cols;
+    if (d <= 0 || d > 512 || e <= 0) return 0;
+    return scan_shape(d, e, &parts, &cols);
+}
+
+// Floats of scratch that a run in chunks needs.
+MRS_EXPORT long long mrs_linear_scan_scratch_floats(int tokens, int sequences, int heads, int d, int e, int normaliser, int chunk_len) {
+    if (chunk_len <= 0) return 0;
+    const long long chunks = (tokens + chunk_len - 1) / chunk_len;
+    return (long long)sequences * heads * chunks * (((long long)d * e + (normaliser ? d : 0) + 3) / 4 * 4 + 1);
+}
+
+// q, k, v: pointers to the columns of the first head in float32 rows of `stride` floats.  `chunk_len` 0: in one go.
+MRS_EXPORT int mrs_linear_scan(const float* q, const float* k, const float* v, int stride, const float* decay, const float* coef,
+                               int coef_stride, float* state, float* norm_state, long long state_stride, const int* positions,
+                               const int* q_start, const int* state_slots, float* out, float* norm_out, int tokens, int sequences,
+                               int heads, int d, int e, int write_state, int chunk_len, float* scratch, void* s) {
+    if (tokens <= 0 || sequences <= 0) return 0;
+    if (heads <= 0 || d <= 0 || d > 512 || e <= 0 || chunk_len < 0 || (chunk_len > 0 && !scratch) || (!decay && !coef) ||
+        (norm_state && !norm_out) || ((uintptr_t)scratch & 15))
+        return MRS_BAD_ARGUMENT;
+    ScanArgs A = {};
+    int parts, cols;
+    const int slices = scan_shape(d, e, &parts, &cols);
+    if ((long long)heads * slices > 65535) return MRS_BAD_ARGUMENT;
+    A.q = q, A.k = k, A.v = v, A.stride = stride, A.decay = decay, A.coef = decay ? nullptr : coef, A.coef_stride = coef_stride;
+    A.state = state, A.norm_state = norm_state, A.state_stride = state_stride;
+    A.positions = positions, A.q_start = q_start, A.state_slots = state_slots, A.out = out, A.norm_out = norm_out;
+    A.heads = heads, A.d = d, A.e = e, A.cols = cols, A.slices = slices, A.write_state = write_state;
+    A.vec_qk = d % 4 == 0 && stride % 4 == 0 && (((uintptr_t)q | (uintptr_t)k) & 15) == 0;
+    A.vec_v = e % 4 == 0 && stride % 4 == 0 && ((uintptr_t)v & 15) == 0;
+    A.vec_out = e % 4 == 0 && ((uintptr_t)out & 15) == 0;
+    const int token_floats = 2 * parts * SCAN_PITCH + cols + 4;
+    int batch = (40 * 1024) / (2 * token_floats * (int)sizeof(float));
+    if (batch > 8) batch = 8;
+    if (tokens < 8 * sequences && batch > (tokens + sequences - 1) / sequences) batch = (tokens + sequences - 1) / sequences;
+    if (batch < 1) return MRS_BAD_ARGUMENT;
+    A.batch = batch;
+    const int threads = cols / (4 * (32 / parts)) * 32;
+    const size_t smem = 2 * (size_t)batch * token_floats * sizeof(float);
+#define SCAN_LAUNCH(MODE, GRID)                                                                          \
+    switch (parts) {                                                                                     \
+        case 1: MRS_LAUNCH((linear_scan_kernel<MODE, 1>), GRID, threads, smem, s, A); break;             \
+        case 2: MRS_LAUNCH((linear_scan_kernel<MODE, 2>), GRID, threads, smem, s, A); break;             \
+        case 4: MRS_LAUNCH((linear_scan_kernel<MODE, 4>), GRID, threads, smem, s, A); break;             \
+        case 8: MRS_LAUNCH((linear_scan_kernel<MODE, 8>), GRID, threads, smem, s, A); break;             \
+        case 16: MRS_LAUNCH((linear_scan_kernel<MODE, 16>), GRID, threads, smem, s, A); break;           \
+        default: MRS_LAUNCH((linear_scan_kernel<MODE, 32>), GRID, threads, smem, s, A); break;           \
+    }
+    if (chunk_len == 0) {
+        A.vec_state = e % 4 == 0 && state_stride % 4 == 0 && ((uintptr_t)state & 15) == 0;
+        SCAN_LAUNCH(SCAN_WHOLE, dim3(sequences, heads * slices));
+        MRS_RETURN_LAUNCH_STATUS();
+    }
+    A.chunk_len = chunk_len;
+    A.max_chunks = (tokens + chunk_len - 1) / chunk_len;
+    if (A.max_chunks > 65535) return MRS_BAD_ARGUMENT;
+    const int elements = d * e + (norm_state ? d : 0);
+    A.chunk_floats = (elements + 3) / 4 * 4;
+    A.chunk_state = scratch;
+    A.chunk_decay = scratch + (size_t)sequences * heads * A.max_chunks * A.chunk_floats;
+    A.vec_state = e % 4 == 0;
+    SCAN_LAUNCH(SCAN_LOCAL, dim3(sequences, heads * slices, A.max_chunks));
+    int across = (elements + 255) / 256;
+    if (across > 64) across = 64;
+    MRS_LAUNCH(scan_chunk_states_kernel, dim3(sequences, heads, across), 256, 0, s, A, elements);
+    SCAN_LAUNCH(SCAN_FINAL, dim3(sequences, heads * slices, A.max_chunks));
+#undef SCAN_LAUNCH
+    MRS_RETURN_LAUNCH_STATUS();
+}

@@ -1,7 +1,9 @@
 // Row-wise kernels of layers whose branches run side by side on one normed input, of plain (ungated) feed-forwards and
 // of capped logits.  Sums, statistics and the activation's arithmetic are float32; T is the engine's dtype.
 //
-//   add_branches_norm   stream += a (+ b);  out = stream / sqrt(mean(stream^2) + eps) * w_next   (w_next may be null: sum only)
+//   add_branches_norm   stream += the sum of up to three branches, each times its factor;  out = stream / sqrt(mean(stream^2)
+//                       + eps) * w for none, one or two weights w of the norms that read the stream next
+//   embed_norm          stream = row / sqrt(mean(row^2) + eps) * w, row the token's row of the embedding table
 //   activation          out = act(in):  0 = gelu with the error function, 0.5 z (1 + erf(z / sqrt 2));
 //                                       1 = gelu with tanh, 0.5 z (1 + tanh(sqrt(2 / pi) (z + 0.044715 z^3)));   2 = silu
 //   scale_softcap       x <- cap * tanh(x * scale / cap)
@@ -20,42 +22,72 @@ template <> __device__ __forceinline__ void st4<bf16>(bf16* p, float4 v) {
     *reinterpret_cast<uint2*>(p) = raw;
 }
 
+#define MAX_BRANCHES 3
+struct BranchSum {
+    const float* x[MAX_BRANCHES];        // the branches, in the order in which they are summed (null: no more)
+    float factor[MAX_BRANCHES];
+};
+struct NextNorms {
+    const float* w[2];                   // the next norms' weights (null: none), one eps for both
+    void* out[2];
+    float eps;
+};
+
+__device__ __forceinline__ float branch_sum(const BranchSum& B, size_t at) {
+    float x = B.factor[0] * B.x[0][at];
+#pragma unroll
+    for (int k = 1; k < MAX_BRANCHES; ++k)
+        if (B.x[k]) x += B.factor[k] * B.x[k][at];
+    return x;
+}
+__device__ __forceinline__ float4 branch_sum4(const BranchSum& B, size_t at) {
+    float4 x = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+#pragma unroll
+    for (int k = 0; k < MAX_BRANCHES; ++k) {
+        if (!B.x[k]) continue;
+        const float4 y = ld4(B.x[k] + at);
+        x.x += B.factor[k] * y.x, x.y += B.factor[k] * y.y, x.z += B.factor[k] * y.z, x.w += B.factor[k] * y.w;
+    }
+    return x;
+}
+
 // Any width: one block a row, the sum is written and read again for the norm.
 template <typename T>
-__global__ void add_branches_norm_kernel(float* __restrict__ stream, const float* __restrict__ a, const float* __restrict__ b,
-                                         const float* __restrict__ w_next, float eps, T* __restrict__ out, int width) {
+__global__ void add_branches_norm_kernel(float* __restrict__ stream, const BranchSum B, const NextNorms N, int width) {
     pdl_launch_dependents();
     pdl_wait();
     __shared__ float scratch[33];
     const size_t r = blockIdx.x;
     float* res = stream + r * width;
-    const float* ar = a + r * width;
-    const float* br = b ? b + r * width : nullptr;
     float sum = 0.0f;
     for (int i = threadIdx.x; i < width; i += blockDim.x) {
-        const float v = res[i] + (br ? ar[i] + br[i] : ar[i]);
-        res[i] = v;
+        float v = res[i];
+        if (B.x[0]) {
+            v += branch_sum(B, r * width + i);
+            res[i] = v;
+        }
         sum += v * v;
     }
-    if (w_next == nullptr) return;
-    const float scale = 1.0f / sqrtf(block_sum(sum, scratch) / (float)width + eps);
-    T* o = out + r * width;
-    for (int i = threadIdx.x; i < width; i += blockDim.x) o[i] = from_float<T>(res[i] * scale * w_next[i]);
+    if (N.w[0] == nullptr) return;
+    const float scale = 1.0f / sqrtf(block_sum(sum, scratch) / (float)width + N.eps);
+#pragma unroll
+    for (int k = 0; k < 2; ++k) {
+        if (N.w[k] == nullptr) continue;
+        T* o = (T*)N.out[k] + r * width;
+        for (int i = threadIdx.x; i < width; i += blockDim.x) o[i] = from_float<T>(res[i] * scale * N.w[k][i]);
+    }
 }
 
 // Width a multiple of 4, at most 16 * blockDim.x, rows on 16-byte boundaries: the row stays in registers between the
 // passes and every element is read once, four a load.
 #define BRANCH_KEEP 4
 template <typename T>
-__global__ void add_branches_norm_kept_kernel(float* __restrict__ stream, const float* __restrict__ a, const float* __restrict__ b,
-                                              const float* __restrict__ w_next, float eps, T* __restrict__ out, int width) {
+__global__ void add_branches_norm_kept_kernel(float* __restrict__ stream, const BranchSum B, const NextNorms N, int width) {
     pdl_launch_dependents();
     pdl_wait();
     __shared__ float scratch[33];
     const size_t r = blockIdx.x;
     float* res = stream + r * width;
-    const float* ar = a + r * width;
-    const float* br = b ? b + r * width : nullptr;
     float4 v[BRANCH_KEEP], w[BRANCH_KEEP];
     float sum = 0.0f;
 #pragma unroll
@@ -64,30 +96,47 @@ __global__ void add_branches_norm_kept_kernel(float* __restrict__ stream, const 
         v[j] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
         if (i < width) {
             v[j] = ld4(res + i);
-            float4 x = ld4(ar + i);
-            if (br) {
-                const float4 y = ld4(br + i);
-                x.x += y.x, x.y += y.y, x.z += y.z, x.w += y.w;
+            if (B.x[0]) {
+                const float4 x = branch_sum4(B, r * width + i);
+                v[j].x += x.x, v[j].y += x.y, v[j].z += x.z, v[j].w += x.w;
+                st4<float>(res + i, v[j]);
             }
-            v[j].x += x.x, v[j].y += x.y, v[j].z += x.z, v[j].w += x.w;
-            st4<float>(res + i, v[j]);
             sum += v[j].x * v[j].x + v[j].y * v[j].y + v[j].z * v[j].z + v[j].w * v[j].w;
         }
     }
-    if (w_next == nullptr) return;
+    if (N.w[0] == nullptr) return;
 #pragma unroll
     for (int j = 0; j < BRANCH_KEEP; ++j) {                  // asked for before the block waits for its sum
         const int i = (threadIdx.x + j * blockDim.x) * 4;
-        w[j] = i < width ? ld4(w_next + i) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        w[j] = i < width ? ld4(N.w[0] + i) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
     }
-    const float scale = 1.0f / sqrtf(block_sum(sum, scratch) / (float)width + eps);
-    T* o = out + r * width;
+    const float scale = 1.0f / sqrtf(block_sum(sum, scratch) / (float)width + N.eps);
 #pragma unroll
-    for (int j = 0; j < BRANCH_KEEP; ++j) {
-        const int i = (threadIdx.x + j * blockDim.x) * 4;
-        if (i < width)
+    for (int k = 0; k < 2; ++k) {
+        if (N.w[k] == nullptr) continue;
+        T* o = (T*)N.out[k] + r * width;
+#pragma unroll
+        for (int j = 0; j < BRANCH_KEEP; ++j) {
+            const int i = (threadIdx.x + j * blockDim.x) * 4;
+            if (i >= width) continue;
+            if (k == 1) w[j] = ld4(N.w[1] + i);
             st4<T>(o + i, make_float4(v[j].x * scale * w[j].x, v[j].y * scale * w[j].y, v[j].z * scale * w[j].z, v[j].w * scale * w[j].w));
+        }
     }
+}
+
+template <typename T>
+__global__ void embed_norm_kernel(const T* __restrict__ table, const int* __restrict__ ids, const float* __restrict__ w, float eps,
+                                  float* __restrict__ stream, int width) {
+    pdl_launch_dependents();
+    pdl_wait();
+    __shared__ float scratch[33];
+    const size_t r = blockIdx.x;
+    const T* from = table + (size_t)ids[r] * width;
+    float sum = 0.0f;
+    for (int i = threadIdx.x; i < width; i += blockDim.x) sum += to_float(from[i]) * to_float(from[i]);
+    const float scale = 1.0f / sqrtf(block_sum(sum, scratch) / (float)width + eps);
+    for (int i = threadIdx.x; i < width; i += blockDim.x) stream[r * width + i] = to_float(from[i]) * scale * w[i];
 }
 
 __device__ __forceinline__ float activate(float z, int kind) {
@@ -154,25 +203,44 @@ __global__ void scale_softcap_kernel(float* __restrict__ x, long long n, float s
 
 }  // namespace
 
-MRS_EXPORT int mrs_add_branches_norm(int is_bf16, float* stream, const float* a, const float* b, const float* w_next, float eps,
-                                     void* out, int rows, int width, void* s) {
+// `a`, `b`, `c`: branches with their factors (null: none; without `a` the stream is only normed); `w0`, `w1`: weights of the
+// next norms.
+MRS_EXPORT int mrs_add_branches_norm(int is_bf16, float* stream, const float* a, float fa, const float* b, float fb, const float* c,
+                                     float fc, const float* w0, const float* w1, float eps, void* out0, void* out1, int rows, int width,
+                                     void* s) {
     if (rows <= 0) return 0;
-    if (width <= 0 || !a || (w_next && !out)) return MRS_BAD_ARGUMENT;
-    const bool aligned = (((uintptr_t)stream | (uintptr_t)a | (uintptr_t)b | (uintptr_t)w_next | (uintptr_t)out) & 15) == 0;
+    if (width <= 0 || (w0 && !out0) || (w1 && (!out1 || !w0)) || (!a && (b || c || !w0))) return MRS_BAD_ARGUMENT;
+    if (!b && c) b = c, fb = fc, c = nullptr;
+    const BranchSum B = {{a, b, c}, {fa, fb, fc}};
+    const NextNorms N = {{w0, w1}, {out0, out1}, eps};
+    const bool aligned = (((uintptr_t)stream | (uintptr_t)a | (uintptr_t)b | (uintptr_t)c | (uintptr_t)w0 | (uintptr_t)w1 |
+                           (uintptr_t)out0 | (uintptr_t)out1) & 15) == 0;
     if (width % 4 == 0 && aligned && width <= 4 * BRANCH_KEEP * 512) {
         int threads = ((width / 4 + BRANCH_KEEP - 1) / BRANCH_KEEP + 31) / 32 * 32;
         if (threads < 64) threads = 64;
         if (is_bf16)
-            MRS_LAUNCH(add_branches_norm_kept_kernel<bf16>, rows, threads, 0, s, stream, a, b, w_next, eps, (bf16*)out, width);
+            MRS_LAUNCH(add_branches_norm_kept_kernel<bf16>, rows, threads, 0, s, stream, B, N, width);
         else
-            MRS_LAUNCH(add_branches_norm_kept_kernel<float>, rows, threads, 0, s, stream, a, b, w_next, eps, (float*)out, width);
+            MRS_LAUNCH(add_branches_norm_kept_kernel<float>, rows, threads, 0, s, stream, B, N, width);
         MRS_RETURN_LAUNCH_STATUS();
     }
     const int threads = width >= 2048 ? 512 : (width >= 512 ? 256 : 128);
     if (is_bf16)
-        MRS_LAUNCH(add_branches_norm_kernel<bf16>, rows, threads, 0, s, stream, a, b, w_next, eps, (bf16*)out, width);
+        MRS_LAUNCH(add_branches_norm_kernel<bf16>, rows, threads, 0, s, stream, B, N, width);
     else
-        MRS_LAUNCH(add_branches_norm_kernel<float>, rows, threads, 0, s, stream, a, b, w_next, eps, (float*)out, width);
+        MRS_LAUNCH(add_branches_norm_kernel<float>, rows, threads, 0, s, stream, B, N, width);
+    MRS_RETURN_LAUNCH_STATUS();
+}
+
+MRS_EXPORT int mrs_embed_norm(int is_bf16, const void* table, const int* ids, const float* w, float eps, float* stream, int rows, int width,
+                              void* s) {
+    if (rows <= 0) return 0;
+    if (width <= 0 || !table || !w) return MRS_BAD_ARGUMENT;
+    const int threads = width >= 2048 ? 512 : (width >= 512 ? 256 : 128);
+    if (is_bf16)
+        MRS_LAUNCH(embed_norm_kernel<bf16>, rows, threads, 0, s, (const bf16*)table, ids, w, eps, stream, width);
+    else
+        MRS_LAUNCH(embed_norm_kernel<float>, rows, threads, 0, s, (const float*)table, ids, w, eps, stream, width);
     MRS_RETURN_LAUNCH_STATUS();
 }
 

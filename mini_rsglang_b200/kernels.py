@@ -1881,17 +1881,20 @@ def moe_combine(y: torch.Tensor | None, h: torch.Tensor, shared_out: torch.Tenso
 # branches side by side, plain feed-forwards, capped logits; the gated delta rule
 # ------------------------------------------------------------------------------------------------
 _PARALLEL_SIGNATURES = {
-    "mrs_add_branches_norm": [_c_int, _c_vp, _c_vp, _c_vp, _c_vp, _c_float, _c_vp, _c_int, _c_int, _c_vp],
+    "mrs_add_branches_norm": [_c_int, _c_vp, _c_vp, _c_float, _c_vp, _c_float, _c_vp, _c_float, _c_vp, _c_vp, _c_float, _c_vp, _c_vp,
+                              _c_int, _c_int, _c_vp],
+    "mrs_embed_norm": [_c_int, _c_vp, _c_vp, _c_vp, _c_float, _c_vp, _c_int, _c_int, _c_vp],
     "mrs_activation": [_c_int, _c_vp, _c_vp, ctypes.c_longlong, _c_int, _c_vp],
     "mrs_scale_softcap": [_c_vp, ctypes.c_longlong, _c_float, _c_float, _c_vp],
     "mrs_gated_activation": [_c_int, _c_vp, _c_vp, _c_int, _c_int, _c_int, _c_int, _c_vp],
 }
 _DELTA_SIGNATURES = {
-    "mrs_delta_prepare": [_c_vp, _c_vp, _c_int, _c_int, _c_int, _c_vp, _c_vp, _c_vp, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float,
-                          _c_float, _c_vp],
-    "mrs_delta_scan": [_c_vp, _c_vp, _c_vp, ctypes.c_longlong, _c_vp, _c_vp, _c_vp, _c_vp, _c_int, _c_int, _c_int, _c_int, _c_int,
-                       _c_int, _c_int, _c_vp],
-    "mrs_head_norm_gate": [_c_int, _c_vp, _c_vp, _c_int, _c_vp, _c_float, _c_vp, _c_int, _c_int, _c_int, _c_vp],
+    "mrs_delta_prepare": [_c_vp, _c_vp, _c_int, _c_int, _c_int, _c_vp, _c_vp, _c_vp, _c_vp, _c_int, _c_int, _c_int, _c_int, _c_int,
+                          _c_int, _c_float, _c_float, _c_vp],
+    "mrs_delta_scan": [_c_vp, _c_vp, _c_vp, _c_int, _c_vp, ctypes.c_longlong, _c_vp, _c_vp, _c_vp, _c_vp, _c_int, _c_int, _c_int, _c_int,
+                       _c_int, _c_int, _c_int, _c_vp],
+    "mrs_head_norm_gate": [_c_int, _c_vp, _c_vp, _c_int, _c_int, _c_vp, _c_int, _c_float, _c_float, _c_vp, _c_vp, _c_int, _c_float, _c_vp,
+                           _c_int, _c_int, _c_int, _c_vp],
 }
 _parallel_lib = None
 _delta_lib = None
@@ -1924,18 +1927,46 @@ def add_branches_norm(stream: torch.Tensor, a: torch.Tensor, b: torch.Tensor | N
                       next_eps: float, out: torch.Tensor | None) -> None:
     """stream += a (+ b), all float32 [rows, width]; with `next_weight`, out = stream / sqrt(mean(stream^2) + eps) * next_weight
     in out's dtype."""
+    branches = [(a, 1.0)] + ([(b, 1.0)] if b is not None else [])
+    add_scaled_branches_norms(stream, branches, [(next_weight, out)] if next_weight is not None else [], next_eps)
+
+
+MAX_BRANCHES = 3
+
+
+def add_scaled_branches_norms(stream: torch.Tensor, branches: list, norms: list, eps: float) -> None:
+    """stream += the sum of factor * branch over `branches` [(tensor, factor), at most three], all float32 [rows, width]; then
+    for each of `norms` [(weight, out), at most two]: out = stream / sqrt(mean(stream^2) + eps) * weight in out's dtype.  No
+    branches: the stream is only normed."""
     rows, width = stream.shape
     _need(stream, torch.float32, "stream")
-    _need(a, torch.float32, "branch", (rows, width))
-    if b is not None:
-        _need(b, torch.float32, "second branch", (rows, width))
-    if next_weight is not None:
-        _need(next_weight, torch.float32, "next norm weight", (width,))
-        _need(out, None, "normed rows", (rows, width))
-    _check(parallel_library().mrs_add_branches_norm(_is_bf16(out.dtype) if out is not None and next_weight is not None else 0,
-                                                    stream.data_ptr(), a.data_ptr(), _ptr(b), _ptr(next_weight), float(next_eps),
-                                                    _ptr(out) if next_weight is not None else None, rows, width, _stream()),
-           "add_branches_norm")
+    if len(branches) > MAX_BRANCHES or len(norms) > 2 or not (branches or norms):
+        raise InvalidRequest("add_scaled_branches_norms: at most three branches and two norms, and something to do")
+    flat = []
+    for x, factor in branches:
+        _need(x, torch.float32, "branch", (rows, width))
+        flat += [x.data_ptr(), float(factor)]
+    flat += [None, 0.0] * (MAX_BRANCHES - len(branches))
+    for weight, out in norms:
+        _need(weight, torch.float32, "next norm weight", (width,))
+        _need(out, norms[0][1].dtype, "normed rows", (rows, width))
+    weights = [w.data_ptr() for w, _ in norms] + [None] * (2 - len(norms))
+    outs = [o.data_ptr() for _, o in norms] + [None] * (2 - len(norms))
+    _check(parallel_library().mrs_add_branches_norm(_is_bf16(norms[0][1].dtype) if norms else 0, stream.data_ptr(), *flat, *weights,
+                                                    float(eps), *outs, rows, width, _stream()), "add_branches_norm")
+
+
+def embed_norm(table: torch.Tensor, ids: torch.Tensor, weight: torch.Tensor, eps: float, stream: torch.Tensor) -> None:
+    """stream[t] = row / sqrt(mean(row^2) + eps) * weight with row = table[ids[t]]; float32 arithmetic and result."""
+    tokens, width = stream.shape
+    _need(table, None, "embed table")
+    _need(ids, torch.int32, "embed ids", (tokens,))
+    _need(weight, torch.float32, "embedding norm weight", (width,))
+    _need(stream, torch.float32, "embed output")
+    if table.shape[1] != width:
+        raise InvalidRequest("embed_norm: width mismatch")
+    _check(parallel_library().mrs_embed_norm(_is_bf16(table.dtype), table.data_ptr(), ids.data_ptr(), weight.data_ptr(), float(eps),
+                                             stream.data_ptr(), tokens, width, _stream()), "embed_norm")
 
 
 def activation(x: torch.Tensor, out: torch.Tensor, kind: str) -> None:
@@ -1971,55 +2002,233 @@ def scale_softcap_(x: torch.Tensor, scale: float, cap: float) -> None:
     _check(parallel_library().mrs_scale_softcap(x.data_ptr(), x.numel(), float(scale), float(cap), _stream()), "scale_softcap")
 
 
+def _check_channels(channels, tokens: int, heads: int, d: int, what: str) -> tuple:
+    """Pointer and row stride of the decays a head and channel: float32 [tokens, heads * d], may be columns of wider rows."""
+    if channels is None:
+        return None, 0
+    if not channels.is_cuda or channels.dtype != torch.float32 or tuple(channels.shape) != (tokens, heads * d) or channels.stride(1) != 1:
+        raise InvalidRequest(f"{what}: the channels' decays must be float32 [tokens, heads * d] with unit column stride")
+    return channels.data_ptr(), channels.stride(0)
+
+
 def delta_prepare(qkv: torch.Tensor, raw: torch.Tensor, b_offset: int, a_offset: int, a_log: torch.Tensor, dt_bias: torch.Tensor,
-                  coef: torch.Tensor, groups: int, d: int, heads: int, e: int, unit_eps: float, q_factor: float) -> None:
+                  coef: torch.Tensor, groups: int, d: int, heads: int, e: int, unit_eps: float, q_factor: float,
+                  channels: torch.Tensor | None = None) -> None:
     """Per token, in place on `qkv` [tokens, 2 * groups * d + heads * e] float32 (q of every group | k of every group | v of
     every head): every q and k becomes x / sqrt(sum x^2 + unit_eps), q also times `q_factor`; `coef` [tokens, 2 * heads]
     gets beta = sigmoid(b) and g = exp(-exp(A_log) * softplus(a + dt_bias)) of every head, b and a read at the columns
-    `b_offset` and `a_offset` of the float32 rows `raw`."""
+    `b_offset` and `a_offset` of the float32 rows `raw`.  With `channels` [tokens, heads * d] (raw decays of every head and
+    channel; `dt_bias` [heads * d] then) these become exp(-exp(A_log) * softplus(raw + dt_bias)) in place, `coef` is
+    [tokens, heads] (beta alone) and `a_offset` is not used."""
     tokens = qkv.shape[0]
     _need(qkv, torch.float32, "q|k|v", (tokens, 2 * groups * d + heads * e))
     _need(raw, torch.float32, "delta projection")
+    if channels is not None:
+        a_offset = b_offset
     if raw.shape[0] != tokens or min(b_offset, a_offset) < 0 or max(b_offset, a_offset) + heads > raw.shape[1]:
         raise InvalidRequest("delta_prepare: b and a lie outside the rows")
+    pointer, stride = _check_channels(channels, tokens, heads, d, "delta_prepare")
     _need(a_log, torch.float32, "A_log", (heads,))
-    _need(dt_bias, torch.float32, "dt_bias", (heads,))
-    _need(coef, torch.float32, "beta|g", (tokens, 2 * heads))
+    _need(dt_bias, torch.float32, "dt_bias", (heads if channels is None else heads * d,))
+    _need(coef, torch.float32, "beta|g", (tokens, (2 if channels is None else 1) * heads))
     _check(delta_library().mrs_delta_prepare(qkv.data_ptr(), raw.data_ptr(), raw.shape[1], int(b_offset), int(a_offset), a_log.data_ptr(),
-                                             dt_bias.data_ptr(), coef.data_ptr(), tokens, groups, d, heads, e, float(unit_eps),
-                                             float(q_factor), _stream()), "delta_prepare")
+                                             dt_bias.data_ptr(), coef.data_ptr(), pointer, stride, tokens, groups, d, heads, e,
+                                             float(unit_eps), float(q_factor), _stream()), "delta_prepare")
 
 
 def delta_scan(qkv: torch.Tensor, coef: torch.Tensor, state: torch.Tensor, positions, q_start, state_slots, out: torch.Tensor,
-               heads: int, groups: int, d: int, e: int, write_state: bool = True) -> None:
+               heads: int, groups: int, d: int, e: int, write_state: bool = True, channels: torch.Tensor | None = None) -> None:
     """The gated delta rule token by token, float32, per (sequence, head): S <- g S; u = beta (v - S^T k); S <- S + k u^T;
-    o = S^T q.  `qkv` as `delta_prepare` leaves it, `coef` its beta | g; `state` [slots, heads, d, e] float32 (a view: dense
-    within a slot); a sequence that starts at position 0 starts from zero; `out` [tokens, heads * e] float32."""
+    o = S^T q.  `qkv` as `delta_prepare` leaves it, `coef` its beta | g (or beta alone, with the decays of the rows of S in
+    `channels`); `state` [slots, heads, d, e] float32 (a view: dense within a slot); a sequence that starts at position 0
+    starts from zero; `out` [tokens, heads * e] float32."""
     tokens = qkv.shape[0]
     _need(qkv, torch.float32, "q|k|v", (tokens, 2 * groups * d + heads * e))
-    _need(coef, torch.float32, "beta|g", (tokens, 2 * heads))
-    if state.dtype != torch.float32 or tuple(state.shape[1:]) != (heads, d, e) or state.stride(3) != 1 or state.stride(2) != e or \
-            state.stride(1) != d * e:
-        raise InvalidRequest("delta_scan: the state must be float32 [slots, heads, d, e], dense within a slot")
+    _need(coef, torch.float32, "beta|g", (tokens, (2 if channels is None else 1) * heads))
+    pointer, stride = _check_channels(channels, tokens, heads, d, "delta_scan")
+    _check_matrix_state(state, heads, d, e, "delta_scan")
     _need(out, torch.float32, "recurrence output", (tokens, heads * e))
     sequences = state_slots.shape[0]
-    _check(delta_library().mrs_delta_scan(qkv.data_ptr(), coef.data_ptr(), state.data_ptr(), state.stride(0), positions.data_ptr(),
-                                          q_start.data_ptr(), state_slots.data_ptr(), out.data_ptr(), tokens, sequences, heads, groups,
-                                          d, e, int(write_state), _stream()), "delta_scan")
+    _check(delta_library().mrs_delta_scan(qkv.data_ptr(), coef.data_ptr(), pointer, stride, state.data_ptr(), state.stride(0),
+                                          positions.data_ptr(), q_start.data_ptr(), state_slots.data_ptr(), out.data_ptr(), tokens,
+                                          sequences, heads, groups, d, e, int(write_state), _stream()), "delta_scan")
 
 
-def head_norm_gate(o: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor, heads: int) -> None:
-    """out = o / sqrt(mean over a head of o^2 + eps) * weight * silu(gate): `o` float32 [tokens, heads * e], `weight` [e]
-    float32 shared by the heads, `gate` float32 of o's shape (may be a column range of wider rows)."""
+def _check_matrix_state(state, heads: int, d: int, e: int, what: str) -> None:
+    if state.dtype != torch.float32 or tuple(state.shape[1:]) != (heads, d, e) or state.stride(3) != 1 or state.stride(2) != e or \
+            state.stride(1) != d * e:
+        raise InvalidRequest(f"{what}: the state must be float32 [slots, heads, d, e], dense within a slot")
+
+
+GATES = {"silu": 0, "sigmoid": 1}
+
+
+def head_norm_gate(o: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor | None, eps: float, out: torch.Tensor, heads: int,
+                   gate_kind: str = "silu", factor: float = 1.0, normaliser: tuple | None = None) -> None:
+    """out = x / sqrt(mean over a head of x^2 + eps) * weight * act(gate), x = o * factor: `o` float32 [tokens, heads * e],
+    `weight` float32 [e] (shared by the heads), [heads * e] or None, `gate` float32 of o's shape (may be a column range of
+    wider rows), act "silu" or "sigmoid".  `normaliser` = (c, floor, floor_eps): x is first divided by
+    max(|c * factor|, floor) + floor_eps; c float32 [tokens, heads], floor of the same shape (may be columns of wider rows)."""
     tokens, inner = o.shape
     e = inner // heads
     _need(o, torch.float32, "recurrence output")
     if not gate.is_cuda or gate.dtype != torch.float32 or tuple(gate.shape) != (tokens, inner) or gate.stride(1) != 1:
         raise InvalidRequest("head_norm_gate: the gate must be float32 [tokens, heads * e] with unit column stride")
-    _need(weight, torch.float32, "head norm weight", (e,))
+    if gate_kind not in GATES:
+        raise InvalidRequest(f"head_norm_gate: unknown gate {gate_kind!r}; known: {sorted(GATES)}")
+    stride = 0
+    if weight is not None:
+        stride = 0 if weight.shape[0] == e else e
+        _need(weight, torch.float32, "head norm weight", (e if stride == 0 else inner,))
+    c = floor = None
+    floor_stride, floor_eps = 0, 0.0
+    if normaliser is not None:
+        c, floor, floor_eps = normaliser
+        _need(c, torch.float32, "normaliser", (tokens, heads))
+        if floor.dtype != torch.float32 or tuple(floor.shape) != (tokens, heads) or floor.stride(1) != 1:
+            raise InvalidRequest("head_norm_gate: the normaliser's floor must be float32 [tokens, heads] with unit column stride")
+        floor_stride = floor.stride(0)
     _need(out, None, "head norm out", (tokens, inner))
-    _check(delta_library().mrs_head_norm_gate(_is_bf16(out.dtype), o.data_ptr(), gate.data_ptr(), gate.stride(0), weight.data_ptr(),
-                                              float(eps), out.data_ptr(), tokens, heads, e, _stream()), "head_norm_gate")
+    _check(delta_library().mrs_head_norm_gate(_is_bf16(out.dtype), o.data_ptr(), gate.data_ptr(), gate.stride(0), GATES[gate_kind],
+                                              _ptr(weight), stride, float(eps), float(factor), _ptr(c), _ptr(floor), floor_stride,
+                                              float(floor_eps), out.data_ptr(), tokens, heads, e, _stream()), "head_norm_gate")
+
+
+# ------------------------------------------------------------------------------------------------
+# recurrences that are linear in their state
+# ------------------------------------------------------------------------------------------------
+_LINEAR_SCAN_SIGNATURES = {
+    "mrs_rotate_heads": [_c_vp, _c_int, _c_int, _c_vp, _c_int, _c_int, _c_int, _c_int, _c_vp],
+    "mrs_narrow_columns": [_c_int, _c_vp, _c_int, _c_int, _c_vp, _c_int, _c_int, _c_int, _c_vp],
+    "mrs_memory_gates": [_c_vp, _c_int, _c_int, _c_int, _c_vp, _c_vp, _c_float, _c_vp, _c_ll, _c_vp, _c_vp, _c_vp, _c_vp, _c_int, _c_int,
+                         _c_int, _c_int, _c_vp],
+    "mrs_linear_scan_slices": [_c_int, _c_int],
+    "mrs_linear_scan": [_c_vp, _c_vp, _c_vp, _c_int, _c_vp, _c_vp, _c_int, _c_vp, _c_vp, _c_ll, _c_vp, _c_vp, _c_vp, _c_vp, _c_vp, _c_int,
+                        _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_vp, _c_vp],
+}
+_linear_scan_lib = None
+LINEAR_SCAN_MAX_DIM = 512
+
+
+def linear_scan_library() -> ctypes.CDLL:
+    global _linear_scan_lib
+    if _linear_scan_lib is None:
+        if not torch.cuda.is_available():
+            raise BackendError("no CUDA device: the engine has no CPU path")
+        from .csrc.build import linear_scan_kernel_library
+
+        lib = _typed(linear_scan_kernel_library(), _LINEAR_SCAN_SIGNATURES)
+        lib.mrs_linear_scan_scratch_floats.argtypes = [_c_int] * 7
+        lib.mrs_linear_scan_scratch_floats.restype = ctypes.c_longlong
+        _linear_scan_lib = lib
+    return _linear_scan_lib
+
+
+def rotate_heads_(rows: torch.Tensor, offset: int, heads: int, d: int, rotations: torch.Tensor, rotary_dim: int) -> None:
+    """`heads` heads of `d` elements from column `offset` of the float32 rows turn in place: element i of the first `rotary_dim`
+    with i + rotary_dim / 2, by `rotations` [tokens, rotary_dim / 2, 2] (cosines and sines)."""
+    tokens = rows.shape[0]
+    _need(rows, torch.float32, "rows")
+    _need(rotations, torch.float32, "rotations", (tokens, rotary_dim // 2, 2))
+    if offset < 0 or offset + heads * d > rows.shape[1] or rotary_dim > d or rotary_dim % 2:
+        raise InvalidRequest("rotate_heads: the heads lie outside the rows, or more than a head turns")
+    _check(linear_scan_library().mrs_rotate_heads(rows.data_ptr(), rows.shape[1], int(offset), rotations.data_ptr(), tokens, heads, d,
+                                                  int(rotary_dim), _stream()), "rotate_heads")
+
+
+def narrow_columns(rows: torch.Tensor, offset: int, live: int, out: torch.Tensor) -> None:
+    """out[:, :live] = rows[:, offset : offset + live] (float32) in out's dtype, zeros behind."""
+    tokens, columns = out.shape
+    _need(rows, torch.float32, "rows")
+    _need(out, None, "narrowed columns")
+    if rows.shape[0] != tokens or offset < 0 or offset + live > rows.shape[1] or live > columns:
+        raise InvalidRequest("narrow_columns: the columns lie outside the rows")
+    _check(linear_scan_library().mrs_narrow_columns(_is_bf16(out.dtype), rows.data_ptr(), rows.shape[1], int(offset), out.data_ptr(), tokens,
+                                                    columns, int(live), _stream()), "narrow_columns")
+
+
+def memory_gates(raw: torch.Tensor, i_offset: int, f_offset: int, i_bias: torch.Tensor, f_bias: torch.Tensor, cap: float,
+                 m_state: torch.Tensor, positions, q_start, state_slots, coef: torch.Tensor, write_state: bool = True) -> None:
+    """Gates of an exponential memory with a running maximum, per (token, head): i = cap tanh((raw_i + i_bias) / cap), f =
+    logsigmoid(cap tanh((raw_f + f_bias) / cap)), m_t = max(f + m_(t-1), i), m starting at 0; `coef` [tokens, 3 * heads] gets
+    exp(f + m_(t-1) - m_t) | exp(i - m_t) | exp(-m_t).  raw: float32 rows with the raw gates at the two columns; `m_state`
+    [slots, heads] float32 (a view: dense within a slot)."""
+    tokens, heads = raw.shape[0], i_bias.shape[0]
+    _need(raw, torch.float32, "raw gates")
+    _need(i_bias, torch.float32, "input gate bias", (heads,))
+    _need(f_bias, torch.float32, "forget gate bias", (heads,))
+    _need(coef, torch.float32, "gates", (tokens, 3 * heads))
+    if min(i_offset, f_offset) < 0 or max(i_offset, f_offset) + heads > raw.shape[1] or not cap > 0:
+        raise InvalidRequest("memory_gates: the gates lie outside the rows, or the cap is not positive")
+    if m_state.dtype != torch.float32 or tuple(m_state.shape[1:]) != (heads,) or m_state.stride(1) != 1:
+        raise InvalidRequest("memory_gates: the maxima must be float32 [slots, heads], dense within a slot")
+    _check(linear_scan_library().mrs_memory_gates(raw.data_ptr(), raw.shape[1], int(i_offset), int(f_offset), i_bias.data_ptr(),
+                                                  f_bias.data_ptr(), float(cap), m_state.data_ptr(), m_state.stride(0), positions.data_ptr(),
+                                                  q_start.data_ptr(), state_slots.data_ptr(), coef.data_ptr(), tokens, state_slots.shape[0],
+                                                  heads, int(write_state), _stream()), "memory_gates")
+
+
+def linear_scan_chunk_length(tokens: int, sequences: int, heads: int, d: int, e: int, slices: int, sms: int) -> int:
+    """Rows of a chunk of the recurrence, 0 for none, from a step's shapes alone (a recorded step keeps its choice): about two
+    blocks an SM, chunks of at least 64 rows, only for portions of 256 rows and more a sequence."""
+    if os.environ.get("MRS_LINEAR_SCAN_CHUNK"):             # the variable: for measuring other chunk lengths
+        return int(os.environ["MRS_LINEAR_SCAN_CHUNK"])
+    if tokens < 256 * sequences:
+        return 0
+    chunks = min((2 * sms) // max(sequences * heads * slices, 1), tokens // 64)
+    if chunks < 3:          # two chunks walk every row twice at twice the width: nothing is won
+        return 0
+    return -(-tokens // chunks)
+
+
+def linear_scan(rows: torch.Tensor, q_offset: int, k_offset: int, v_offset: int, decay: torch.Tensor | None, coef: torch.Tensor | None,
+                state: torch.Tensor, norm_state: torch.Tensor | None, positions, q_start, state_slots, out: torch.Tensor,
+                norm_out: torch.Tensor | None, heads: int, d: int, e: int, write_state: bool = True,
+                chunk_len: int | None = None) -> None:
+    """S_t = keep_t S_(t-1) + take_t k_t v_t^T, o_t = S_t^T q_t per (sequence, head), float32: q, k [heads * d] and v [heads * e]
+    are columns of the float32 `rows`; keep is `decay` [heads] (take = 1), or keep | take are the first 2 * heads columns of
+    `coef`; `state` [slots, heads, d, e] float32 (a view: dense within a slot), zero where a sequence starts at position 0;
+    `out` [tokens, heads * e].  With `norm_state` [slots, heads, d]: n_t likewise with k alone, `norm_out` [tokens, heads] gets
+    n_t . q_t.  `chunk_len` 0: every sequence in one go; n > 0: chunks of n rows side by side in three passes; None: chosen
+    from the step's shapes."""
+    global launch_count
+    tokens = rows.shape[0]
+    _need(rows, torch.float32, "projection")
+    if min(q_offset, k_offset, v_offset) < 0 or max(q_offset, k_offset) + heads * d > rows.shape[1] or v_offset + heads * e > rows.shape[1]:
+        raise InvalidRequest("linear_scan: q, k or v lie outside the rows")
+    if not 0 < d <= LINEAR_SCAN_MAX_DIM:
+        raise InvalidRequest(f"linear_scan: query/key heads of up to {LINEAR_SCAN_MAX_DIM} elements are built")
+    if (decay is None) == (coef is None):
+        raise InvalidRequest("linear_scan: either a decay a head or coefficients a token")
+    if decay is not None:
+        _need(decay, torch.float32, "decays", (heads,))
+    else:
+        _need(coef, torch.float32, "coefficients")
+        if coef.shape[0] != tokens or coef.shape[1] < 2 * heads:
+            raise InvalidRequest("linear_scan: keep and take of every head are wanted")
+    _check_matrix_state(state, heads, d, e, "linear_scan")
+    if (norm_state is None) != (norm_out is None):
+        raise InvalidRequest("linear_scan: a normaliser has a state and an output")
+    if norm_state is not None:
+        if norm_state.dtype != torch.float32 or tuple(norm_state.shape[1:]) != (heads, d) or norm_state.stride(2) != 1 or \
+                norm_state.stride(1) != d or norm_state.stride(0) != state.stride(0):
+            raise InvalidRequest("linear_scan: the normaliser's state must be float32 [slots, heads, d], dense within a slot, in the same slots")
+        _need(norm_out, torch.float32, "normaliser", (tokens, heads))
+    _need(out, torch.float32, "recurrence output", (tokens, heads * e))
+    sequences = state_slots.shape[0]
+    lib = linear_scan_library()
+    if chunk_len is None:
+        chunk_len = linear_scan_chunk_length(tokens, sequences, heads, d, e, lib.mrs_linear_scan_slices(d, e), sm_count(rows.device))
+    scratch = None
+    if chunk_len:
+        need = lib.mrs_linear_scan_scratch_floats(tokens, sequences, heads, d, e, int(norm_state is not None), int(chunk_len))
+        scratch = attention_scratch(rows.device, need, lane=2)
+        launch_count += 2
+    base = rows.data_ptr()
+    _check(lib.mrs_linear_scan(base + 4 * q_offset, base + 4 * k_offset, base + 4 * v_offset, rows.shape[1], _ptr(decay), _ptr(coef),
+                               coef.shape[1] if coef is not None else 0, state.data_ptr(), _ptr(norm_state), state.stride(0),
+                               positions.data_ptr(), q_start.data_ptr(), state_slots.data_ptr(), out.data_ptr(), _ptr(norm_out), tokens,
+                               sequences, heads, d, e, int(write_state), int(chunk_len), _ptr(scratch), _stream()), "linear_scan")
 
 
 # ------------------------------------------------------------------------------------------------

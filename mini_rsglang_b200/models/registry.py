@@ -8,11 +8,12 @@ import os
 from dataclasses import dataclass
 from typing import Callable
 
-from ..config.model_config import MigenexConfig, ModelConfig, NiduvikConfig, NubipelConfig, Qwen3Config, SatedraConfig
+from ..config.model_config import MigenexConfig, ModelConfig, NiduvikConfig, NubipelConfig, PisatarConfig, Qwen3Config, SatedraConfig
 from ..errors import InvalidRequest
 from .migenex import migenex_spec
 from .niduvik import niduvik_spec
 from .nubipel import nubipel_spec
+from .pisatar import pisatar_spec
 from .qwen3 import qwen3_spec
 from .satedra import satedra_spec
 from .spec import ModelSpec
@@ -39,6 +40,7 @@ register_architecture("niduvik", NiduvikConfig, niduvik_spec)
 register_architecture("satedra", SatedraConfig, satedra_spec)
 register_architecture("nubipel", NubipelConfig, nubipel_spec)
 register_architecture("migenex", MigenexConfig, migenex_spec)
+register_architecture("pisatar", PisatarConfig, pisatar_spec)
 
 
 def config_from_dict(raw: dict) -> ModelConfig:

@@ -188,9 +188,18 @@ class BiasedWindowAttention(Mixer):
             self.sinks = tensors[self.name(n["sink"])].float().contiguous()
 
     def forward(self, h, ctx, cache, write_cache=True):
-        tokens = h.shape[0]
+        return self.forward_projected(linear(h, self.fused, out_dtype=torch.float32), 0, ctx, cache, write_cache)
+
+    def projection(self):
+        # the kernel with rotations leaves the columns behind q, k and v alone; the others want rows of their own
+        return self.fused if self.rotary_store and self.output_gate is None else None
+
+    def forward_projected(self, proj, offset, ctx, cache, write_cache=True):
+        """From the float32 sums of the fused projection on (`offset` 0: this mixer's columns come first)."""
+        if offset:
+            raise InvalidRequest(f"{self.prefix}: an attention's columns come first in a shared projection")
+        tokens = proj.shape[0]
         device, dtype = self.o.device, self.runtime.dtype
-        proj = linear(h, self.fused, out_dtype=torch.float32)
         q = torch.empty((tokens, self.nq * self.d), dtype=dtype, device=device)
         gate = torch.empty((tokens, self.nq), dtype=torch.float32, device=device) if self.output_gate == "heads" else None
         v_first, mode = None, 0

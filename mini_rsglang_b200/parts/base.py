@@ -165,15 +165,24 @@ class Prenormed:
 @dataclass
 class Normed:
     """Rows that the norm after a block has been run on already, by the kernel that added the block's last
-    branch to the stream: `rows` = norm(stream) in the engine's dtype.  The stream holds the sum."""
+    branch to the stream: `rows` = norm(stream) in the engine's dtype (a pair of norms: a tuple of both norms' rows).
+    The stream holds the sum."""
 
-    rows: torch.Tensor
+    rows: Any
     norm: "Norm"
     stream: torch.Tensor
 
     @property
     def shape(self):
         return self.rows.shape
+
+
+@dataclass
+class BranchSum:
+    """A mixer's output as a sum that nobody has formed yet: the terms [(float32 [T, width], factor)].  A block whose kernel adds
+    several branches to the stream takes it as it is (`Mixer.gives_terms`)."""
+
+    terms: list
 
 
 def observing(ctx) -> bool:
@@ -269,8 +278,15 @@ class Mixer(Part):
     replayable = False
     adds_to_stream = False        # `forward` takes `into=ResidualLink` and may return a `Prenormed`
     takes_prenormed = False       # `forward` takes a `Prenormed` as `h`
+    gives_terms = False           # `forward` takes `as_terms=True` and then returns a `BranchSum`
 
     def cache_need(self) -> KVNeed | None:
+        return None
+
+    def projection(self) -> torch.Tensor | None:
+        """The rows of the one product by which this mixer reads its input ([rows, width], bound), if another part may run
+        that product together with its own; `forward_projected(proj, offset, ctx, cache, write_cache)` then goes on from the
+        float32 sums `proj`, this mixer's columns beginning at `offset`."""
         return None
 
     def step_signature(self, facts: "StepFacts"):

@@ -1,6 +1,7 @@
 """How a layer's parts are arranged.  "pre_norm": x + mixer(norm1(x)), then
 + feed_forward(norm2(.)) (reference: crates/models/src/qwen3.rs:176-225).  "sandwich_norm": a norm before and after
 each branch.  "parallel": both branches read one norm's output, x + (mixer(norm1(x)) + feed_forward(norm1(x))).
+"parallel_two_norms": each branch reads a norm of its own, x + (mixer(norm1(x)) + feed_forward(norm2(x))).
 
 The residual stream is float32.  A branch's output is not added by a kernel of its own: it
 is handed on as `pending`, and the next norm adds it while it reads the stream anyway; or,
@@ -13,6 +14,7 @@ import torch
 from .. import kernels
 from ..errors import InvalidRequest
 from .base import BLOCKS, FEED_FORWARDS, MIXERS, NORMS, Block, Normed, Prenormed, ResidualLink, observing, plain
+from .norm import NormPair
 
 
 def _branch(part, h, stream, norm, *args):
@@ -142,3 +144,59 @@ class ParallelBlock(Block):
         if observing(ctx):
             ctx.observe(f"{ctx.label}-output", stream.clone())
         return Normed(out, next_norm, stream) if fused else None
+
+
+@BLOCKS.register("parallel_two_norms")
+class ParallelTwoNormsBlock(Block):
+    """Both branches side by side, each on a norm of its own of the same stream: x <- x + (mixer(norm1(x)) +
+    feed_forward(norm2(x))); a layer may be a mixer alone (it then has no norm2).
+
+    The branches' last products leave float32 sums (a mixer may hand on several terms with factors); one kernel adds them all
+    to the float32 stream and runs the norms that read the stream next: both of the next layer's, which share their
+    statistic, or the one that stands there.  A layer is one norm launch."""
+
+    links_norms = True
+    roles = {"norm1": NORMS, "mixer": MIXERS, "norm2": NORMS, "feed_forward": FEED_FORWARDS}
+    optional_roles = ("norm2", "feed_forward")
+    entry_role = "norm1"
+
+    def __init__(self, prefix: str, **parts):
+        super().__init__(prefix, **parts)
+        if (self.norm2 is None) != (self.feed_forward is None):
+            raise InvalidRequest(f"block at {prefix!r}: a feed-forward comes with the norm before it")
+        self.pair = NormPair(self.norm1, self.norm2) if self.norm2 is not None else None
+
+    @property
+    def entry_norm(self):
+        return self.pair if self.pair is not None else self.norm1
+
+    def forward(self, stream, pending, ctx, cache, write_cache=True, next_norm=None):
+        if self.pair is not None:
+            h, h2 = self.pair.add_norm(stream, pending)
+        else:
+            h = plain(self.norm1.add_norm(stream, pending))
+        if observing(ctx):
+            ctx.observe(f"{ctx.label}-input_norm", h)
+        if self.mixer.gives_terms:
+            terms = list(self.mixer.forward(h, ctx, cache, write_cache, as_terms=True).terms)
+        else:
+            terms = [(self.mixer.forward(h, ctx, cache, write_cache), 1.0)]
+        if self.feed_forward is not None:
+            terms.append((self.feed_forward.forward(h2, ctx), 1.0))
+        terms = [(x if x.dtype is torch.float32 else x.float(), factor) for x, factor in terms]      # branches written for other arrangements
+        while len(terms) > kernels.MAX_BRANCHES:
+            kernels.add_scaled_branches_norms(stream, [terms.pop(0)], [], 0.0)
+        pending = None
+        if isinstance(next_norm, NormPair):
+            outs = next_norm.outputs(stream, self.runtime.dtype)
+            kernels.add_scaled_branches_norms(stream, terms, outs, next_norm.eps)
+            pending = Normed(tuple(out for _, out in outs), next_norm, stream)
+        elif next_norm is not None and getattr(next_norm, "rides_on_products", False) and not next_norm.gathers_rows:
+            out = torch.empty(stream.shape, dtype=self.runtime.dtype, device=stream.device)
+            kernels.add_scaled_branches_norms(stream, terms, [(next_norm.weight, out)], next_norm.eps)
+            pending = Normed(out, next_norm, stream)
+        else:
+            kernels.add_scaled_branches_norms(stream, terms, [], 0.0)
+        if observing(ctx):
+            ctx.observe(f"{ctx.label}-output", stream.clone())
+        return pending

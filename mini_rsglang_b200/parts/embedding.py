@@ -8,14 +8,16 @@ import torch
 from .. import kernels
 from ..errors import InvalidRequest
 from ..weights.spec import WeightSpec
-from .base import EMBEDDINGS, HEADS, Embedding, Head, StateNeed
+from .base import EMBEDDINGS, HEADS, NORMS, Embedding, Head, PartSpec, StateNeed
 from .linear import linear
 
 
 @EMBEDDINGS.register("token_embedding")
 class TokenEmbedding(Embedding):
-    def __init__(self, prefix: str, vocab: int, width: int, leaf: str = "weight", scale: float = 1.0, pairs: dict | None = None):
-        """`scale`: a constant that multiplies every embedding on its way into the float32 stream (the table is unchanged).
+    def __init__(self, prefix: str, vocab: int, width: int, leaf: str = "weight", scale: float = 1.0, pairs: dict | None = None,
+                 norm: PartSpec | None = None, norm_name: str = "norm"):
+        """`norm`: an RMS norm that the embeddings pass on their way into the stream, its tensors below `norm_name`.
+        `scale`: a constant that multiplies every embedding on its way into the float32 stream (the table is unchanged).
         `pairs`: a second table, of token pairs, whose row is added (unscaled): {"table": its checkpoint name, "buckets",
         "mul_prev", "mul_cur"}; a token takes row (previous token * mul_prev + token * mul_cur) mod buckets, the first token
         of a sequence row number `buckets` (the table has buckets + 1 rows).  The last token that a request brought is then
@@ -28,9 +30,14 @@ class TokenEmbedding(Embedding):
             if missing or int(self.pairs["buckets"]) <= 0:
                 raise InvalidRequest(f"a table of token pairs needs its name, a positive number of buckets and two multipliers; missing {missing}")
         self.table = self.pair_table = None
+        self.norm = NORMS.build(norm, self.name(norm_name)) if norm is not None else None
+        if self.norm is not None and (self.pairs is not None or self.scale != 1.0 or not self.norm.rides_on_products):
+            raise InvalidRequest("normed embeddings: an RMS norm, without a scale and without a table of token pairs")
 
     def weight_specs(self):
         specs = [WeightSpec(self.name(self.leaf), (self.vocab, self.width))]
+        if self.norm is not None:
+            specs += self.norm.weight_specs()
         if self.pairs is not None:
             specs.append(WeightSpec(self.pairs["table"], (int(self.pairs["buckets"]) + 1, self.width)))
         return specs
@@ -41,13 +48,17 @@ class TokenEmbedding(Embedding):
     def bind(self, tensors, runtime):
         super().bind(tensors, runtime)
         self.table = tensors[self.name(self.leaf)]
+        if self.norm is not None:
+            self.norm.bind(tensors, runtime)
         if self.pairs is not None:
             self.pair_table = tensors[self.pairs["table"]]
 
     def forward(self, ctx, state=None) -> torch.Tensor:
         """`state`: the requests' last tokens, int32 [slots] (an embedding with a table of pairs)."""
         stream = torch.empty((ctx.num_tokens, self.width), dtype=torch.float32, device=self.table.device)
-        if self.pairs is None:
+        if self.norm is not None:
+            kernels.embed_norm(self.table, ctx.token_ids, self.norm.weight, self.norm.eps, stream)
+        elif self.pairs is None:
             kernels.embed(self.table, ctx.token_ids, stream, self.scale)
         else:
             if state is None:

@@ -1,11 +1,13 @@
 """RMSNorm: y = x * rsqrt(mean(x^2) + eps) * weight, statistics in float32
-(reference: crates/kernels/src/ops.cu:66-78).  The weight multiplies plainly (no 1 + w).
+(reference: crates/kernels/src/ops.cu:66-78).  The weight multiplies plainly unless the checkpoint stores it as its
+distance from one (`weight_offset`): it is then held as offset + w in float32.
 LayerNorm: y = (x - mean) / sqrt(var + eps) * weight + bias, var the mean of the squared deviations."""
 from __future__ import annotations
 
 import torch
 
 from .. import kernels
+from ..errors import InvalidRequest
 from ..weights.spec import WeightSpec
 from .base import NORMS, Norm, Normed, Prenormed
 
@@ -14,18 +16,21 @@ from .base import NORMS, Norm, Normed, Prenormed
 class RMSNorm(Norm):
     rides_on_products = True
 
-    def __init__(self, prefix: str, width: int, eps: float, leaf: str = "weight"):
+    def __init__(self, prefix: str, width: int, eps: float, leaf: str = "weight", weight_offset: float = 0.0):
         super().__init__(prefix)
         self.width, self.eps = int(width), float(eps)
+        self.weight_offset = float(weight_offset)
         self.leaf = leaf                   # the weights' name below the part's root ("": the root itself)
         self.weight: torch.Tensor | None = None
 
     def weight_specs(self):
-        return [WeightSpec(self.name(self.leaf), (self.width,), "vector")]
+        return [WeightSpec(self.name(self.leaf), (self.width,), "offset_vector" if self.weight_offset else "vector")]
 
     def bind(self, tensors, runtime):
         super().bind(tensors, runtime)
         self.weight = tensors[self.name(self.leaf)]
+        if self.weight_offset:
+            self.weight = (self.weight + self.weight_offset).contiguous()
 
     def forward(self, x):
         out = torch.empty_like(x)
@@ -45,6 +50,34 @@ class RMSNorm(Norm):
         out = torch.empty((n, self.width), dtype=self.runtime.dtype, device=residual.device)
         kernels.add_rmsnorm(residual, delta, self.weight, self.eps, out, rows, write_back)
         return out
+
+
+class NormPair(Norm):
+    """Two RMS norms of one stream, read side by side: `add_norm` returns the rows of both.  They share their statistic, so
+    one kernel makes both (and adds the branches that came before); it is what a block with two entry norms hands to the
+    block before it as the norm that follows."""
+
+    def __init__(self, first: RMSNorm, second: RMSNorm):
+        super().__init__(first.prefix)
+        if not first.rides_on_products or not second.rides_on_products or (first.width, first.eps) != (second.width, second.eps):
+            raise InvalidRequest(f"norms at {first.prefix!r} and {second.prefix!r}: a pair is two RMS norms of one width and epsilon")
+        self.first, self.second = first, second
+        self.width, self.eps = first.width, first.eps
+
+    def outputs(self, stream, dtype) -> list:
+        """[(weight, rows to fill)] of both norms."""
+        return [(norm.weight, torch.empty(stream.shape, dtype=dtype, device=stream.device)) for norm in (self.first, self.second)]
+
+    def add_norm(self, residual, delta, rows=None, write_back=True):
+        if isinstance(delta, Normed) and delta.norm is self:
+            return delta.rows
+        if isinstance(delta, (Prenormed, Normed)):       # the stream holds the sum already
+            delta = None
+        if rows is not None or not write_back:
+            raise InvalidRequest("a pair of norms reads whole streams")
+        outs = self.outputs(residual, self.first.runtime.dtype)
+        kernels.add_scaled_branches_norms(residual, [(delta.float(), 1.0)] if delta is not None else [], outs, self.eps)
+        return tuple(out for _, out in outs)
 
 
 @NORMS.register("layernorm")

@@ -38,9 +38,12 @@ class RotaryPosition(PositionEncoding):
         power = torch.pow(torch.tensor(theta, dtype=torch.float64), 2.0 * j / head_dim)
         return 1.0 / power.to(torch.float32)
 
+    def frequencies(self) -> torch.Tensor:
+        return self.inverse_frequencies(self.rotary_dim, self.theta)
+
     def bind(self, tensors, runtime):
         super().bind(tensors, runtime)
-        frequencies = self.inverse_frequencies(self.rotary_dim, self.theta)
+        frequencies = self.frequencies()
         self.inv_freq = frequencies.to(runtime.device)
         self.shared_key = ("rotations", frequencies.numpy().tobytes())     # layers with the same frequencies share a step's table
 
@@ -57,6 +60,35 @@ class RotaryPosition(PositionEncoding):
         if shared is not None:
             shared[self.shared_key] = table
         return table
+
+
+@POSITION_ENCODINGS.register("banded_rope")
+class BandedRotaryPosition(RotaryPosition):
+    """Rotary positions whose slow pairs are slowed down further, for contexts beyond the length the model was trained at: with
+    a pair's wavelength l = 2 pi / f, a pair with l < original / high keeps its frequency f, one with l > original / low turns
+    by f / factor, and between the two bounds s = (original / l - low) / (high - low) blends them, (1 - s) f / factor + s f.
+    The table is made on the host in float64 and held in float32; cosines and sines are not scaled."""
+
+    def __init__(self, prefix: str, head_dim: int, theta: float, factor: float, low: float, high: float, original: float,
+                 rotary_dim: int | None = None, pairing: str = "split_half"):
+        super().__init__(prefix, head_dim, theta, rotary_dim, pairing)
+        self.factor, self.low, self.high, self.original = float(factor), float(low), float(high), float(original)
+        if min(self.factor, self.low, self.high, self.original) <= 0.0 or self.high < self.low:
+            raise InvalidRequest("banded rotary positions need positive numbers and bounds with low <= high")
+
+    def frequencies(self) -> torch.Tensor:
+        out = []
+        for i in range(self.rotary_dim // 2):
+            f = self.theta ** (-2.0 * i / self.rotary_dim)
+            turns = self.original * f / (2.0 * math.pi)          # turns of the pair over the original length
+            if turns > self.high:
+                out.append(f)
+            elif turns < self.low:
+                out.append(f / self.factor)
+            else:
+                s = (turns - self.low) / (self.high - self.low) if self.high > self.low else 0.0
+                out.append((1.0 - s) * f / self.factor + s * f)
+        return torch.tensor(out, dtype=torch.float64).to(torch.float32)
 
 
 @POSITION_ENCODINGS.register("yarn_rope")

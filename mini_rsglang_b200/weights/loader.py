@@ -54,7 +54,7 @@ def open_checkpoint(folder: str) -> dict[str, StoredTensor]:
 
 
 def held_dtype(role: str, engine_dtype: torch.dtype) -> torch.dtype:
-    if role in ("vector", "bias"):
+    if role in ("vector", "offset_vector", "bias"):
         return torch.float32
     if role == "int_table":
         return torch.int32

@@ -38,9 +38,11 @@ def random_tensor(spec: WeightSpec, seed: int, dtype: torch.dtype,
     gen.manual_seed(_stream_seed(seed, spec.name))
     if spec.role == "int_table":
         return torch.randint(0, 2**15, spec.shape, generator=gen, device=device, dtype=torch.int32)
-    values = torch.empty(spec.shape, dtype=torch.float32 if spec.role in ("vector", "bias") else dtype, device=device)
+    values = torch.empty(spec.shape, dtype=torch.float32 if spec.role in ("vector", "offset_vector", "bias") else dtype, device=device)
     if spec.role == "vector":
         values.normal_(1.0, VECTOR_STD, generator=gen)
+    elif spec.role == "offset_vector":
+        values.normal_(0.0, VECTOR_STD, generator=gen)
     elif spec.role == "bias":
         values.normal_(0.0, BIAS_STD, generator=gen)
     else:

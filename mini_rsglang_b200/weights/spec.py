@@ -11,6 +11,7 @@ class WeightSpec:
       (bfloat16 when serving, float32 on the 32-bit path); drawn N(0, 0.02);
     - "vector": a norm's scale; always held in float32 (widening bfloat16 is exact, a tensor
       stored in 32-bit stays so); drawn 1 + N(0, 0.05);
+    - "offset_vector": a norm's scale stored as its distance from one; held in float32; drawn N(0, 0.05);
     - "bias": a bias, a small table or a constant of a recurrence, wanted in full precision; always held in
       float32; drawn N(0, 0.5);
     - "int_table": integers; held as int32.
