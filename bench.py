@@ -298,12 +298,38 @@ def looped_configs(size: dict, vocab: int = 32768):
     return migenex, latent_configs(size, vocab)[0]
 
 
+def recurrent_configs(size: dict, vocab: int = 32768):
+    """Pisatar at these layer sizes: four layers (a retention, a channel-decayed delta rule, attention beside a matrix memory, a
+    retention) that are run twice, the second four with the weights of the first and states of their own (eight layer runs).
+    The retention has width / 128 heads of 128 query/key and 256 value elements; the delta rule width / 128 heads of 128 value
+    elements, a quarter as many query/key heads of 128, 4 taps, thin products of 128; the attention heads of 128, rotated whole,
+    and beside it width / 512 memory heads of 256 query/key and 512 value elements; every layer with the gated feed-forward
+    beside its mixer.  Beside it Nubipel, the engine's other model of parallel branches with a delta rule, at equal width,
+    heads, feed-forward and depth."""
+    w = size["width"]
+    mlp = {"kind": "dense", "ff": size["ff"]}
+    heads = w // 128
+    retention = {"type": "retention", "mlp": mlp, "mixer": {"heads": heads, "dim": 128, "vdim": 256, "rot": {"base": 10000.0, "dims": 128},
+                                                            "decay": [1.0 - 2.0 ** (-5.0 - 7.0 * i / heads) for i in range(heads)]}}
+    delta = {"type": "channel_delta", "mlp": mlp, "mixer": {"heads": heads, "kv_heads": max(w // 512, 1), "dim": 128, "vdim": 128, "conv": 4,
+                                                            "decay_rank": 128, "gate_rank": 128}}
+    both = {"type": "parallel", "mlp": mlp, "mixer": {
+        "left": {"heads": size["heads"], "kv_heads": size["kv_heads"], "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
+                 "rot": {"base": 500000.0, "dims": 128, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}},
+        "right": {"heads": w // 512, "dim": 256, "vdim": 512, "gate_cap": 15.0}, "left_scale": 0.7, "right_scale": 0.7}}
+    first = (retention, delta, both, retention)
+    layers = [first[i] if i < 4 else dict(first[i % 4], weights_of=i % 4) for i in range(size["layers"])]
+    pisatar = {"architecture": "Pisatar", "vocab": vocab, "width": w, "norm": {"eps": 1e-6}, "layers": layers}
+    return pisatar, parallel_configs(size, vocab)[0]
+
+
 # design: (title, what stands beside it, the key of that model in the output, the two configurations)
 DESIGNS = {"niduvik": ("Niduvik", "Qwen3 of equal width, heads, feed-forward and depth", "qwen3", hybrid_configs),
            "satedra": ("Satedra", "Qwen3 of equal width, heads and depth, its feed-forward as wide as the experts a token passes", "qwen3",
                        latent_configs),
            "nubipel": ("Nubipel", "Niduvik of equal width, heads, feed-forward and depth", "niduvik", parallel_configs),
-           "migenex": ("Migenex", "Satedra of equal width, heads, experts and depth", "satedra", looped_configs)}
+           "migenex": ("Migenex", "Satedra of equal width, heads, experts and depth", "satedra", looped_configs),
+           "pisatar": ("Pisatar", "Nubipel of equal width, heads, feed-forward and depth", "nubipel", recurrent_configs)}
 
 
 def hybrid_run(args, torch, peak: dict) -> dict:

@@ -19,6 +19,7 @@
 //                     inputs staged through shared memory ahead of their use
 //   head_norm_gate    o / rms(o) * weight * act(gate) per (token, head), o first divided by a normaliser where there is one
 #include "common.cuh"
+#include "pairs.cuh"
 
 namespace {
 
@@ -35,7 +36,7 @@ __global__ void delta_prepare_kernel(float* __restrict__ qkv, int qkv_width, con
     pdl_launch_dependents();
     pdl_wait();
     const size_t t = blockIdx.x;
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
+    const int lane = threadIdx.x & 31, warp = blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5), warps = gridDim.y * (blockDim.x >> 5);
     float* row = qkv + t * qkv_width;
     for (int unit = warp; unit < 2 * groups; unit += warps) {          // units 0 .. groups - 1: q; the rest: k
         float* x = row + (size_t)unit * d;
@@ -46,7 +47,8 @@ __global__ void delta_prepare_kernel(float* __restrict__ qkv, int qkv_width, con
     }
     const float* r = raw + t * raw_stride;
     if (channels) {
-        for (int h = threadIdx.x; h < heads; h += blockDim.x) coef[t * heads + h] = 1.0f / (1.0f + expf(-r[b_offset + h]));
+        if (blockIdx.y == 0)
+            for (int h = threadIdx.x; h < heads; h += blockDim.x) coef[t * heads + h] = 1.0f / (1.0f + expf(-r[b_offset + h]));
         float* z = channels + t * channels_stride;
         for (int h = warp; h < heads; h += warps) {
             const float rate = -expf(a_log[h]);
@@ -54,6 +56,7 @@ __global__ void delta_prepare_kernel(float* __restrict__ qkv, int qkv_width, con
         }
         return;
     }
+    if (blockIdx.y != 0) return;
     for (int h = threadIdx.x; h < heads; h += blockDim.x) {
         coef[t * 2 * heads + h] = 1.0f / (1.0f + expf(-r[b_offset + h]));
         coef[t * 2 * heads + heads + h] = expf(-expf(a_log[h]) * softplus_f(r[a_offset + h] + dt_bias[h]));
@@ -70,21 +73,44 @@ __device__ __forceinline__ void copy_async4(void* dst, const void* src) {
 __device__ __forceinline__ void copy_async_commit() { asm volatile("cp.async.commit_group;\n" ::); }
 template <int N> __device__ __forceinline__ void copy_async_wait() { asm volatile("cp.async.wait_group %0;\n" ::"n"(N)); }
 
-// Thread (column c of the block's slice, part p): rows p * PER .. p * PER + PER - 1 of column c of S in registers (PER is
-// 16 or 8, the launcher's choice); the
-// PARTS lanes of one column are neighbours, so that the two sums over d are log2(PARTS) shuffles.  The tokens' inputs (k and
+// Thread (column c of the block's slice, part p): rows p * PER .. p * PER + PER - 1 of column c of S in registers, two to a
+// register pair (PER is 16 or 8, the launcher's choice); the PARTS lanes of one column lie in one warp, so that the two sums
+// over d are log2(PARTS) shuffles.  The tokens' inputs (k and
 // q of the head's group, the slice of v, beta and g; CHANNEL: also the head's d decays) come in batches of `batch_tokens` through two stages of shared memory:
 // the next batch is copied while this one is computed, and the threads of a block share what they read.  A token in shared
 // memory: k [PARTS * PITCH] | q [PARTS * PITCH] (| decays [PARTS * PITCH]) | v [cols rounded up to 4] | beta, g, 0, 0, with PITCH = PER + 4, so that
 // the 16-byte reads of the parts fall on different banks; the rows beyond d stay zero.
 //
 // One warp a scheduler is all that a single sequence offers, so every instruction's latency shows.  What a thread copies is
-// therefore the same in every batch and worked out once, ahead of the loop (`Copies`); and the chain from token to token is
-// only: the sum over S's old rows times k, the shuffles, u, one fused multiply-add a row.  The decay is applied to S beside
-// the shuffles (r = g * sum(S_old k)), and the read-out of one token overlaps the next one's chain.
+// therefore the same in every batch and worked out once, ahead of the loop (`Copies`); and the chain from token to token is only: the sum over S's old rows times k (CHANNEL: times k
+// already multiplied by the decays), the shuffles, u, one fused multiply-add a row.  The decay is applied to S beside the
+// shuffles, and a token's read-out is summed over its lanes by the next token's shuffles.
 template <int N>
 struct Copies {
     int src[N], dst[N], token[N];      // offsets in floats from the batch's first row and from the stage; a huge token: none
+};
+
+// What a thread needs of one token.
+template <int PER, bool CHANNEL>
+struct Token {
+    pair k[PER / 2], q[PER / 2], fade[CHANNEL ? PER / 2 : 1], faded[CHANNEL ? PER / 2 : 1];      // faded: k times the decays
+    float v, beta, decay;
+
+    __device__ __forceinline__ void read(const float* token, int rows, int tail_at, int cols_pad, int col_in_slice) {
+#pragma unroll
+        for (int i = 0; i < PER / 2; i += 2) {
+            const ulonglong2 kk = *reinterpret_cast<const ulonglong2*>(token + 2 * i);
+            const ulonglong2 qq = *reinterpret_cast<const ulonglong2*>(token + rows + 2 * i);
+            k[i] = kk.x, k[i + 1] = kk.y, q[i] = qq.x, q[i + 1] = qq.y;
+            if (CHANNEL) {
+                const ulonglong2 ff = *reinterpret_cast<const ulonglong2*>(token + 2 * rows + 2 * i);
+                fade[i] = ff.x, fade[i + 1] = ff.y;
+                faded[i] = mul2(kk.x, ff.x), faded[i + 1] = mul2(kk.y, ff.y);
+            }
+        }
+        const float* tail = token + tail_at;
+        v = (tail - cols_pad)[col_in_slice], beta = tail[0], decay = CHANNEL ? 1.0f : tail[1];
+    }
 };
 
 template <int PER, int PARTS, bool CHANNEL>
@@ -108,16 +134,21 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(const float* __restrict
     const int first = q_start[seq], last = q_start[seq + 1];
     const int slot = state_slots[seq];
     if (slot < 0 || last <= first) return;
-    const int part = threadIdx.x % PARTS, col_in_slice = threadIdx.x / PARTS, col = blockIdx.z * cols + col_in_slice;
+    // a warp's GROUPS columns lie side by side in its lanes: a 16-byte read by half a warp then has few distinct addresses
+    constexpr int GROUPS = 32 / PARTS;
+    const int lane = threadIdx.x & 31, part = lane / GROUPS, col_in_slice = (threadIdx.x >> 5) * GROUPS + lane % GROUPS;
+    const int col = blockIdx.z * cols + col_in_slice;
     const bool live = col < e;                       // a slice may overhang the head; its threads still take part in the shuffles
     const int c = live ? col : 0;
     const int group = head / (heads / groups);
     const int row0 = part * PER;
     float* mine = state + (long long)slot * state_stride + ((size_t)head * d) * e + c;
-    float s[PER];
+    pair s[PER / 2];                                 // the rows two by two
     const bool fresh = positions[first] == 0;
 #pragma unroll
-    for (int i = 0; i < PER; ++i) s[i] = (!fresh && live && row0 + i < d) ? mine[(size_t)(row0 + i) * e] : 0.0f;
+    for (int i = 0; i < PER; i += 2)
+        s[i / 2] = make_pair((!fresh && live && row0 + i < d) ? mine[(size_t)(row0 + i) * e] : 0.0f,
+                             (!fresh && live && row0 + i + 1 < d) ? mine[(size_t)(row0 + i + 1) * e] : 0.0f);
 
     const int q_at = group * d, k_at = (groups + group) * d, v_at = 2 * groups * d + head * e + (int)blockIdx.z * cols;
     const int live_cols = min(cols, e - (int)blockIdx.z * cols);
@@ -192,6 +223,8 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(const float* __restrict
     float* out_at = out + (size_t)first * heads * e + (size_t)head * e + c;
     const size_t out_step = (size_t)heads * e;
     const bool writes = live && part == 0;
+    float y = 0.0f;                                       // this lane's part of the last token's read-out
+    bool pending = false;
     issue(first, min(batch_tokens, last - first), 0);
     for (int b = 0; b < batches; ++b) {
         const int t0 = first + b * batch_tokens, n = min(batch_tokens, last - t0);
@@ -203,53 +236,46 @@ __global__ void __launch_bounds__(128) delta_scan_kernel(const float* __restrict
         }
         __syncthreads();
         const float* token = stage + (b & 1) * stage_floats + part * PITCH;
-#pragma unroll 2
-        for (int j = 0; j < n; ++j, token += token_floats, out_at += out_step) {
-            float k[PER], q[PER], fade[CHANNEL ? PER : 1];
+#pragma unroll 1
+        for (int j = 0; j < n; ++j, token += token_floats) {
+            Token<PER, CHANNEL> now;
+            now.read(token, ROWS, token_tail - part * PITCH, cols_pad, col_in_slice);
+            pair r2[2] = {0ull, 0ull};
 #pragma unroll
-            for (int i = 0; i < PER; i += 4) {
-                if (CHANNEL) {
-                    const float4 ff = *reinterpret_cast<const float4*>(token + 2 * ROWS + i);
-                    fade[i] = ff.x, fade[i + 1] = ff.y, fade[i + 2] = ff.z, fade[i + 3] = ff.w;
-                }
-                const float4 kk = *reinterpret_cast<const float4*>(token + i);
-                const float4 qq = *reinterpret_cast<const float4*>(token + ROWS + i);
-                k[i] = kk.x, k[i + 1] = kk.y, k[i + 2] = kk.z, k[i + 3] = kk.w;
-                q[i] = qq.x, q[i + 1] = qq.y, q[i + 2] = qq.z, q[i + 3] = qq.w;
+            for (int i = 0; i < PER / 2; ++i) r2[i & 1] = fma2(s[i], CHANNEL ? now.faded[CHANNEL ? i : 0] : now.k[i], r2[i & 1]);
+            float r = both(r2[0]) + both(r2[1]);
+#pragma unroll
+            for (int o = GROUPS; o < 32; o <<= 1) {                   // this token's sum and the one before's read-out side by side
+                const float other_r = __shfl_xor_sync(0xffffffffu, r, o), other_y = __shfl_xor_sync(0xffffffffu, y, o);
+                r += other_r, y += other_y;
             }
-            const float* tail = token - part * PITCH + token_tail;
-            const float v = (tail - cols_pad)[col_in_slice], beta = tail[0], decay = CHANNEL ? 1.0f : tail[1];
-            if (CHANNEL) {                                               // S forgets before the correction reads it
+            if (writes && pending) *out_at = y, out_at += out_step;
+            pending = true;
+            const pair decays = make_pair(now.decay, now.decay);
 #pragma unroll
-                for (int i = 0; i < PER; ++i) s[i] *= fade[i];
+            for (int i = 0; i < PER / 2; ++i) s[i] = mul2(s[i], CHANNEL ? now.fade[CHANNEL ? i : 0] : decays);      // off the chain
+            const float u = now.beta * (now.v - (CHANNEL ? r : now.decay * r));
+            const pair uu = make_pair(u, u);
+            pair y2[2] = {0ull, 0ull};
+#pragma unroll
+            for (int i = 0; i < PER / 2; ++i) {
+                s[i] = fma2(now.k[i], uu, s[i]);
+                y2[i & 1] = fma2(s[i], now.q[i], y2[i & 1]);
             }
-            float r4[4] = {0.0f, 0.0f, 0.0f, 0.0f};
-#pragma unroll
-            for (int i = 0; i < PER; ++i) r4[i & 3] = fmaf(s[i], k[i], r4[i & 3]);
-            float r = (r4[0] + r4[1]) + (r4[2] + r4[3]);
-#pragma unroll
-            for (int o = PARTS >> 1; o > 0; o >>= 1) r += __shfl_xor_sync(0xffffffffu, r, o);
-#pragma unroll
-            for (int i = 0; i < PER; ++i)
-                if (!CHANNEL) s[i] *= decay;                             // beside the shuffles, off the chain
-            const float u = beta * (v - decay * r);
-            float y4[4] = {0.0f, 0.0f, 0.0f, 0.0f};
-#pragma unroll
-            for (int i = 0; i < PER; ++i) {
-                s[i] = fmaf(k[i], u, s[i]);
-                y4[i & 3] = fmaf(s[i], q[i], y4[i & 3]);
-            }
-            float y = (y4[0] + y4[1]) + (y4[2] + y4[3]);
-#pragma unroll
-            for (int o = PARTS >> 1; o > 0; o >>= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
-            if (writes) *out_at = y;
+            y = both(y2[0]) + both(y2[1]);
         }
         __syncthreads();                                  // the stage is copied into again two batches on
     }
+#pragma unroll
+    for (int o = GROUPS; o < 32; o <<= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
+    if (writes) *out_at = y;                              // the last token's
     if (write_state && live) {
 #pragma unroll
-        for (int i = 0; i < PER; ++i)
-            if (row0 + i < d) mine[(size_t)(row0 + i) * e] = s[i];
+        for (int i = 0; i < PER; i += 2) {
+            const float2 x = split(s[i / 2]);
+            if (row0 + i < d) mine[(size_t)(row0 + i) * e] = x.x;
+            if (row0 + i + 1 < d) mine[(size_t)(row0 + i + 1) * e] = x.y;
+        }
     }
 }
 
@@ -359,8 +385,9 @@ MRS_EXPORT int mrs_delta_prepare(float* qkv, const float* raw, int raw_stride, i
     if (tokens <= 0) return 0;
     if (groups <= 0 || d <= 0 || heads <= 0 || e <= 0 || heads % groups) return MRS_BAD_ARGUMENT;
     const int units = 2 * groups;
-    const int threads = units >= 8 ? 256 : (units >= 4 ? 128 : 64);
-    MRS_LAUNCH(delta_prepare_kernel, tokens, threads, 0, stream, qkv, 2 * groups * d + heads * e, raw, raw_stride, b_offset, a_offset,
+    const int threads = units >= 8 || channels ? 256 : (units >= 4 ? 128 : 64);
+    const int across = channels && tokens < mrs_sm_count() ? 4 : 1;      // few tokens: their heads' decays over several blocks
+    MRS_LAUNCH(delta_prepare_kernel, dim3(tokens, across), threads, 0, stream, qkv, 2 * groups * d + heads * e, raw, raw_stride, b_offset, a_offset,
                a_log, dt_bias, coef, channels, channels_stride, groups, d, heads, unit_eps, q_factor);
     MRS_RETURN_LAUNCH_STATUS();
 }
@@ -386,9 +413,10 @@ MRS_EXPORT int mrs_delta_scan(const float* qkv, const float* coef, const float* 
         slices = (e + cols - 1) / cols;
     };
     // rows of a column a thread: 16; 8 where long portions come as more blocks than multiprocessors, so that more of them
-    // are resident side by side (measured: from 1.1 to 1.3 times as fast there, slower for short portions and few blocks)
+    // are resident side by side (measured: from 1.1 to 1.3 times as fast there, slower for short portions and few blocks), and
+    // for all long portions with a decay a channel (535 against 624 us for 2,048 tokens of 16 heads)
     plan(16);
-    if (d <= 256 && tokens >= 256LL * sequences && pairs * slices > mrs_sm_count()) plan(8);
+    if (d <= 256 && tokens >= 256LL * sequences && (channels || pairs * slices > mrs_sm_count())) plan(8);
     if (slices > 65535) return MRS_BAD_ARGUMENT;
     const int qkv_width = 2 * groups * d + heads * e;
     const int token_floats = (channels ? 3 : 2) * parts * (per + 4) + ((cols + 3) & ~3) + 4;

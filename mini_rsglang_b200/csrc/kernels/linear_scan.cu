@@ -13,6 +13,7 @@
 //   linear_scan        the recurrence
 //   narrow_columns     a range of float32 columns as rows of the engine's dtype
 #include "common.cuh"
+#include "pairs.cuh"
 
 namespace {
 
@@ -127,14 +128,16 @@ __global__ void memory_gates_kernel(const float* __restrict__ raw, int raw_strid
 }
 
 // ---------------------------------------------------------------------------------------------
-// The recurrence.  A thread keeps SCAN_ROWS rows x 4 neighbouring columns of S in registers; the PARTS lanes that share four
-// columns cover the d rows, so what a thread reads of k and q from shared memory serves four columns, and a token's
-// read-out is a reduction that hands its columns out while it sums (2 + 1 + 1 ... shuffles).  The tokens' k, q, v and gates
+// The recurrence.  A thread keeps SCAN_ROWS rows x 4 neighbouring columns of S in registers, two rows to a 64-bit register
+// pair, so that one instruction (fma.rn.f32x2, two independent float32 multiply-adds) serves two rows; the PARTS lanes that
+// share four columns cover the d rows, so what a thread reads of k and q from shared memory serves four columns, and a
+// token's read-out is a reduction that hands its columns out while it sums (2 + 1 + 1 ... shuffles).  The tokens' k, q and v
 // come through two stages of shared memory, filled by cp.async a batch ahead.
 //
 // The decay costs no instruction an element: with P the product of the keeps since S was last rescaled, the registers hold
-// S / P, a token adds (take / P) k v^T and its read-out is P (S / P)^T q; where P falls below SCAN_LEAST the registers are
-// multiplied by it and P starts again at 1.
+// S / P, a token adds (take / P) k v^T and its read-out is P (S / P)^T q.  A batch's prefix products are made by one warp a
+// batch ahead; where P would fall below SCAN_LEAST within a batch the registers are first multiplied by it and P starts
+// again at 1, and a batch whose own product falls below it is walked with the decay applied token by token.
 //
 // SCAN_WHOLE: a sequence's rows in one go, from the slot's state to the slot's state.  Long portions of few sequences are cut
 // into chunks of `chunk_len` rows that run side by side: SCAN_LOCAL runs every chunk from zero and leaves its end state and
@@ -144,13 +147,14 @@ __global__ void memory_gates_kernel(const float* __restrict__ raw, int raw_strid
 #define SCAN_ROWS 16
 #define SCAN_PITCH (SCAN_ROWS + 4)       // 16-byte reads of the parts fall on different banks
 #define SCAN_LEAST 1e-8f
+#define SCAN_BATCH 8                     // tokens a batch, at most
 enum { SCAN_WHOLE = 0, SCAN_LOCAL = 1, SCAN_FINAL = 2 };
 
 struct ScanArgs {
     const float *q, *k, *v;              // columns of float32 rows of `stride` floats; heads of d, d and e elements
     int stride;
     const float* decay;                  // [heads], or null: the coefficients
-    const float* coef;                   // [tokens, coef_stride]: keep of every head, then take
+    const float* coef;                   // [tokens, coef_stride]: keep of every head, then take; keeps lie in 0 .. 1
     int coef_stride;
     float* state;                        // [slots][heads, d, e]
     float* norm_state;                   // [slots][heads, d], or null: no normaliser
@@ -171,13 +175,15 @@ __device__ __forceinline__ void scan_copy4(float* to, const float* from) {
 }
 
 template <int MODE, int PARTS>
-__global__ void __launch_bounds__(256) linear_scan_kernel(const ScanArgs A) {
+__global__ void __launch_bounds__(256, 2) linear_scan_kernel(const ScanArgs A) {
     extern __shared__ __align__(16) float stage[];
+    __shared__ __align__(16) float4 facts[2][SCAN_BATCH];    // of a token: take / p, p, keep, take; p the batch's product of keeps so far
     constexpr int GROUPS = 32 / PARTS;                       // groups of four columns a warp covers
     constexpr int VECTOR = PARTS * SCAN_PITCH;               // floats of a k (or q) in shared memory
+    constexpr int PAIRS = SCAN_ROWS / 2;
     pdl_launch_dependents();
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
-    const int token_floats = 2 * VECTOR + A.cols + 4, stage_floats = A.batch * token_floats;
+    const int token_floats = 2 * VECTOR + A.cols, stage_floats = A.batch * token_floats;
     for (int i = threadIdx.x; i < 2 * stage_floats; i += blockDim.x) stage[i] = 0.0f;      // rows beyond d, columns beyond e
     __syncthreads();
     pdl_wait();
@@ -190,7 +196,10 @@ __global__ void __launch_bounds__(256) linear_scan_kernel(const ScanArgs A) {
     if (first >= last) return;
     const int part = lane / GROUPS, place = (warp * GROUPS + lane % GROUPS) * 4, col = slice * A.cols + place;
     const int row0 = part * SCAN_ROWS;
-    const bool owns_norm = A.norm_state != nullptr && slice == 0 && warp == 0;
+    // a normaliser is one more column behind S's (at a multiple of four), whose value is always 1
+    const int norm_col = A.norm_state ? (A.e + 3) / 4 * 4 : -4;
+    const bool is_norm = col == norm_col;
+    const bool idle = slice * A.cols + warp * GROUPS * 4 >= max(A.e, norm_col + 4);      // a warp without columns
     const size_t chunk_at = (((size_t)seq * A.heads + head) * A.max_chunks + chunk);
     float* mine = MODE == SCAN_WHOLE ? A.state + (long long)slot * A.state_stride + (size_t)head * A.d * A.e : A.chunk_state + chunk_at * A.chunk_floats;
     float* norm_mine = MODE == SCAN_WHOLE ? A.norm_state + (long long)slot * A.state_stride + (size_t)head * A.d : mine + (size_t)A.d * A.e;
@@ -220,168 +229,236 @@ __global__ void __launch_bounds__(256) linear_scan_kernel(const ScanArgs A) {
             } else {
                 for (int i = lane; i < live_cols; i += 32) scan_copy4(to + 2 * VECTOR + i, A.v + row + v_at + i);
             }
-            if (A.coef && lane < 2) scan_copy4(to + 2 * VECTOR + A.cols + lane, A.coef + (size_t)(t0 + j) * A.coef_stride + lane * A.heads + head);
         }
         asm volatile("cp.async.commit_group;\n" ::);
     };
-    issue(first, min(A.batch, last - first), 0);
-
-    float4 s[SCAN_ROWS];
-    float norm[SCAN_ROWS];
-#pragma unroll
-    for (int i = 0; i < SCAN_ROWS; ++i) {
-        s[i] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-        norm[i] = 0.0f;
-        if (!zero && row0 + i < A.d) {
-            const float* from = mine + (size_t)(row0 + i) * A.e + col;
-            if (A.vec_state) {
-                if (col < A.e) s[i] = *reinterpret_cast<const float4*>(from);
-            } else {
-                if (col < A.e) s[i].x = from[0];
-                if (col + 1 < A.e) s[i].y = from[1];
-                if (col + 2 < A.e) s[i].z = from[2];
-                if (col + 3 < A.e) s[i].w = from[3];
-            }
-            if (owns_norm) norm[i] = norm_mine[row0 + i];
-        }
-    }
     const float fixed = A.decay ? A.decay[head] : 1.0f;
+    auto read_facts = [&](int t0, int n) {                   // keep and take of token t0 + lane, warp 0
+        if (A.decay || lane >= n) return make_float2(lane < n ? fixed : 1.0f, 1.0f);
+        const float* c = A.coef + (size_t)(t0 + lane) * A.coef_stride + head;
+        return make_float2(c[0], c[A.heads]);
+    };
+    auto write_facts = [&](float2 raw, int buffer) {
+        float p = raw.x;
+#pragma unroll
+        for (int o = 1; o < SCAN_BATCH; o <<= 1) {
+            const float before = __shfl_up_sync(0xffffffffu, p, o);
+            if (lane >= o) p *= before;
+        }
+        if (lane < A.batch) facts[buffer][lane] = make_float4(raw.y / p, p, raw.x, raw.y);
+    };
+    issue(first, min(A.batch, last - first), 0);
+    if (warp == 0) write_facts(read_facts(first, min(A.batch, last - first)), 0);
+
+    pair s[4][PAIRS];                                        // a column's rows two by two
+#pragma unroll
+    for (int i = 0; i < PAIRS; ++i) {
+        float x[4][2] = {{0.0f, 0.0f}, {0.0f, 0.0f}, {0.0f, 0.0f}, {0.0f, 0.0f}};
+#pragma unroll
+        for (int u = 0; u < 2; ++u) {
+            const int row = row0 + 2 * i + u;
+            if (zero || row >= A.d) continue;
+            const float* from = mine + (size_t)row * A.e + col;
+            if (A.vec_state) {
+                if (col < A.e) {
+                    const float4 f = *reinterpret_cast<const float4*>(from);
+                    x[0][u] = f.x, x[1][u] = f.y, x[2][u] = f.z, x[3][u] = f.w;
+                }
+            } else {
+#pragma unroll
+                for (int c = 0; c < 4; ++c)
+                    if (col + c < A.e) x[c][u] = from[c];
+            }
+            if (is_norm) x[0][u] = norm_mine[row];
+        }
+#pragma unroll
+        for (int c = 0; c < 4; ++c) s[c][i] = make_pair(x[c][0], x[c][1]);
+    }
+    auto rescale = [&](float by) {
+        const pair f = make_pair(by, by);
+#pragma unroll
+        for (int i = 0; i < PAIRS; ++i) {
+#pragma unroll
+            for (int c = 0; c < 4; ++c) s[c][i] = mul2(s[c][i], f);
+        }
+    };
+    // one token: `weight` multiplies what is added, `factor` what is read
+    float* to = A.out + (size_t)first * A.heads * A.e + (size_t)head * A.e + col;
+    if (is_norm) to = A.norm_out + (size_t)first * A.heads + head;
+    const size_t out_step = is_norm ? A.heads : (size_t)A.heads * A.e;
+    const int live = is_norm ? 1 : A.e - col;                // columns of these four that are there
+    auto walk = [&](const float* token, float weight, float factor) {
+        float4 vv = *reinterpret_cast<const float4*>(token + 2 * VECTOR + place);
+        if (is_norm) vv.x = 1.0f;                            // the columns behind e are zero
+        const pair tv[4] = {make_pair(vv.x * weight, vv.x * weight), make_pair(vv.y * weight, vv.y * weight),
+                            make_pair(vv.z * weight, vv.z * weight), make_pair(vv.w * weight, vv.w * weight)};
+        pair y[4];
+        const float* kp = token + part * SCAN_PITCH;
+#pragma unroll
+        for (int i = 0; i < PAIRS; i += 2) {
+            const ulonglong2 kk = *reinterpret_cast<const ulonglong2*>(kp + 2 * i);
+            ulonglong2 qq = make_ulonglong2(0ull, 0ull);
+            if (MODE != SCAN_LOCAL) qq = *reinterpret_cast<const ulonglong2*>(kp + VECTOR + 2 * i);
+#pragma unroll
+            for (int c = 0; c < 4; ++c) {
+                s[c][i] = fma2(kk.x, tv[c], s[c][i]);
+                s[c][i + 1] = fma2(kk.y, tv[c], s[c][i + 1]);
+                if (MODE != SCAN_LOCAL) {
+                    y[c] = i == 0 ? mul2(s[c][i], qq.x) : fma2(s[c][i], qq.x, y[c]);
+                    y[c] = fma2(s[c][i + 1], qq.y, y[c]);
+                }
+            }
+        }
+        if (MODE == SCAN_LOCAL) return;
+        const float z[4] = {both(y[0]), both(y[1]), both(y[2]), both(y[3])};
+        if (PARTS == 1) {
+            if (A.vec_out && !is_norm) {
+                if (live > 0) *reinterpret_cast<float4*>(to) = make_float4(z[0] * factor, z[1] * factor, z[2] * factor, z[3] * factor);
+            } else {
+#pragma unroll
+                for (int c = 0; c < 4; ++c)
+                    if (c < live) to[c] = z[c] * factor;
+            }
+            return;
+        }
+        const bool upper = part & 1;                         // this lane goes on with the upper two of the four columns
+        float z0 = upper ? z[2] : z[0], z1 = upper ? z[3] : z[1];
+        z0 += __shfl_xor_sync(0xffffffffu, upper ? z[0] : z[2], GROUPS);
+        z1 += __shfl_xor_sync(0xffffffffu, upper ? z[1] : z[3], GROUPS);
+        const int at = upper ? 2 : 0;
+        if (PARTS == 2) {
+            if (at < live) to[at] = z0 * factor;
+            if (at + 1 < live) to[at + 1] = z1 * factor;
+            return;
+        }
+        const bool second = part & 2;
+        float one = second ? z1 : z0;
+        one += __shfl_xor_sync(0xffffffffu, second ? z0 : z1, 2 * GROUPS);
+#pragma unroll
+        for (int o = 4 * GROUPS; o < 32; o <<= 1) one += __shfl_xor_sync(0xffffffffu, one, o);
+        if (part < 4 && at + (second ? 1 : 0) < live) to[at + (second ? 1 : 0)] = one * factor;
+    };
+
     float P = 1.0f, product = 1.0f;
     const int batches = (last - first + A.batch - 1) / A.batch;
     for (int b = 0; b < batches; ++b) {
         const int t0 = first + b * A.batch, n = min(A.batch, last - t0);
+        float2 next = make_float2(1.0f, 1.0f);
         if (b + 1 < batches) {
-            issue(t0 + A.batch, min(A.batch, last - t0 - A.batch), (b + 1) & 1);
+            const int n1 = min(A.batch, last - t0 - A.batch);
+            issue(t0 + A.batch, n1, (b + 1) & 1);
+            if (warp == 0) next = read_facts(t0 + A.batch, n1);
             asm volatile("cp.async.wait_group 1;\n" ::);
         } else {
             asm volatile("cp.async.wait_group 0;\n" ::);
         }
         __syncthreads();
         const float* token = stage + (b & 1) * stage_floats;
-        for (int j = 0; j < n; ++j, token += token_floats) {
-            float keep = fixed, take = 1.0f;
-            if (A.coef) keep = token[2 * VECTOR + A.cols], take = token[2 * VECTOR + A.cols + 1];
-            P *= keep;
-            if (MODE == SCAN_LOCAL) product *= keep;
-            if (P < SCAN_LEAST) {                            // the same for every thread of the block
-#pragma unroll
-                for (int i = 0; i < SCAN_ROWS; ++i) {
-                    s[i].x *= P, s[i].y *= P, s[i].z *= P, s[i].w *= P;
-                    norm[i] *= P;
-                }
-                P = 1.0f;
+        const float4* fact = facts[b & 1];
+        const float end = fact[n - 1].y;                     // the batch's product of keeps, the same for every thread
+        if (MODE == SCAN_LOCAL) product *= end;
+        if (P * end < SCAN_LEAST) {
+            rescale(P);
+            P = 1.0f;
+        }
+        if (idle) {
+        } else if (end < SCAN_LEAST) {
+#pragma unroll 1
+            for (int j = 0; j < n; ++j, token += token_floats) {
+                rescale(fact[j].z);
+                walk(token, fact[j].w, 1.0f);
+                to += out_step;
             }
-            const float weight = take / P;
-            const float4 vv = *reinterpret_cast<const float4*>(token + 2 * VECTOR + place);
-            const float4 tv = make_float4(vv.x * weight, vv.y * weight, vv.z * weight, vv.w * weight);
-            float4 y = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-            const float* kp = token + part * SCAN_PITCH;
-#pragma unroll
-            for (int i4 = 0; i4 < SCAN_ROWS; i4 += 4) {
-                const float4 k4 = *reinterpret_cast<const float4*>(kp + i4);
-                const float kk[4] = {k4.x, k4.y, k4.z, k4.w};
-                float qq[4] = {0.0f, 0.0f, 0.0f, 0.0f};
-                if (MODE != SCAN_LOCAL) {
-                    const float4 q4 = *reinterpret_cast<const float4*>(kp + VECTOR + i4);
-                    qq[0] = q4.x, qq[1] = q4.y, qq[2] = q4.z, qq[3] = q4.w;
-                }
-#pragma unroll
-                for (int i = 0; i < 4; ++i) {
-                    float4& r = s[i4 + i];
-                    r.x = fmaf(kk[i], tv.x, r.x), r.y = fmaf(kk[i], tv.y, r.y), r.z = fmaf(kk[i], tv.z, r.z), r.w = fmaf(kk[i], tv.w, r.w);
-                    if (MODE != SCAN_LOCAL)
-                        y.x = fmaf(r.x, qq[i], y.x), y.y = fmaf(r.y, qq[i], y.y), y.z = fmaf(r.z, qq[i], y.z), y.w = fmaf(r.w, qq[i], y.w);
-                }
-            }
-            if (owns_norm) {                                 // n takes k alone: a column whose value is always 1
-                float c = 0.0f;
-#pragma unroll
-                for (int i = 0; i < SCAN_ROWS; ++i) {
-                    norm[i] = fmaf(kp[i], weight, norm[i]);
-                    if (MODE != SCAN_LOCAL) c = fmaf(norm[i], kp[VECTOR + i], c);
-                }
-                if (MODE != SCAN_LOCAL) {
-#pragma unroll
-                    for (int o = GROUPS; o < 32; o <<= 1) c += __shfl_xor_sync(0xffffffffu, c, o);
-                    if (lane == 0) A.norm_out[(size_t)(t0 + j) * A.heads + head] = c * P;
-                }
-            }
-            if (MODE == SCAN_LOCAL) continue;
-            float* to = A.out + (size_t)(t0 + j) * A.heads * A.e + (size_t)head * A.e + col;
-            if (PARTS == 1) {
-                if (A.vec_out) {
-                    if (col < A.e) *reinterpret_cast<float4*>(to) = make_float4(y.x * P, y.y * P, y.z * P, y.w * P);
-                } else {
-                    if (col < A.e) to[0] = y.x * P;
-                    if (col + 1 < A.e) to[1] = y.y * P;
-                    if (col + 2 < A.e) to[2] = y.z * P;
-                    if (col + 3 < A.e) to[3] = y.w * P;
-                }
-            } else {
-                const bool upper = part & 1;                 // this lane goes on with the upper two of the four columns
-                float y0 = upper ? y.z : y.x, y1 = upper ? y.w : y.y;
-                y0 += __shfl_xor_sync(0xffffffffu, upper ? y.x : y.z, GROUPS);
-                y1 += __shfl_xor_sync(0xffffffffu, upper ? y.y : y.w, GROUPS);
-                if (PARTS == 2) {
-                    const int at = upper ? 2 : 0;
-                    if (col + at < A.e) to[at] = y0 * P;
-                    if (col + at + 1 < A.e) to[at + 1] = y1 * P;
-                } else {
-                    const bool second = part & 2;
-                    float z = second ? y1 : y0;
-                    z += __shfl_xor_sync(0xffffffffu, second ? y0 : y1, 2 * GROUPS);
-#pragma unroll
-                    for (int o = 4 * GROUPS; o < 32; o <<= 1) z += __shfl_xor_sync(0xffffffffu, z, o);
-                    const int at = (upper ? 2 : 0) + (second ? 1 : 0);
-                    if (part < 4 && col + at < A.e) to[at] = z * P;
-                }
+        } else {
+            const float inverse = 1.0f / P;
+#pragma unroll 1
+            for (int j = 0; j < n; ++j, token += token_floats) {
+                const float2 f = *reinterpret_cast<const float2*>(&fact[j]);
+                walk(token, f.x * inverse, f.y * P);
+                to += out_step;
             }
         }
+        if (end >= SCAN_LEAST) P *= end;
+        if (warp == 0 && b + 1 < batches) write_facts(next, (b + 1) & 1);
         __syncthreads();                                     // the stage is copied into again two batches on
     }
     if (MODE == SCAN_LOCAL && threadIdx.x == 0 && slice == 0) A.chunk_decay[chunk_at] = product;
     if (MODE == SCAN_LOCAL || (MODE == SCAN_WHOLE && A.write_state)) {
+        rescale(P);
 #pragma unroll
-        for (int i = 0; i < SCAN_ROWS; ++i) {
-            if (row0 + i >= A.d) continue;
-            float* to = mine + (size_t)(row0 + i) * A.e + col;
-            if (A.vec_state) {
-                if (col < A.e) *reinterpret_cast<float4*>(to) = make_float4(s[i].x * P, s[i].y * P, s[i].z * P, s[i].w * P);
-            } else {
-                if (col < A.e) to[0] = s[i].x * P;
-                if (col + 1 < A.e) to[1] = s[i].y * P;
-                if (col + 2 < A.e) to[2] = s[i].z * P;
-                if (col + 3 < A.e) to[3] = s[i].w * P;
+        for (int i = 0; i < PAIRS; ++i) {
+            const float2 x[4] = {split(s[0][i]), split(s[1][i]), split(s[2][i]), split(s[3][i])};
+#pragma unroll
+            for (int u = 0; u < 2; ++u) {
+                const int row = row0 + 2 * i + u;
+                if (row >= A.d) continue;
+                const float4 f = u ? make_float4(x[0].y, x[1].y, x[2].y, x[3].y) : make_float4(x[0].x, x[1].x, x[2].x, x[3].x);
+                float* to = mine + (size_t)row * A.e + col;
+                if (A.vec_state) {
+                    if (col < A.e) *reinterpret_cast<float4*>(to) = f;
+                } else {
+                    if (col < A.e) to[0] = f.x;
+                    if (col + 1 < A.e) to[1] = f.y;
+                    if (col + 2 < A.e) to[2] = f.z;
+                    if (col + 3 < A.e) to[3] = f.w;
+                }
+                if (is_norm) norm_mine[row] = f.x;
             }
-            if (owns_norm && lane % GROUPS == 0) norm_mine[row0 + i] = norm[i] * P;
         }
     }
 }
 
-// One thread an element of a (sequence, head)'s S (and n behind it): chunk c's entry goes from the chunk's end state from zero
-// to the state at its start, in[0] = the slot's state (zero at position 0), in[c + 1] = product_c in[c] + end_c.
+// A thread takes one element (VEC: four neighbouring ones) of a (sequence, head)'s S (and n behind it): chunk c's entry goes from
+// the chunk's end state from zero to the state at its start, in[0] = the slot's state (zero at position 0), in[c + 1] =
+// product_c in[c] + end_c.  The end states of eight chunks are asked for together.
+template <bool VEC>
 __global__ void scan_chunk_states_kernel(const ScanArgs A, int elements) {
     pdl_launch_dependents();
     pdl_wait();
+    constexpr int W = VEC ? 4 : 1, AHEAD = 8;
     const int seq = blockIdx.x, head = blockIdx.y;
     const int first = A.q_start[seq], rows = A.q_start[seq + 1] - first;
     const int slot = A.state_slots[seq];
     if (slot < 0 || rows <= 0) return;
+    const int i = (blockIdx.z * blockDim.x + threadIdx.x) * W;
+    if (i >= elements) return;
     const int chunks = (rows + A.chunk_len - 1) / A.chunk_len, matrix = A.d * A.e;
     const bool fresh = A.positions[first] == 0;
-    float* local = A.chunk_state + ((size_t)seq * A.heads + head) * A.max_chunks * A.chunk_floats;
+    float* local = A.chunk_state + ((size_t)seq * A.heads + head) * A.max_chunks * A.chunk_floats + i;
     const float* product = A.chunk_decay + ((size_t)seq * A.heads + head) * A.max_chunks;
-    for (int i = blockIdx.z * blockDim.x + threadIdx.x; i < elements; i += gridDim.z * blockDim.x) {
-        float* slot_at = (i < matrix ? A.state + (size_t)head * matrix + i : A.norm_state + (size_t)head * A.d + (i - matrix)) +
-                         (long long)slot * A.state_stride;
-        float value = fresh ? 0.0f : *slot_at;
-        for (int c = 0; c < chunks; ++c) {
-            const float end = local[(size_t)c * A.chunk_floats + i];
-            local[(size_t)c * A.chunk_floats + i] = value;
-            value = product[c] * value + end;
+    float* slot_at = (i < matrix ? A.state + (size_t)head * matrix + i : A.norm_state + (size_t)head * A.d + (i - matrix)) +
+                     (long long)slot * A.state_stride;
+    float value[W];
+#pragma unroll
+    for (int u = 0; u < W; ++u) value[u] = fresh ? 0.0f : slot_at[u];
+    for (int c0 = 0; c0 < chunks; c0 += AHEAD) {
+        float end[AHEAD][W], keep[AHEAD];
+#pragma unroll
+        for (int c = 0; c < AHEAD; ++c) {
+            if (c0 + c >= chunks) continue;
+            const float* from = local + (size_t)(c0 + c) * A.chunk_floats;
+            keep[c] = product[c0 + c];
+            if (VEC) {
+                const float4 f = *reinterpret_cast<const float4*>(from);
+                end[c][0] = f.x;
+                if (VEC) end[c][W > 1 ? 1 : 0] = f.y, end[c][W > 2 ? 2 : 0] = f.z, end[c][W > 3 ? 3 : 0] = f.w;
+            } else {
+                end[c][0] = from[0];
+            }
         }
-        if (A.write_state) *slot_at = value;
+#pragma unroll
+        for (int c = 0; c < AHEAD; ++c) {
+            if (c0 + c >= chunks) continue;
+            float* to = local + (size_t)(c0 + c) * A.chunk_floats;
+            if (VEC) *reinterpret_cast<float4*>(to) = make_float4(value[0], value[W > 1 ? 1 : 0], value[W > 2 ? 2 : 0], value[W > 3 ? 3 : 0]);
+            else to[0] = value[0];
+#pragma unroll
+            for (int u = 0; u < W; ++u) value[u] = fmaf(keep[c], value[u], end[c][u]);
+        }
     }
+    if (!A.write_state) return;
+#pragma unroll
+    for (int u = 0; u < W; ++u) slot_at[u] = value[u];
 }
 
 }  // namespace
@@ -427,7 +504,7 @@ MRS_EXPORT int mrs_memory_gates(const float* raw, int raw_stride, int i_offset, 
 }
 
 // How the recurrence is cut: lanes that share a column group, columns a block, slices of the columns.  Returns the slices.
-static int scan_shape(int d, int e, int* parts_out, int* cols_out) {
+static int scan_shape(int d, int e, bool normaliser, int* parts_out, int* cols_out) {
     int parts = 1;
     while (parts * SCAN_ROWS < d) parts <<= 1;
     const int per_warp = 4 * (32 / parts);
@@ -435,13 +512,14 @@ static int scan_shape(int d, int e, int* parts_out, int* cols_out) {
     if (warps > 8) warps = 8;
     *parts_out = parts;
     *cols_out = warps * per_warp;
-    return (e + *cols_out - 1) / *cols_out;
+    const int columns = normaliser ? (e + 3) / 4 * 4 + 4 : e;
+    return (columns + *cols_out - 1) / *cols_out;
 }
 
-MRS_EXPORT int mrs_linear_scan_slices(int d, int e) {
+MRS_EXPORT int mrs_linear_scan_slices(int d, int e, int normaliser) {
     int parts, cols;
     if (d <= 0 || d > 512 || e <= 0) return 0;
-    return scan_shape(d, e, &parts, &cols);
+    return scan_shape(d, e, normaliser != 0, &parts, &cols);
 }
 
 // Floats of scratch that a run in chunks needs.
@@ -462,7 +540,7 @@ MRS_EXPORT int mrs_linear_scan(const float* q, const float* k, const float* v, i
         return MRS_BAD_ARGUMENT;
     ScanArgs A = {};
     int parts, cols;
-    const int slices = scan_shape(d, e, &parts, &cols);
+    const int slices = scan_shape(d, e, norm_state != nullptr, &parts, &cols);
     if ((long long)heads * slices > 65535) return MRS_BAD_ARGUMENT;
     A.q = q, A.k = k, A.v = v, A.stride = stride, A.decay = decay, A.coef = decay ? nullptr : coef, A.coef_stride = coef_stride;
     A.state = state, A.norm_state = norm_state, A.state_stride = state_stride;
@@ -471,10 +549,10 @@ MRS_EXPORT int mrs_linear_scan(const float* q, const float* k, const float* v, i
     A.vec_qk = d % 4 == 0 && stride % 4 == 0 && (((uintptr_t)q | (uintptr_t)k) & 15) == 0;
     A.vec_v = e % 4 == 0 && stride % 4 == 0 && ((uintptr_t)v & 15) == 0;
     A.vec_out = e % 4 == 0 && ((uintptr_t)out & 15) == 0;
-    const int token_floats = 2 * parts * SCAN_PITCH + cols + 4;
+    const int token_floats = 2 * parts * SCAN_PITCH + cols;
     int batch = (40 * 1024) / (2 * token_floats * (int)sizeof(float));
-    if (batch > 8) batch = 8;
-    if (tokens < 8 * sequences && batch > (tokens + sequences - 1) / sequences) batch = (tokens + sequences - 1) / sequences;
+    if (batch > SCAN_BATCH) batch = SCAN_BATCH;
+    if (tokens < SCAN_BATCH * sequences && batch > (tokens + sequences - 1) / sequences) batch = (tokens + sequences - 1) / sequences;
     if (batch < 1) return MRS_BAD_ARGUMENT;
     A.batch = batch;
     const int threads = cols / (4 * (32 / parts)) * 32;
@@ -502,9 +580,10 @@ MRS_EXPORT int mrs_linear_scan(const float* q, const float* k, const float* v, i
     A.chunk_decay = scratch + (size_t)sequences * heads * A.max_chunks * A.chunk_floats;
     A.vec_state = e % 4 == 0;
     SCAN_LAUNCH(SCAN_LOCAL, dim3(sequences, heads * slices, A.max_chunks));
-    int across = (elements + 255) / 256;
-    if (across > 64) across = 64;
-    MRS_LAUNCH(scan_chunk_states_kernel, dim3(sequences, heads, across), 256, 0, s, A, elements);
+    if (d * e % 4 == 0 && elements % 4 == 0 && A.vec_state)
+        MRS_LAUNCH(scan_chunk_states_kernel<true>, dim3(sequences, heads, (elements / 4 + 127) / 128), 128, 0, s, A, elements);
+    else
+        MRS_LAUNCH(scan_chunk_states_kernel<false>, dim3(sequences, heads, (elements + 127) / 128), 128, 0, s, A, elements);
     SCAN_LAUNCH(SCAN_FINAL, dim3(sequences, heads * slices, A.max_chunks));
 #undef SCAN_LAUNCH
     MRS_RETURN_LAUNCH_STATUS();

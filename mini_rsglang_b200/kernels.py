@@ -2102,7 +2102,7 @@ _LINEAR_SCAN_SIGNATURES = {
     "mrs_narrow_columns": [_c_int, _c_vp, _c_int, _c_int, _c_vp, _c_int, _c_int, _c_int, _c_vp],
     "mrs_memory_gates": [_c_vp, _c_int, _c_int, _c_int, _c_vp, _c_vp, _c_float, _c_vp, _c_ll, _c_vp, _c_vp, _c_vp, _c_vp, _c_int, _c_int,
                          _c_int, _c_int, _c_vp],
-    "mrs_linear_scan_slices": [_c_int, _c_int],
+    "mrs_linear_scan_slices": [_c_int, _c_int, _c_int],
     "mrs_linear_scan": [_c_vp, _c_vp, _c_vp, _c_int, _c_vp, _c_vp, _c_int, _c_vp, _c_vp, _c_ll, _c_vp, _c_vp, _c_vp, _c_vp, _c_vp, _c_int,
                         _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_vp, _c_vp],
 }
@@ -2211,14 +2211,14 @@ def linear_scan(rows: torch.Tensor, q_offset: int, k_offset: int, v_offset: int,
         raise InvalidRequest("linear_scan: a normaliser has a state and an output")
     if norm_state is not None:
         if norm_state.dtype != torch.float32 or tuple(norm_state.shape[1:]) != (heads, d) or norm_state.stride(2) != 1 or \
-                norm_state.stride(1) != d or norm_state.stride(0) != state.stride(0):
+                norm_state.stride(1) != d or norm_state.shape[0] != state.shape[0] or (state.shape[0] > 1 and norm_state.stride(0) != state.stride(0)):
             raise InvalidRequest("linear_scan: the normaliser's state must be float32 [slots, heads, d], dense within a slot, in the same slots")
         _need(norm_out, torch.float32, "normaliser", (tokens, heads))
     _need(out, torch.float32, "recurrence output", (tokens, heads * e))
     sequences = state_slots.shape[0]
     lib = linear_scan_library()
     if chunk_len is None:
-        chunk_len = linear_scan_chunk_length(tokens, sequences, heads, d, e, lib.mrs_linear_scan_slices(d, e), sm_count(rows.device))
+        chunk_len = linear_scan_chunk_length(tokens, sequences, heads, d, e, lib.mrs_linear_scan_slices(d, e, int(norm_state is not None)), sm_count(rows.device))
     scratch = None
     if chunk_len:
         need = lib.mrs_linear_scan_scratch_floats(tokens, sequences, heads, d, e, int(norm_state is not None), int(chunk_len))
