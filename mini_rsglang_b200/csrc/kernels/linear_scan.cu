@@ -10,7 +10,7 @@
 //   rotate_heads       q and k heads inside the float32 projection turn by their token's position, in place
 //   memory_gates       keep, take and exp(-m) of every (token, head) from the raw gates of an exponential memory with a running
 //                      maximum m (which starts at 0)
-//   linear_scan        the recurrence
+//   linear_scan        the recurrence (linear_step: the same for decoded tokens)
 //   narrow_columns     a range of float32 columns as rows of the engine's dtype
 #include "common.cuh"
 #include "pairs.cuh"
@@ -408,6 +408,107 @@ __global__ void __launch_bounds__(256, 2) linear_scan_kernel(const ScanArgs A) {
     }
 }
 
+// The recurrence for decoded tokens (a token or a few a sequence), where S is read and written once and that is the time: a warp
+// takes SCAN_ROWS rows of up to 128 neighbouring columns, four a lane, so that every access is a whole row of them and all of a
+// thread's loads are in flight together; the warps' parts of a token's read-out meet in shared memory.  Nothing is staged: k
+// and q are the same for a warp's lanes.  At most 16 warps (d up to 256).
+#define STEP_COLUMNS 128
+__global__ void __launch_bounds__(512) linear_step_kernel(const ScanArgs A) {
+    __shared__ __align__(16) float parts[2][16][STEP_COLUMNS];
+    pdl_launch_dependents();
+    pdl_wait();
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
+    const int seq = blockIdx.x, head = blockIdx.y;
+    const int first = A.q_start[seq], last = A.q_start[seq + 1];
+    const int slot = A.state_slots[seq];
+    if (slot < 0 || last <= first) return;
+    const int col = blockIdx.z * STEP_COLUMNS + 4 * lane, row0 = warp * SCAN_ROWS;
+    const int norm_col = A.norm_state ? (A.e + 3) / 4 * 4 : -4;
+    const bool is_norm = col == norm_col;
+    const int live = is_norm ? 1 : min(A.e - col, 4);        // columns of these four that are there
+    float* mine = A.state + (long long)slot * A.state_stride + (size_t)head * A.d * A.e + col;
+    int step = A.e;                                          // from row to row
+    if (is_norm) mine = A.norm_state + (long long)slot * A.state_stride + (size_t)head * A.d, step = 1;
+    const bool whole = A.vec_state && !is_norm && live == 4;
+    const bool zero = A.positions[first] == 0;
+    float4 s[SCAN_ROWS];
+#pragma unroll
+    for (int i = 0; i < SCAN_ROWS; ++i) {
+        s[i] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        const float* from = mine + (size_t)(row0 + i) * step;
+        if (zero || row0 + i >= A.d) continue;
+        if (whole) {
+            s[i] = *reinterpret_cast<const float4*>(from);
+        } else {
+            if (live > 0) s[i].x = from[0];
+            if (live > 1) s[i].y = from[1];
+            if (live > 2) s[i].z = from[2];
+            if (live > 3) s[i].w = from[3];
+        }
+    }
+    for (int t = first; t < last; ++t) {
+        const size_t row = (size_t)t * A.stride;
+        const float *k = A.k + row + head * A.d + row0, *q = A.q + row + head * A.d + row0, *v = A.v + row + head * A.e + col;
+        float keep = 1.0f, take = 1.0f;
+        if (A.decay) keep = A.decay[head];
+        else keep = A.coef[(size_t)t * A.coef_stride + head], take = A.coef[(size_t)t * A.coef_stride + A.heads + head];
+        float4 tv = make_float4(0.0f, 0.0f, 0.0f, 0.0f), y = tv;
+        if (is_norm) {
+            tv.x = take;                                     // n takes k alone: a column whose value is always 1
+        } else {
+            if (live > 0) tv.x = take * v[0];
+            if (live > 1) tv.y = take * v[1];
+            if (live > 2) tv.z = take * v[2];
+            if (live > 3) tv.w = take * v[3];
+        }
+#pragma unroll
+        for (int i = 0; i < SCAN_ROWS; i += 4) {
+            float4 k4 = make_float4(0.0f, 0.0f, 0.0f, 0.0f), q4 = k4;
+            if (A.vec_qk) {
+                if (row0 + i < A.d) k4 = *reinterpret_cast<const float4*>(k + i), q4 = *reinterpret_cast<const float4*>(q + i);
+            } else {
+                if (row0 + i < A.d) k4.x = k[i], q4.x = q[i];
+                if (row0 + i + 1 < A.d) k4.y = k[i + 1], q4.y = q[i + 1];
+                if (row0 + i + 2 < A.d) k4.z = k[i + 2], q4.z = q[i + 2];
+                if (row0 + i + 3 < A.d) k4.w = k[i + 3], q4.w = q[i + 3];
+            }
+            const float kk[4] = {k4.x, k4.y, k4.z, k4.w}, qq[4] = {q4.x, q4.y, q4.z, q4.w};
+#pragma unroll
+            for (int u = 0; u < 4; ++u) {
+                float4& r = s[i + u];
+                r.x = fmaf(keep, r.x, kk[u] * tv.x), r.y = fmaf(keep, r.y, kk[u] * tv.y);
+                r.z = fmaf(keep, r.z, kk[u] * tv.z), r.w = fmaf(keep, r.w, kk[u] * tv.w);
+                y.x = fmaf(r.x, qq[u], y.x), y.y = fmaf(r.y, qq[u], y.y), y.z = fmaf(r.z, qq[u], y.z), y.w = fmaf(r.w, qq[u], y.w);
+            }
+        }
+        float (*met)[STEP_COLUMNS] = parts[(t - first) & 1];     // two in turn: one barrier a token is enough
+        *reinterpret_cast<float4*>(&met[warp][4 * lane]) = y;
+        __syncthreads();
+        for (int c = threadIdx.x; c < STEP_COLUMNS; c += blockDim.x) {
+            const int at = blockIdx.z * STEP_COLUMNS + c;
+            if (at >= A.e && at != norm_col) continue;
+            float sum = 0.0f;
+            for (int w = 0; w < warps; ++w) sum += met[w][c];
+            if (at == norm_col) A.norm_out[(size_t)t * A.heads + head] = sum;
+            else A.out[(size_t)t * A.heads * A.e + (size_t)head * A.e + at] = sum;
+        }
+    }
+    if (!A.write_state) return;
+#pragma unroll
+    for (int i = 0; i < SCAN_ROWS; ++i) {
+        float* to = mine + (size_t)(row0 + i) * step;
+        if (row0 + i >= A.d) continue;
+        if (whole) {
+            *reinterpret_cast<float4*>(to) = s[i];
+        } else {
+            if (live > 0) to[0] = s[i].x;
+            if (live > 1) to[1] = s[i].y;
+            if (live > 2) to[2] = s[i].z;
+            if (live > 3) to[3] = s[i].w;
+        }
+    }
+}
+
 // A thread takes one element (VEC: four neighbouring ones) of a (sequence, head)'s S (and n behind it): chunk c's entry goes from
 // the chunk's end state from zero to the state at its start, in[0] = the slot's state (zero at position 0), in[c + 1] =
 // product_c in[c] + end_c.  The end states of eight chunks are asked for together.
@@ -568,6 +669,12 @@ MRS_EXPORT int mrs_linear_scan(const float* q, const float* k, const float* v, i
     }
     if (chunk_len == 0) {
         A.vec_state = e % 4 == 0 && state_stride % 4 == 0 && ((uintptr_t)state & 15) == 0;
+        if (d <= 256 && tokens < 4LL * sequences) {
+            const int columns = norm_state ? (e + 3) / 4 * 4 + 4 : e;
+            MRS_LAUNCH(linear_step_kernel, dim3(sequences, heads, (columns + STEP_COLUMNS - 1) / STEP_COLUMNS),
+                       (d + SCAN_ROWS - 1) / SCAN_ROWS * 32, 0, s, A);
+            MRS_RETURN_LAUNCH_STATUS();
+        }
         SCAN_LAUNCH(SCAN_WHOLE, dim3(sequences, heads * slices));
         MRS_RETURN_LAUNCH_STATUS();
     }
