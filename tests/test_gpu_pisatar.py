@@ -173,7 +173,7 @@ def test_a_prompt_of_more_rows_than_a_recorded_step_holds(tmp_path_factory):
     recurrences in many chunks; then decoded tokens from the states that it left."""
     raw = {"architecture": "Pisatar", "vocab": 97, "width": 64, "norm": {"eps": 1e-5}, "layers": [
         dict(retention(2, 16, 32, [0.99, 0.9995]), mlp=dense(64)),
-        dict(both((2, 1, 16, 16), (2, 16, 16), 10.0, (0.7, 0.9), dims=8, scaling=(4.0, 1.0, 4.0, 512)), mlp=dense(96)),
+        dict(both((2, 1, 16, 16), (2, 16, 16), 10.0, (0.7, 0.9), dims=8, scaling=(5.0, 1.0, 3.0, 300)), mlp=dense(96)),
         dict(channel_delta(2, 1, 16, 16, 2, 8, 4), mlp=dense(32))]}
     folder = write_model(str(tmp_path_factory.mktemp("pisatar_long")), raw, 61)
     config, weights = load_plain(folder)
