@@ -534,6 +534,79 @@ def test_a_channel_decay_acts_on_its_own_row():
     assert (S[0] == 5.0).all()
 
 
+def one_sequence(at, m, table, slots):
+    """The context of a step that brings the tokens at .. at + m - 1 of one sequence."""
+    from mini_rsglang_b200.engine.context import StepContext
+    from mini_rsglang_b200.parts.base import StepFacts
+
+    zeros = torch.zeros(m, dtype=torch.int32, device=DEV)
+    return StepContext(num_tokens=m, num_sequences=1, token_ids=None, positions=torch.arange(at, at + m, dtype=torch.int32, device=DEV),
+                       seq_of_token=zeros, q_start=torch.tensor([0, m], dtype=torch.int32, device=DEV),
+                       context_len=torch.tensor([at + m], dtype=torch.int32, device=DEV), state_slots=zeros[:1].clone(), want_rows=None,
+                       block_tables=[table.view(1, -1).to(DEV)], slots=[slots.to(torch.int32).to(DEV)], host_q_start=[0, m], host_start_pos=[at],
+                       max_query_len=m, max_context_len=at + m, facts=StepFacts([0, m], [at], at + m))
+
+
+@pytest.mark.parametrize("gated", [False, True])
+def test_a_sum_of_mixers_is_the_mixers_each_alone(gated):
+    """Terms and sum, with one projection for both mixers and (an attention whose gates are columns of its own) without."""
+    from mini_rsglang_b200.cache.storage import CacheEntry
+    from mini_rsglang_b200.parts.base import MIXERS, PartSpec, Runtime
+    from mini_rsglang_b200.weights import random_weights
+
+    width, n, page = 24, 21, 4
+    attention = PartSpec("biased_window_attention", {"width": width, "num_heads": 2, "num_kv_heads": 1, "head_dim": 10, "value_dim": 6,
+                                                     "position": PartSpec("rope", {"head_dim": 10, "theta": 100.0}),
+                                                     "output_gate": "elements" if gated else False})
+    memory = PartSpec("matrix_memory", {"width": width, "heads": 3, "head_dim": 6, "value_dim": 10, "gate_cap": 5.0, "eps": 1e-5})
+    both_of = MIXERS.build(PartSpec("mixer_sum", {"width": width, "branches": [("x", attention, 0.7), ("y", memory, -2.0)]}), "m")
+    alone = [MIXERS.build(attention, "m.x"), MIXERS.build(memory, "m.y")]
+    tensors = random_weights(both_of.weight_specs(), 3, torch.float32, DEV)
+    tensors = {name: t * 10.0 for name, t in tensors.items()}
+    for part in (both_of, *alone):
+        part.bind(tensors, Runtime(torch.device(DEV), torch.float32, page))
+    assert (both_of.fused is None) == gated
+
+    def cache():
+        return CacheEntry(group=0, k=torch.zeros(6, 1, page, 10, device=DEV), v=torch.zeros(6, 1, page, 6, device=DEV),
+                          state=torch.full((2, *both_of.state_need().shape), 3.0, device=DEV))
+
+    torch.manual_seed(1)
+    h = torch.randn(n, width, device=DEV)
+    table = torch.randperm(6).to(torch.int32)
+    caches = [cache() for _ in range(3)]
+    for at, m in ((0, 15), (15, 1), (16, 5)):
+        places = torch.arange(at, at + m)
+        ctx = one_sequence(at, m, table, table.long()[places // page] * page + places % page)
+        x = h[at:at + m].contiguous()
+        want = 0.7 * alone[0].forward(x, ctx, caches[0]).double() - 2.0 * alone[1].forward(x, ctx, caches[0]).double()
+        got = both_of.forward(x, ctx, caches[1])
+        terms = both_of.forward(x, ctx, caches[2], as_terms=True).terms
+        scale = want.abs().max()
+        assert scale > 1e-3 and (got.double() - want).abs().max() < 1e-5 * scale
+        assert (sum(f * t.double() for t, f in terms) - want).abs().max() < 1e-5 * scale
+
+
+def test_the_stream_after_every_layer(folders, tmp_path_factory):
+    """`bin/trace_run --observe`: the float32 residual stream after the embedding and after every layer run against the plain
+    implementation, in a prompt's portion and in decoded tokens."""
+    import numpy as np
+
+    config, weights = load_plain(folders["X"])
+    tokens = T.requests_for(config["vocab"], [19], seed=77)["r0"]
+    layers = []
+    P.forward(config, weights, tokens, layers_out=layers)
+    out = str(tmp_path_factory.mktemp("observed"))
+    run = T.TraceRun(folders["X"], "float32", out, 64, extra=("--page-size", "4", "--observe", "a"))
+    for step, (at, m) in enumerate(((0, 16), (16, 1), (17, 2))):
+        run.step({"step": step, "entries": [{"id": "a", "tokens": tokens[at:at + m], "want": []}], "end": []}, config["vocab"])
+        for i, stream in enumerate(layers):
+            got = np.fromfile(os.path.join(out, "observe", f"{step}.layer{i}-output.f32"), dtype="<f4").reshape(m, config["width"])
+            want = stream[at:at + m]
+            assert (torch.from_numpy(got).double() - want).abs().max() < 2e-5 * max(1.0, want.abs().max().item()), (step, i)
+    assert run.close() == 0
+
+
 @pytest.mark.parametrize("H,G,d,e,page", [(6, 2, 20, 12, 4), (4, 2, 64, 64, 16), (8, 1, 32, 48, 16), (8, 1, 64, 128, 16), (2, 1, 128, 128, 16)])
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 def test_attention_reads_far_keys_and_page_borders(tmp_path_factory, H, G, d, e, page, dtype):
@@ -541,10 +614,8 @@ def test_attention_reads_far_keys_and_page_borders(tmp_path_factory, H, G, d, e,
     places (the first tokens, both sides of page borders, far back, the last one) is the only key that answers the queries, whose
     output is then that place's value."""
     from mini_rsglang_b200 import kernels
-    from mini_rsglang_b200.parts.attention import StepFacts
-    from mini_rsglang_b200.parts.base import MIXERS, PartSpec, Runtime
     from mini_rsglang_b200.cache.storage import CacheEntry
-    from mini_rsglang_b200.engine.context import StepContext
+    from mini_rsglang_b200.parts.base import MIXERS, PartSpec, Runtime
 
     torch_dtype = getattr(torch, dtype)
     width, n = 16, 333
@@ -574,12 +645,7 @@ def test_attention_reads_far_keys_and_page_borders(tmp_path_factory, H, G, d, e,
         for m in cuts:
             positions = torch.arange(at, at + m, dtype=torch.int32)
             slots = table.long()[positions.long() // page] * page + positions % page
-            ctx = StepContext(num_tokens=m, num_sequences=1, token_ids=None, positions=positions.to(DEV),
-                              seq_of_token=torch.zeros(m, dtype=torch.int32, device=DEV), q_start=torch.tensor([0, m], dtype=torch.int32, device=DEV),
-                              context_len=torch.tensor([at + m], dtype=torch.int32, device=DEV), state_slots=torch.zeros(1, dtype=torch.int32, device=DEV),
-                              want_rows=None, block_tables=[table.view(1, -1).to(DEV)], slots=[slots.to(torch.int32).to(DEV)],
-                              host_q_start=[0, m], host_start_pos=[at], max_query_len=m, max_context_len=at + m,
-                              facts=StepFacts([0, m], [at], at + m))
+            ctx = one_sequence(at, m, table, slots)
             out = part.forward_projected(proj[at:at + m].to(DEV).contiguous(), 0, ctx, cache).cpu()
             kernels.check_device_errors()
             first = max(place - at, 0)
