@@ -914,3 +914,158 @@ class PisatarConfig(ModelConfig):
         if self.eos_token_id is not None:
             out["eos_token_id"] = self.eos_token_id
         return out
+
+
+@dataclass
+class BilipelConfig(ModelConfig):
+    """Bilipel: a decoder of pre-norm layers (layer norms with bias) whose branches join the stream times a constant.  The mixer is
+    a gated linear attention (a matrix state a head that forgets by one decay a key channel and token), an attention (one norm over
+    all query heads and one over all key heads, partly rotated heads with stretched rotary positions, a learned sink a head) or a
+    latent attention (part of every head rotated in interleaved pairs, a sliding window, a learned sink a head); the feed-forward a
+    gated unit or routed experts whose router has a bias.  A run of layers may be passed several times with the same weights, every
+    pass with caches and states of its own: a vector of the pass, and from the second pass on the embedding, is added to the
+    stream before it.  config.json names the design under `architecture`; its keys are read as they stand there:
+
+      vocab, width, norm.eps, residual_mult, loop.{start, stop, times}
+      layers[i].type = "gla":              mixer.{heads, dim, vdim, tau}
+      layers[i].type = "attention":        mixer.{heads, kv_heads, dim, vdim, scale, rot.{base, dims, scaling.{factor, original, fast, slow}}}
+      layers[i].type = "latent_attention": mixer.{heads, dim, rot_dim, vdim, kv_rank, scale, mask.size, rot.{base, dims}}
+      layers[i].mlp = null | {kind: "dense", ff} | {kind: "moe", expert.ff, router.{experts, top}}
+
+    `residual_mult` (1), `loop`, `rot.scaling` (plain rotary positions), a latent attention's `mask` (every earlier key) and `mlp` may
+    be absent.  The inner size of a gla's thin products stands in the checkpoint; `mixer.decay_rank` gives it for a model that is
+    drawn at random.  The design states no longest context and no end-of-sequence token; `max_position_embeddings` and
+    `eos_token_id` are read if a file has them."""
+
+    width: int = 0
+    norm_eps: float = 0.0
+    residual_mult: float = 1.0
+    loop: dict | None = None
+    layers: list = None
+
+    MODEL_TYPES: ClassVar[tuple[str, ...]] = ("bilipel",)
+    NO_CONTEXT_LIMIT: ClassVar[int] = 1 << 22
+    MIXER_SIZES: ClassVar[dict] = {"gla": ("heads", "dim", "vdim"), "attention": ("heads", "kv_heads", "dim", "vdim"),
+                                   "latent_attention": ("heads", "dim", "rot_dim", "vdim", "kv_rank")}
+
+    @staticmethod
+    def _object(raw: dict, key: str, where: str) -> dict:
+        value = raw.get(key)
+        if not isinstance(value, dict):
+            raise InvalidRequest(f"config.json: {where}.{key} must be an object")
+        return value
+
+    @classmethod
+    def _mixer(cls, i: int, kind: str, mixer: dict) -> dict:
+        where = f"layers[{i}].mixer"
+        out = {key: _require(mixer, key, int, where) for key in cls.MIXER_SIZES[kind]}
+        if kind == "gla":
+            out["tau"] = _require(mixer, "tau", float, where)
+            if mixer.get("decay_rank") is not None:          # not a key of the design: for models without a checkpoint
+                out["decay_rank"] = _require(mixer, "decay_rank", int, "inner size of a thin product")
+            return out
+        out["scale"] = _require(mixer, "scale", float, where)
+        rot = cls._object(mixer, "rot", where)
+        out["rot"] = {"base": _require(rot, "base", float, "rotary base"), "dims": _require(rot, "dims", int, "rotated elements")}
+        if kind == "attention" and rot.get("scaling") is not None:
+            scaling = cls._object(rot, "scaling", f"{where}.rot")
+            out["rot"]["scaling"] = {key: _require(scaling, key, float, f"{where}.rot.scaling") for key in ("factor", "original", "fast", "slow")}
+        if kind == "latent_attention" and mixer.get("mask") is not None:
+            out["mask"] = {"size": _require(cls._object(mixer, "mask", where), "size", int, "window")}
+        return out
+
+    @classmethod
+    def _mlp(cls, i: int, layer: dict) -> dict | None:
+        if layer.get("mlp") is None:
+            return None
+        where = f"layers[{i}].mlp"
+        mlp = cls._object(layer, "mlp", f"layers[{i}]")
+        kind = _require(mlp, "kind", str, "feed-forward kind")
+        if kind == "dense":
+            return {"kind": kind, "ff": _require(mlp, "ff", int, "feed-forward width")}
+        if kind != "moe":
+            raise InvalidRequest(f"config.json: {where}.kind {kind!r}; known: dense, moe")
+        expert, router = cls._object(mlp, "expert", where), cls._object(mlp, "router", where)
+        return {"kind": kind, "expert": {"ff": _require(expert, "ff", int, "expert width")},
+                "router": {"experts": _require(router, "experts", int, "experts"), "top": _require(router, "top", int, "choices")}}
+
+    @classmethod
+    def from_dict(cls, raw: dict) -> "BilipelConfig":
+        norm = cls._object(raw, "norm", "config")
+        layers = raw.get("layers")
+        if not isinstance(layers, list) or not layers:
+            raise InvalidRequest("config.json: `layers` must be a list of layers")
+        read = []
+        for i, layer in enumerate(layers):
+            if not isinstance(layer, dict):
+                raise InvalidRequest(f"config.json: layers[{i}] must be an object")
+            kind = _require(layer, "type", str, f"mixer of layer {i}")
+            if kind not in cls.MIXER_SIZES:
+                raise InvalidRequest(f"config.json: layers[{i}].type {kind!r}; known: {', '.join(sorted(cls.MIXER_SIZES))}")
+            read.append({"type": kind, "mixer": cls._mixer(i, kind, cls._object(layer, "mixer", f"layers[{i}]")), "mlp": cls._mlp(i, layer)})
+        loop = raw.get("loop")
+        if loop is not None:
+            loop = {key: _require(cls._object(raw, "loop", "config"), key, int, "loop") for key in ("start", "stop", "times")}
+        cfg = cls(model_type="bilipel", architectures=["Bilipel"], vocab_size=_require(raw, "vocab", int, "vocabulary"),
+                  max_position_embeddings=int(raw.get("max_position_embeddings") or cls.NO_CONTEXT_LIMIT),
+                  eos_token_id=raw.get("eos_token_id"), width=_require(raw, "width", int, "model width"),
+                  norm_eps=_require(norm, "eps", float, "norm epsilon"),
+                  residual_mult=_require(raw, "residual_mult", float, "branch multiplier") if raw.get("residual_mult") is not None else 1.0,
+                  loop=loop, layers=read)
+        cfg.validate()
+        return cfg
+
+    def validate(self) -> None:
+        if self.vocab_size <= 0 or self.width <= 0 or self.max_position_embeddings <= 0:
+            raise InvalidRequest("invalid Bilipel dimensions: every size must be a positive integer")
+        if not math.isfinite(self.norm_eps) or self.norm_eps <= 0 or not math.isfinite(self.residual_mult):
+            raise InvalidRequest("invalid normalization parameters or branch multiplier")
+        if self.loop is not None:
+            lo, hi, times = self.loop["start"], self.loop["stop"], self.loop["times"]
+            if not 0 <= lo < hi <= len(self.layers) or times < 1:
+                raise InvalidRequest("loop: start < stop within the layers, and at least one pass")
+        for i, layer in enumerate(self.layers):
+            m, where = layer["mixer"], f"layers[{i}].mixer"
+            if any(m[key] <= 0 for key in (*self.MIXER_SIZES[layer["type"]], "decay_rank") if key in m):
+                raise InvalidRequest(f"{where}: sizes must be positive")
+            if layer["type"] == "gla":
+                if not m["tau"] > 0 or not math.isfinite(m["tau"]):
+                    raise InvalidRequest(f"{where}.tau must be positive")
+            else:
+                if not m["scale"] > 0 or not math.isfinite(m["scale"]):
+                    raise InvalidRequest(f"{where}.scale must be positive")
+                rot, most = m["rot"], m["dim"] if layer["type"] == "attention" else m["rot_dim"]
+                if rot["dims"] < 0 or rot["dims"] % 2 or rot["dims"] > most or not rot["base"] > 1:
+                    raise InvalidRequest(f"{where}.rot: an even number of elements, at most those of the part, and a base above 1")
+                if "scaling" in rot and min(rot["scaling"].values()) <= 0:
+                    raise InvalidRequest(f"{where}.rot.scaling: every number must be positive")
+            if layer["type"] == "attention" and (m["heads"] % m["kv_heads"] or max(m["dim"], m["vdim"]) > 256):
+                raise InvalidRequest(f"{where}: query heads must be a multiple of key/value heads, heads of at most 256 elements")
+            if "mask" in m and m["mask"]["size"] <= 0:
+                raise InvalidRequest(f"{where}.mask.size must be positive")
+            mlp = layer["mlp"]
+            if mlp is None:
+                continue
+            if mlp["kind"] == "dense":
+                if mlp["ff"] <= 0:
+                    raise InvalidRequest(f"layers[{i}].mlp.ff must be positive")
+            elif not 0 < mlp["router"]["top"] <= mlp["router"]["experts"] or mlp["expert"]["ff"] <= 0:
+                raise InvalidRequest(f"layers[{i}].mlp: experts and choices out of range")
+        if self.eos_token_id is not None:
+            self.eos_ids()
+
+    def eos_ids(self, folder: str | None = None) -> list[int]:
+        if self.eos_token_id is None and (folder is None or not os.path.exists(os.path.join(folder, "generation_config.json"))):
+            return []                # the design names no end-of-sequence token: generation ends by length
+        return super().eos_ids(folder)
+
+    def to_dict(self) -> dict:
+        out = {"architecture": "Bilipel", "vocab": self.vocab_size, "width": self.width, "norm": {"eps": self.norm_eps},
+               "residual_mult": self.residual_mult, "layers": self.layers}
+        if self.loop is not None:
+            out["loop"] = self.loop
+        if self.max_position_embeddings != self.NO_CONTEXT_LIMIT:
+            out["max_position_embeddings"] = self.max_position_embeddings
+        if self.eos_token_id is not None:
+            out["eos_token_id"] = self.eos_token_id
+        return out

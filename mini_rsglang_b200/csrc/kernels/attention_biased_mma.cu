@@ -76,12 +76,15 @@ struct Extras {            // what is put around the scores
     int bias_rows;
     float scale, cap;      // cap 0: none
     int window, keep_first, sink;
-    const float* sink_logits;   // [nq]: the sink's term is exp(sink_logits[head]); null: exp(0)
+    const float* sink_logits;   // [sink_heads]: the sink's term is exp(sink_logits[head]); null: exp(0)
+    int sink_heads;             // query heads of the layer: nq, or a multiple of it where a token's heads come as several rows
     int chunk;                  // > 0 (and no window): a query sees the keys of its own chunk of positions only
 };
 
-// The sink's logit of a query head, in units of log 2.
-__device__ __forceinline__ float sink_of(const Extras& x, int head) { return x.sink_logits ? x.sink_logits[head] * LOG2E : 0.0f; }
+// The sink's logit of a row's query head, in units of log 2.
+__device__ __forceinline__ float sink_of(const Extras& x, int row_token, int nq, int head) {
+    return x.sink_logits ? x.sink_logits[(row_token % (x.sink_heads / nq)) * nq + head] * LOG2E : 0.0f;
+}
 
 // Keys [key0, key0 + KV) of one kv head into a [KV][W] shared tile; rows at or beyond `key_end` or on a page that was
 // given back are zeros.
@@ -260,7 +263,7 @@ __global__ void __launch_bounds__(THREADS) attention_biased_rows_kernel(
     float row_max[2], row_sum[2];
 #pragma unroll
     for (int r = 0; r < 2; ++r) {
-        row_max[r] = x.sink ? sink_of(x, row_head[r]) : -CUDART_INF_F;
+        row_max[r] = x.sink ? sink_of(x, tile.first_token + (warp * 16 + (lane >> 2) + 8 * r) / group, nq, row_head[r]) : -CUDART_INF_F;
         row_sum[r] = x.sink && (lane & 3) == 0 ? 1.0f : 0.0f;
     }
 
@@ -411,7 +414,7 @@ __global__ void __launch_bounds__(THREADS) attention_biased_keys_kernel(
         const int row = idx / E, col = idx % E;
         if (row >= rows) continue;
         const bool with_sink = x.sink && splits == 1;          // among several CTAs the sink joins in the combine kernel
-        const float sink_logit = with_sink ? sink_of(x, kv_head * group + row % group) : 0.0f;
+        const float sink_logit = with_sink ? sink_of(x, tile.first_token + row / group, nq, kv_head * group + row % group) : 0.0f;
         float m = with_sink ? sink_logit : -CUDART_INF_F;
 #pragma unroll
         for (int w = 0; w < 4; ++w) m = fmaxf(m, merge_ml[(w * ROWS_NARROW + row) * 2]);
@@ -438,7 +441,7 @@ __global__ void __launch_bounds__(THREADS) attention_biased_keys_kernel(
 // Merges the partial results of a tile's `splits` CTAs, adds the sink and applies the gate.
 __global__ void __launch_bounds__(THREADS) attention_biased_combine_kernel(
     const float* __restrict__ part_o, const float* __restrict__ part_ml, const Tile* __restrict__ tiles, bf16* __restrict__ out,
-    const float* __restrict__ gate, int nq, int nkv, int splits, int sink, const float* __restrict__ sink_logits) {
+    int nq, int nkv, int splits, Extras x) {
     pdl_launch_dependents();
     pdl_wait();
     const Tile tile = tiles[blockIdx.x];
@@ -446,7 +449,9 @@ __global__ void __launch_bounds__(THREADS) attention_biased_combine_kernel(
     const size_t base_slot = ((size_t)blockIdx.x * nkv + kv_head) * splits * ROWS_NARROW;
     const int row = blockIdx.z;                       // a CTA a row: few tiles still fill the GPU
     if (row >= rows) return;
-    const float sink_logit = sink && sink_logits ? sink_logits[kv_head * group + row % group] * LOG2E : 0.0f;
+    const bool sink = x.sink;
+    const float* gate = x.gate;
+    const float sink_logit = sink ? sink_of(x, tile.first_token + row / group, nq, kv_head * group + row % group) : 0.0f;
     for (int col = threadIdx.x; col < E; col += THREADS) {
         float m = sink ? sink_logit : -CUDART_INF_F;
         for (int s = 0; s < splits; ++s) m = fmaxf(m, part_ml[(base_slot + (size_t)s * ROWS_NARROW + row) * 2]);
@@ -492,16 +497,16 @@ MRS_EXPORT int mrs_attention_biased_mma(int narrow, const void* q, const void* k
                                         const int* block_table, int table_width, const int* tiles, int num_tiles, void* out,
                                         const float* bias, int bias_rows, const float* gate, int nq, int nkv, int page_size,
                                         float scale, float cap, int window, int keep_first, int sink, int splits, float* scratch,
-                                        const float* sink_logits, int chunk, void* stream) {
+                                        const float* sink_logits, int sink_heads, int chunk, void* stream) {
     if (num_tiles <= 0) return 0;
     if (splits < 1 || splits > 65535 || (splits > 1 && (!narrow || !scratch)) || (!IN_KEYS && !v_cache)) return MRS_BAD_ARGUMENT;
     const int shift = page_shift_of(page_size);
     if (shift < 0 || nkv <= 0 || nq % nkv || nq / nkv > (narrow ? ROWS_NARROW : ROWS_WIDE) || (bias && bias_rows <= 0) || window < 0 ||
-        keep_first < 0 || chunk < 0 || (chunk > 0 && window > 0) || (sink_logits && !sink))
+        keep_first < 0 || chunk < 0 || (chunk > 0 && window > 0) || (sink_logits && (!sink || sink_heads < nq || sink_heads % nq)))
         return MRS_BAD_ARGUMENT;
     Extras x;
     x.bias = bias, x.gate = gate, x.bias_rows = bias_rows, x.scale = scale, x.cap = cap, x.window = window, x.keep_first = keep_first;
-    x.sink = sink, x.sink_logits = sink_logits, x.chunk = chunk;
+    x.sink = sink, x.sink_logits = sink_logits, x.sink_heads = sink_heads, x.chunk = chunk;
     static bool configured[2] = {false, false};
     if (!configured[narrow ? 1 : 0]) {
         cudaError_t e = narrow
@@ -518,7 +523,7 @@ MRS_EXPORT int mrs_attention_biased_mma(int narrow, const void* q, const void* k
                    page_size, shift, x, part_o, part_ml, splits);
         if (splits > 1)
             MRS_LAUNCH(attention_biased_combine_kernel, dim3(num_tiles, nkv, ROWS_NARROW), E < THREADS ? 32 * ((E + 31) / 32) : THREADS, 0, stream, (const float*)part_o,
-                       (const float*)part_ml, (const Tile*)tiles, (bf16*)out, gate, nq, nkv, splits, sink, sink_logits);
+                       (const float*)part_ml, (const Tile*)tiles, (bf16*)out, nq, nkv, splits, x);
     } else
         MRS_LAUNCH(attention_biased_rows_kernel, dim3(num_tiles, nkv), THREADS, smem_rows, stream, (const bf16*)q, (const bf16*)k_cache,
                    (const bf16*)v_cache, positions, block_table, table_width, (const Tile*)tiles, (bf16*)out, nq, nkv, page_size, shift, x);

@@ -298,21 +298,21 @@ __global__ void qk_norm_rope_store_kernel(const T* __restrict__ qkv, T* __restri
 // The cosines and sines of every token's angles, once a step for all layers that share the
 // frequencies: out[t][j] = (cos, sin)(position[t] * inv_freq[j]), float32.
 __global__ void rotation_table_kernel(const int* __restrict__ positions, const float* __restrict__ inv_freq, long long total,
-                                      int half, float2* __restrict__ out) {
+                                      int half, float magnitude, float2* __restrict__ out) {
     pdl_launch_dependents();
     pdl_wait();
     const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
     if (i >= total) return;
     float s, c;
     sincosf((float)positions[i / half] * inv_freq[i % half], &s, &c);
-    out[i] = make_float2(c, s);
+    out[i] = make_float2(c * magnitude, s * magnitude);
 }
 
-MRS_EXPORT int mrs_rotation_table(const int* positions, const float* inv_freq, int tokens, int half, float* out, void* stream) {
+MRS_EXPORT int mrs_rotation_table(const int* positions, const float* inv_freq, int tokens, int half, float magnitude, float* out, void* stream) {
     const long long total = (long long)tokens * half;
     if (total <= 0) return 0;
     if (!positions || !inv_freq || !out || ((uintptr_t)out & 15)) return MRS_BAD_ARGUMENT;
-    MRS_LAUNCH(rotation_table_kernel, (unsigned)((total + 255) / 256), 256, 0, stream, positions, inv_freq, total, half,
+    MRS_LAUNCH(rotation_table_kernel, (unsigned)((total + 255) / 256), 256, 0, stream, positions, inv_freq, total, half, magnitude,
                reinterpret_cast<float2*>(out));
     MRS_RETURN_LAUNCH_STATUS();
 }

@@ -1,6 +1,6 @@
 // Routed experts with shapes that do not depend on the routing, so that a step can be recorded and replayed:
 //
-//   moe_route      float32 router logits [tokens, all experts (+ 1 gate of the shared expert)] -> scores by softmax
+//   moe_route      float32 router logits [tokens, all experts (+ 1 gate of the shared expert)] (+ a bias an expert) -> scores by softmax
 //                  (or sigmoid) over all experts, the `top` largest of score + correction (ties: the lower number),
 //                  their weights score / (sum of the chosen scores + 1e-20) * scale (or, not normalised, score * scale),
 //                  sigmoid of the shared gate
@@ -27,7 +27,7 @@
 namespace {
 
 // One warp a token.  Dynamic shared memory: warps * 2 * all floats (scores, choice scores).
-__global__ void moe_route_kernel(const float* __restrict__ logits, int stride, const float* __restrict__ correction,
+__global__ void moe_route_kernel(const float* __restrict__ logits, int stride, const float* __restrict__ bias, const float* __restrict__ correction,
                                  int* __restrict__ chosen, float* __restrict__ weights, float* __restrict__ shared_gate, int tokens,
                                  int all, int top, float scale, int sigmoid_scores, int has_shared, int normalize) {
     pdl_launch_dependents();
@@ -40,11 +40,12 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, int stride, c
     float* choice = score + all;
     const float* z = logits + (size_t)t * stride;
     float top_z = -CUDART_INF_F;
-    for (int e = lane; e < all; e += 32) top_z = fmaxf(top_z, z[e]);
+    auto logit = [&](int e) { return bias ? z[e] + bias[e] : z[e]; };
+    for (int e = lane; e < all; e += 32) top_z = fmaxf(top_z, logit(e));
     top_z = warp_max(top_z);
     float sum = 0.0f;
     for (int e = lane; e < all; e += 32) {
-        const float s = sigmoid_scores ? 1.0f / (1.0f + expf(-z[e])) : expf(z[e] - top_z);
+        const float s = sigmoid_scores ? 1.0f / (1.0f + expf(-logit(e))) : expf(logit(e) - top_z);
         score[e] = s;
         sum += s;
     }
@@ -430,7 +431,7 @@ __global__ void moe_combine_vec_kernel(const T* __restrict__ y, const T* __restr
 
 MRS_EXPORT int mrs_moe_simt_tile() { return SIMT_TM; }
 
-MRS_EXPORT int mrs_moe_route(const float* logits, int stride, const float* correction, int* chosen, float* weights, float* shared_gate,
+MRS_EXPORT int mrs_moe_route(const float* logits, int stride, const float* bias, const float* correction, int* chosen, float* weights, float* shared_gate,
                              int tokens, int all, int top, float scale, int sigmoid_scores, int has_shared, int normalize, void* stream) {
     if (tokens <= 0) return 0;
     if (all <= 0 || top <= 0 || top > all || stride < all + (has_shared ? 1 : 0) || (has_shared && !shared_gate)) return MRS_BAD_ARGUMENT;
@@ -438,7 +439,7 @@ MRS_EXPORT int mrs_moe_route(const float* logits, int stride, const float* corre
     while (warps > 1 && (size_t)warps * 2 * all * sizeof(float) > 40 * 1024) warps >>= 1;
     const size_t smem = (size_t)warps * 2 * all * sizeof(float);
     if (smem > 48 * 1024) return MRS_BAD_ARGUMENT;
-    MRS_LAUNCH(moe_route_kernel, (tokens + warps - 1) / warps, 32 * warps, smem, stream, logits, stride, correction, chosen, weights,
+    MRS_LAUNCH(moe_route_kernel, (tokens + warps - 1) / warps, 32 * warps, smem, stream, logits, stride, bias, correction, chosen, weights,
                shared_gate, tokens, all, top, scale, sigmoid_scores, has_shared, normalize);
     MRS_RETURN_LAUNCH_STATUS();
 }

@@ -1,8 +1,9 @@
 // Kernels around a latent attention and a layer norm with bias (every size at run time, float32 or bfloat16
 // activations, statistics, angles and gates in float32):
 //
-//   add_layernorm     v = residual (+ delta);  out = (v - mean) / sqrt(var + eps) * weight + bias, var the mean of the
-//                     squared deviations (computed from the mean, not from the mean of squares)
+//   add_layernorm     v = residual (+ factor * delta + extra + row, each where given; extra a second branch, row a vector that
+//                     every row gets);  out = (v - mean) / sqrt(var + eps) * weight + bias, var the mean of the squared
+//                     deviations (computed from the mean, not from the mean of squares)
 //   latent_prepare    what follows the fused projection q | latent, rotated key | gate of a latent attention:
 //                     the unrotated query parts head-major for the product that carries them into the latent space,
 //                     the rotated query parts behind the latent columns of the query rows, the latent divided by its
@@ -13,7 +14,7 @@
 //                     their weights; the first goes on to the queries' up-projection, the second into the cache row
 //   sigmoid_gate_mul  x <- x * sigmoid(gate) element by element, the gate a column range of wider float32 rows
 //
-// Rotation: of the first `rotary` elements of a rotated part element i pairs with i + rotary / 2; the pair (u, v) at
+// Rotation: of the first `rotary` elements of a rotated part element i pairs with i + rotary / 2, or (interleaved) element 2 i with 2 i + 1; the pair (u, v) at
 // position p becomes (u c - v s, v c + u s) with c = m cos(p f_i), s = m sin(p f_i); the rest passes unchanged.
 #include "common.cuh"
 
@@ -42,9 +43,18 @@ template <> struct Row4<bf16> {
     }
 };
 
+// What is added to the stream before it is normed; D: the delta's type.
+template <typename D>
+struct Added {
+    const D* delta;          // [rows, width] or null
+    float factor;            // of the delta
+    const float* extra;      // [rows, width] or null
+    const float* row;        // [width] or null
+};
+
 // Any width: the row is read three times (sum, squared deviations, output).
-template <typename T>
-__global__ void add_layernorm_kernel(float* __restrict__ residual, const T* __restrict__ delta, const float* __restrict__ weight,
+template <typename T, typename D>
+__global__ void add_layernorm_kernel(float* __restrict__ residual, const Added<D> add, const float* __restrict__ weight,
                                      const float* __restrict__ bias, float eps, T* __restrict__ out, const int* __restrict__ rows,
                                      int width, int write_back) {
     pdl_launch_dependents();
@@ -53,32 +63,40 @@ __global__ void add_layernorm_kernel(float* __restrict__ residual, const T* __re
     const int r = blockIdx.x;
     const size_t src = rows ? (size_t)rows[r] : (size_t)r;
     float* res = residual + src * width;
-    const T* del = delta ? delta + src * width : nullptr;
+    const D* del = add.delta ? add.delta + src * width : nullptr;
+    const float* extra = add.extra ? add.extra + src * width : nullptr;
+    auto more = [&](int i) {
+        float v = del ? add.factor * to_float(del[i]) : 0.0f;
+        if (extra) v += extra[i];
+        if (add.row) v += add.row[i];
+        return v;
+    };
+    const bool adds = del || extra || add.row;
     float sum = 0.0f;
     for (int i = threadIdx.x; i < width; i += blockDim.x) {
         float v = res[i];
-        if (del) v += to_float(del[i]);
-        if (write_back && del) res[i] = v;
+        if (adds) v += more(i);
+        if (write_back && adds) res[i] = v;
         sum += v;
     }
-    const bool again = del && !write_back;         // the sum is not in memory: add the branch again
+    const bool again = adds && !write_back;        // the sum is not in memory: add the branch again
     const float mean = block_sum(sum, scratch) / (float)width;
     float dev = 0.0f;
     for (int i = threadIdx.x; i < width; i += blockDim.x) {
-        const float v = res[i] + (again ? to_float(del[i]) : 0.0f) - mean;
+        const float v = res[i] + (again ? more(i) : 0.0f) - mean;
         dev += v * v;
     }
     const float scale = rsqrtf(block_sum(dev, scratch) / (float)width + eps);
     T* o = out + (size_t)r * width;
     for (int i = threadIdx.x; i < width; i += blockDim.x) {
-        const float v = res[i] + (again ? to_float(del[i]) : 0.0f) - mean;
+        const float v = res[i] + (again ? more(i) : 0.0f) - mean;
         o[i] = from_float<T>(v * scale * weight[i] + bias[i]);
     }
 }
 
 // Width a multiple of 4, at most 4 * LN_CHUNKS * blockDim.x: the row stays in registers between the passes.
-template <typename T>
-__global__ void add_layernorm_vec_kernel(float* __restrict__ residual, const T* __restrict__ delta, const float* __restrict__ weight,
+template <typename T, typename D>
+__global__ void add_layernorm_vec_kernel(float* __restrict__ residual, const Added<D> add, const float* __restrict__ weight,
                                          const float* __restrict__ bias, float eps, T* __restrict__ out, const int* __restrict__ rows,
                                          int width, int write_back) {
     pdl_launch_dependents();
@@ -87,7 +105,9 @@ __global__ void add_layernorm_vec_kernel(float* __restrict__ residual, const T* 
     const int r = blockIdx.x;
     const size_t src = rows ? (size_t)rows[r] : (size_t)r;
     float* res = residual + src * width;
-    const T* del = delta ? delta + src * width : nullptr;
+    const D* del = add.delta ? add.delta + src * width : nullptr;
+    const float* extra = add.extra ? add.extra + src * width : nullptr;
+    const bool adds = del || extra || add.row;
     float4 v[LN_CHUNKS];
     float sum = 0.0f;
 #pragma unroll
@@ -97,10 +117,18 @@ __global__ void add_layernorm_vec_kernel(float* __restrict__ residual, const T* 
         if (i < width) {
             v[c] = Row4<float>::load(res + i);
             if (del) {
-                const float4 d = Row4<T>::load(del + i);
-                v[c].x += d.x, v[c].y += d.y, v[c].z += d.z, v[c].w += d.w;
-                if (write_back) Row4<float>::store(res + i, v[c]);
+                const float4 d = Row4<D>::load(del + i);
+                v[c].x += add.factor * d.x, v[c].y += add.factor * d.y, v[c].z += add.factor * d.z, v[c].w += add.factor * d.w;
             }
+            if (extra) {
+                const float4 d = Row4<float>::load(extra + i);
+                v[c].x += d.x, v[c].y += d.y, v[c].z += d.z, v[c].w += d.w;
+            }
+            if (add.row) {
+                const float4 d = Row4<float>::load(add.row + i);
+                v[c].x += d.x, v[c].y += d.y, v[c].z += d.z, v[c].w += d.w;
+            }
+            if (write_back && adds) Row4<float>::store(res + i, v[c]);
             sum += (v[c].x + v[c].y) + (v[c].z + v[c].w);
         }
     }
@@ -135,7 +163,7 @@ __global__ void scale_kernel(float* __restrict__ x, long long n, float factor) {
 
 struct LatentSizes {
     int heads, plain, rotated, latent, rotary;      // per head: unrotated and rotated query/key elements; latent size; rotated pairs * 2
-    int has_latent, has_gate;
+    int has_latent, has_gate, interleaved;
 };
 
 // One block a token.  Columns of a projected row: heads * (plain + rotated) of q, then (has_latent) latent + rotated,
@@ -163,6 +191,11 @@ __global__ void latent_prepare_kernel(const float* __restrict__ proj, int proj_w
     const int per_head = z.plain + z.rotated, key_width = z.latent + z.rotated;
     auto rotated_at = [&](const float* part, int i) {        // element i of a rotated part
         if (i >= z.rotary) return part[i];
+        if (z.interleaved) {
+            const int j = i >> 1;
+            const float u = part[2 * j], v = part[2 * j + 1], c = turn[j], s = turn[half + j];
+            return (i & 1) == 0 ? u * c - v * s : v * c + u * s;
+        }
         const int j = i < half ? i : i - half;
         const float u = part[j], v = part[j + half], c = turn[j], s = turn[half + j];
         return i < half ? u * c - v * s : v * c + u * s;
@@ -231,30 +264,33 @@ __global__ void sigmoid_gate_mul_kernel(T* __restrict__ x, const float* __restri
 
 }  // namespace
 
-MRS_EXPORT int mrs_add_layernorm(int is_bf16, float* residual, const void* delta, const float* weight, const float* bias, float eps,
-                                 void* out, const int* rows, int n_rows, int width, int write_back, void* stream) {
-    if (n_rows <= 0) return 0;
-    if (width <= 0) return MRS_BAD_ARGUMENT;
-    const bool aligned = (((uintptr_t)residual | (uintptr_t)delta | (uintptr_t)weight | (uintptr_t)bias | (uintptr_t)out) & 15) == 0;
+template <typename T, typename D>
+static int launch_add_layernorm(float* residual, const void* delta, float factor, const float* extra, const float* row, const float* weight,
+                                const float* bias, float eps, void* out, const int* rows, int n_rows, int width, int write_back, void* stream) {
+    Added<D> add;
+    add.delta = (const D*)delta, add.factor = factor, add.extra = extra, add.row = row;
+    const bool aligned = (((uintptr_t)residual | (uintptr_t)delta | (uintptr_t)extra | (uintptr_t)row | (uintptr_t)weight | (uintptr_t)bias |
+                           (uintptr_t)out) & 15) == 0;
     if (width % 4 == 0 && aligned && width <= 4 * LN_CHUNKS * 1024) {
         int threads = ((width + 4 * LN_CHUNKS - 1) / (4 * LN_CHUNKS) + 31) / 32 * 32;
         if (threads < 64) threads = 64;
-        if (is_bf16)
-            MRS_LAUNCH(add_layernorm_vec_kernel<bf16>, n_rows, threads, 0, stream, residual, (const bf16*)delta, weight, bias, eps,
-                       (bf16*)out, rows, width, write_back);
-        else
-            MRS_LAUNCH(add_layernorm_vec_kernel<float>, n_rows, threads, 0, stream, residual, (const float*)delta, weight, bias, eps,
-                       (float*)out, rows, width, write_back);
+        MRS_LAUNCH((add_layernorm_vec_kernel<T, D>), n_rows, threads, 0, stream, residual, add, weight, bias, eps, (T*)out, rows, width, write_back);
         MRS_RETURN_LAUNCH_STATUS();
     }
     const int threads = width >= 2048 ? 512 : (width >= 512 ? 256 : 128);
-    if (is_bf16)
-        MRS_LAUNCH(add_layernorm_kernel<bf16>, n_rows, threads, 0, stream, residual, (const bf16*)delta, weight, bias, eps, (bf16*)out,
-                   rows, width, write_back);
-    else
-        MRS_LAUNCH(add_layernorm_kernel<float>, n_rows, threads, 0, stream, residual, (const float*)delta, weight, bias, eps,
-                   (float*)out, rows, width, write_back);
+    MRS_LAUNCH((add_layernorm_kernel<T, D>), n_rows, threads, 0, stream, residual, add, weight, bias, eps, (T*)out, rows, width, write_back);
     MRS_RETURN_LAUNCH_STATUS();
+}
+
+// The delta has out's type, or is float32 (`delta_float32`).
+MRS_EXPORT int mrs_add_layernorm(int is_bf16, float* residual, const void* delta, int delta_float32, float factor, const float* extra,
+                                 const float* row, const float* weight, const float* bias, float eps, void* out, const int* rows, int n_rows,
+                                 int width, int write_back, void* stream) {
+    if (n_rows <= 0) return 0;
+    if (width <= 0) return MRS_BAD_ARGUMENT;
+    if (!is_bf16) return launch_add_layernorm<float, float>(residual, delta, factor, extra, row, weight, bias, eps, out, rows, n_rows, width, write_back, stream);
+    if (delta_float32) return launch_add_layernorm<bf16, float>(residual, delta, factor, extra, row, weight, bias, eps, out, rows, n_rows, width, write_back, stream);
+    return launch_add_layernorm<bf16, bf16>(residual, delta, factor, extra, row, weight, bias, eps, out, rows, n_rows, width, write_back, stream);
 }
 
 // x *= factor over n float32 elements (logits that a design scales by a constant).
@@ -271,7 +307,7 @@ MRS_EXPORT int mrs_scale(float* x, long long n, float factor, void* stream) {
 MRS_EXPORT int mrs_latent_prepare(int is_bf16, const float* proj, int proj_width, const float* latent_weight, float eps,
                                   const float* inv_freq, float magnitude, const int* positions, const int* slots, void* q_plain,
                                   void* q_rows, void* cache, float* gate, int tokens, int heads, int plain, int rotated, int latent,
-                                  int rotary, int has_latent, int has_gate, void* stream) {
+                                  int rotary, int interleaved, int has_latent, int has_gate, void* stream) {
     if (tokens <= 0) return 0;
     if (heads <= 0 || plain <= 0 || rotated < 0 || latent <= 0 || rotary < 0 || rotary > rotated || rotary % 2 || (rotary && !inv_freq) ||
         (has_latent && !latent_weight) || (has_gate && !gate) ||
@@ -279,6 +315,7 @@ MRS_EXPORT int mrs_latent_prepare(int is_bf16, const float* proj, int proj_width
         return MRS_BAD_ARGUMENT;
     LatentSizes z;
     z.heads = heads, z.plain = plain, z.rotated = rotated, z.latent = latent, z.rotary = rotary, z.has_latent = has_latent, z.has_gate = has_gate;
+    z.interleaved = interleaved;
     const size_t smem = (size_t)(rotary > 0 ? rotary : 1) * sizeof(float);
     if (is_bf16)
         MRS_LAUNCH(latent_prepare_kernel<bf16>, tokens, 256, smem, stream, proj, proj_width, latent_weight, eps, inv_freq, magnitude,

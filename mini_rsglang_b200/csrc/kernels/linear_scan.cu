@@ -2,8 +2,8 @@
 //
 //     S_t = keep_t S_(t-1) + take_t k_t v_t^T,   o_t = S_t^T q_t          (and with a normaliser n_t likewise with k alone, c_t = n_t . q_t)
 //
-// keep is a constant a head (a retention: take = 1) or comes a token with take (gates of an exponential memory).  Everything
-// here is float32.  S (and n) live in the request's state slot between steps; where a sequence starts at position 0 its
+// keep is a constant a head (a retention: take = 1), comes a token with take (gates of an exponential memory), or is one number
+// a token and key channel, which then acts on the rows of S (a gated linear attention: take = 1).  Everything here is float32.  S (and n) live in the request's state slot between steps; where a sequence starts at position 0 its
 // state counts as zero, whatever the slot held (slots are used again).  State slot -1: a padding sequence, nothing is read or
 // written.  The step's facts come from device arrays only, so a step can be recorded.
 //
@@ -11,6 +11,7 @@
 //   memory_gates       keep, take and exp(-m) of every (token, head) from the raw gates of an exponential memory with a running
 //                      maximum m (which starts at 0)
 //   linear_scan        the recurrence (linear_step: the same for decoded tokens)
+//   channel_fold       keeps a key channel from two thin products, folded into k and q so that the recurrence itself meets none
 //   narrow_columns     a range of float32 columns as rows of the engine's dtype
 #include "common.cuh"
 #include "pairs.cuh"
@@ -165,7 +166,88 @@ struct ScanArgs {
     int heads, d, e, cols, slices, batch, write_state, vec_qk, vec_v, vec_state, vec_out;
     float *chunk_state, *chunk_decay;
     int chunk_len, max_chunks, chunk_floats;
+    // keeps a key channel (CHANNEL); rows of a batch are then counted from the step's first row, and so are those of a chunk
+    float* keeps;                        // [tokens, heads * d]: what channel_fold leaves
+    int* direct;                         // [batches, heads]: the batch's keeps are applied token by token
+    int vec_keeps;
+    // what a decoded token's keeps are made of
+    const float* low;                    // a column range of the float32 rows: the first thin product, `rank` wide
+    const void* up;                      // [heads * d, rank], float32 or bfloat16: the second
+    const float* keep_bias;              // [heads * d]
+    float inverse_tau;
+    int rank;
 };
+
+// sigmoid(z)^(1 / tau)
+__device__ __forceinline__ float channel_keep(float z, float inverse_tau) { return expf(log_sigmoid_f(z) * inverse_tau); }
+
+// ---------------------------------------------------------------------------------------------
+// Keeps a key channel: a_t = sigmoid(up low_t + bias)^(1 / tau), [heads * d] a token.  The decay acts on the rows of S, so with P_t
+// a channel's product of keeps since its batch (of `batch` rows, counted from the step's first row) or its sequence began,
+// S_t = diag(P_t) U_t with U_t = U_(t-1) + (k_t / P_t) v_t^T and o_t = U_t^T (P_t q_t): k and q are divided and multiplied in place,
+// P goes to `keeps`, and the recurrence multiplies S by P once a batch.  Where some P of a (batch, head) falls below FOLD_LEAST
+// nothing is folded there: `keeps` gets the keeps themselves and `direct` says so.
+// A thread takes a channel and the rows of a batch; a block whole heads.  Dynamic shared memory: batch * rank floats.
+// ---------------------------------------------------------------------------------------------
+#define FOLD_LEAST 1e-15f
+template <typename W>
+__global__ void channel_fold_kernel(const ScanArgs A, float* __restrict__ q, float* __restrict__ k, const int* __restrict__ seq_of_token,
+                                    int tokens, int heads_a_block) {
+    extern __shared__ __align__(16) float low_rows[];
+    __shared__ int small[32];
+    pdl_launch_dependents();
+    pdl_wait();
+    const int t0 = blockIdx.x * A.batch, n = min(A.batch, tokens - t0);
+    const int head0 = blockIdx.y * heads_a_block, own = threadIdx.x / A.d;
+    const bool live = own < heads_a_block && head0 + own < A.heads;
+    for (int i = threadIdx.x; i < n * A.rank; i += blockDim.x)
+        low_rows[i] = A.low[(size_t)(t0 + i / A.rank) * A.stride + i % A.rank];
+    if (threadIdx.x < 32) small[threadIdx.x] = 0;
+    __syncthreads();
+    const int channel = head0 * A.d + threadIdx.x;
+    float a[SCAN_BATCH], P[SCAN_BATCH];
+    if (live) {
+        const float b = A.keep_bias[channel];
+#pragma unroll
+        for (int j = 0; j < SCAN_BATCH; ++j) a[j] = b;
+        const W* up = (const W*)A.up + (size_t)channel * A.rank;
+        for (int r = 0; r < A.rank; ++r) {
+            const float w = to_float(up[r]);
+#pragma unroll
+            for (int j = 0; j < SCAN_BATCH; ++j)
+                if (j < n) a[j] = fmaf(w, low_rows[j * A.rank + r], a[j]);
+        }
+        float p = 1.0f;
+        bool tiny = false;
+        int before = -1;
+#pragma unroll
+        for (int j = 0; j < SCAN_BATCH; ++j) {
+            if (j >= n) continue;
+            const int seq = seq_of_token[t0 + j];
+            if (seq != before) p = 1.0f;
+            before = seq;
+            a[j] = channel_keep(a[j], A.inverse_tau);
+            p *= a[j];
+            P[j] = p;
+            tiny = tiny || p < FOLD_LEAST;
+        }
+        if (tiny) small[own] = 1;
+    }
+    __syncthreads();
+    if (!live) return;
+    const bool direct = small[own];
+#pragma unroll
+    for (int j = 0; j < SCAN_BATCH; ++j) {
+        if (j >= n) continue;
+        const size_t t = t0 + j;
+        A.keeps[t * A.heads * A.d + channel] = direct ? a[j] : P[j];
+        if (!direct) {
+            k[t * A.stride + channel] /= P[j];
+            q[t * A.stride + channel] *= P[j];
+        }
+    }
+    if (threadIdx.x % A.d == 0) A.direct[(size_t)blockIdx.x * A.heads + head0 + own] = direct;
+}
 
 __device__ __forceinline__ void scan_copy16(float* to, const float* from) {
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"((uint32_t)__cvta_generic_to_shared(to)), "l"(from));
@@ -174,7 +256,7 @@ __device__ __forceinline__ void scan_copy4(float* to, const float* from) {
     asm volatile("cp.async.ca.shared.global [%0], [%1], 4;\n" ::"r"((uint32_t)__cvta_generic_to_shared(to)), "l"(from));
 }
 
-template <int MODE, int PARTS>
+template <int MODE, int PARTS, bool CHANNEL>
 __global__ void __launch_bounds__(256, 2) linear_scan_kernel(const ScanArgs A) {
     extern __shared__ __align__(16) float stage[];
     __shared__ __align__(16) float4 facts[2][SCAN_BATCH];    // of a token: take / p, p, keep, take; p the batch's product of keeps so far
@@ -183,7 +265,7 @@ __global__ void __launch_bounds__(256, 2) linear_scan_kernel(const ScanArgs A) {
     constexpr int PAIRS = SCAN_ROWS / 2;
     pdl_launch_dependents();
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
-    const int token_floats = 2 * VECTOR + A.cols, stage_floats = A.batch * token_floats;
+    const int token_floats = 2 * VECTOR + A.cols, stage_floats = A.batch * token_floats + (CHANNEL ? VECTOR : 0);
     for (int i = threadIdx.x; i < 2 * stage_floats; i += blockDim.x) stage[i] = 0.0f;      // rows beyond d, columns beyond e
     __syncthreads();
     pdl_wait();
@@ -191,8 +273,9 @@ __global__ void __launch_bounds__(256, 2) linear_scan_kernel(const ScanArgs A) {
     const int seq_first = A.q_start[seq], seq_last = A.q_start[seq + 1];
     const int slot = A.state_slots[seq];
     if (slot < 0 || seq_last <= seq_first) return;
-    const int first = MODE == SCAN_WHOLE ? seq_first : seq_first + chunk * A.chunk_len;
-    const int last = MODE == SCAN_WHOLE ? seq_last : min(seq_last, first + A.chunk_len);
+    const int chunk_first = MODE == SCAN_WHOLE ? 0 : ((CHANNEL ? seq_first / A.chunk_len : 0) + chunk) * A.chunk_len + (CHANNEL ? 0 : seq_first);
+    const int first = MODE == SCAN_WHOLE ? seq_first : max(seq_first, chunk_first);
+    const int last = MODE == SCAN_WHOLE ? seq_last : min(seq_last, chunk_first + A.chunk_len);
     if (first >= last) return;
     const int part = lane / GROUPS, place = (warp * GROUPS + lane % GROUPS) * 4, col = slice * A.cols + place;
     const int row0 = part * SCAN_ROWS;
@@ -230,8 +313,20 @@ __global__ void __launch_bounds__(256, 2) linear_scan_kernel(const ScanArgs A) {
                 for (int i = lane; i < live_cols; i += 32) scan_copy4(to + 2 * VECTOR + i, A.v + row + v_at + i);
             }
         }
+        if (CHANNEL && warp == warps - 1) {                  // what S is multiplied by behind the batch
+            const float* from = A.keeps + (size_t)(t0 + n - 1) * A.heads * A.d + q_at;
+            float* to = base + A.batch * token_floats;
+            if (A.vec_keeps) {
+                for (int i = 4 * lane; i < A.d; i += 128) scan_copy16(to + (i / SCAN_ROWS) * SCAN_PITCH + i % SCAN_ROWS, from + i);
+            } else {
+                for (int i = lane; i < A.d; i += 32) scan_copy4(to + (i / SCAN_ROWS) * SCAN_PITCH + i % SCAN_ROWS, from + i);
+            }
+        }
         asm volatile("cp.async.commit_group;\n" ::);
     };
+    // rows of the batch that begins at row t
+    auto rows_at = [&](int t) { return min(CHANNEL ? A.batch - t % A.batch : A.batch, last - t); };
+    auto direct_at = [&](int t) { return CHANNEL && A.direct[(size_t)(t / A.batch) * A.heads + head] != 0; };
     const float fixed = A.decay ? A.decay[head] : 1.0f;
     auto read_facts = [&](int t0, int n) {                   // keep and take of token t0 + lane, warp 0
         if (A.decay || lane >= n) return make_float2(lane < n ? fixed : 1.0f, 1.0f);
@@ -247,8 +342,9 @@ __global__ void __launch_bounds__(256, 2) linear_scan_kernel(const ScanArgs A) {
         }
         if (lane < A.batch) facts[buffer][lane] = make_float4(raw.y / p, p, raw.x, raw.y);
     };
-    issue(first, min(A.batch, last - first), 0);
-    if (warp == 0) write_facts(read_facts(first, min(A.batch, last - first)), 0);
+    issue(first, rows_at(first), 0);
+    if (!CHANNEL && warp == 0) write_facts(read_facts(first, rows_at(first)), 0);
+    bool direct = direct_at(first);
 
     pair s[4][PAIRS];                                        // a column's rows two by two
 #pragma unroll
@@ -340,20 +436,54 @@ __global__ void __launch_bounds__(256, 2) linear_scan_kernel(const ScanArgs A) {
     };
 
     float P = 1.0f, product = 1.0f;
-    const int batches = (last - first + A.batch - 1) / A.batch;
-    for (int b = 0; b < batches; ++b) {
-        const int t0 = first + b * A.batch, n = min(A.batch, last - t0);
+    for (int t0 = first, b = 0; t0 < last; ++b) {
+        const int n = rows_at(t0), t1 = t0 + n;
         float2 next = make_float2(1.0f, 1.0f);
-        if (b + 1 < batches) {
-            const int n1 = min(A.batch, last - t0 - A.batch);
-            issue(t0 + A.batch, n1, (b + 1) & 1);
-            if (warp == 0) next = read_facts(t0 + A.batch, n1);
+        bool next_direct = false;
+        if (t1 < last) {
+            const int n1 = rows_at(t1);
+            issue(t1, n1, (b + 1) & 1);
+            if (!CHANNEL && warp == 0) next = read_facts(t1, n1);
+            next_direct = direct_at(t1);
             asm volatile("cp.async.wait_group 1;\n" ::);
         } else {
             asm volatile("cp.async.wait_group 0;\n" ::);
         }
         __syncthreads();
         const float* token = stage + (b & 1) * stage_floats;
+        if constexpr (CHANNEL) {
+            if (!idle && direct) {
+                for (int j = 0; j < n; ++j, token += token_floats) {
+                    const float* keep = A.keeps + (size_t)(t0 + j) * A.heads * A.d + q_at;
+#pragma unroll
+                    for (int i = 0; i < PAIRS; ++i) {
+                        const int row = row0 + 2 * i;
+                        const pair f = make_pair(row < A.d ? keep[row] : 0.0f, row + 1 < A.d ? keep[row + 1] : 0.0f);
+#pragma unroll
+                        for (int c = 0; c < 4; ++c) s[c][i] = mul2(s[c][i], f);
+                    }
+                    walk(token, 1.0f, 1.0f);
+                    to += out_step;
+                }
+            } else if (!idle) {
+                const float* keep = token + A.batch * token_floats + part * SCAN_PITCH;
+#pragma unroll 1
+                for (int j = 0; j < n; ++j, token += token_floats) {
+                    walk(token, 1.0f, 1.0f);
+                    to += out_step;
+                }
+#pragma unroll
+                for (int i = 0; i < PAIRS; i += 2) {
+                    const ulonglong2 f = *reinterpret_cast<const ulonglong2*>(keep + 2 * i);
+#pragma unroll
+                    for (int c = 0; c < 4; ++c) s[c][i] = mul2(s[c][i], f.x), s[c][i + 1] = mul2(s[c][i + 1], f.y);
+                }
+            }
+            direct = next_direct;
+            t0 = t1;
+            __syncthreads();                                 // the stage is copied into again two batches on
+            continue;
+        }
         const float4* fact = facts[b & 1];
         const float end = fact[n - 1].y;                     // the batch's product of keeps, the same for every thread
         if (MODE == SCAN_LOCAL) product *= end;
@@ -379,10 +509,26 @@ __global__ void __launch_bounds__(256, 2) linear_scan_kernel(const ScanArgs A) {
             }
         }
         if (end >= SCAN_LEAST) P *= end;
-        if (warp == 0 && b + 1 < batches) write_facts(next, (b + 1) & 1);
+        if (warp == 0 && t1 < last) write_facts(next, (b + 1) & 1);
+        t0 = t1;
         __syncthreads();                                     // the stage is copied into again two batches on
     }
-    if (MODE == SCAN_LOCAL && threadIdx.x == 0 && slice == 0) A.chunk_decay[chunk_at] = product;
+    if (MODE == SCAN_LOCAL && !CHANNEL && threadIdx.x == 0 && slice == 0) A.chunk_decay[chunk_at] = product;
+    if (MODE == SCAN_LOCAL && CHANNEL && slice == 0) {
+        for (int i = threadIdx.x; i < A.d; i += blockDim.x) {
+            float p = 1.0f;
+            for (int t0 = first; t0 < last;) {
+                const int n = rows_at(t0);
+                if (direct_at(t0)) {
+                    for (int j = 0; j < n; ++j) p *= A.keeps[(size_t)(t0 + j) * A.heads * A.d + q_at + i];
+                } else {
+                    p *= A.keeps[(size_t)(t0 + n - 1) * A.heads * A.d + q_at + i];
+                }
+                t0 += n;
+            }
+            A.chunk_decay[chunk_at * A.d + i] = p;
+        }
+    }
     if (MODE == SCAN_LOCAL || (MODE == SCAN_WHOLE && A.write_state)) {
         rescale(P);
 #pragma unroll
@@ -412,7 +558,9 @@ __global__ void __launch_bounds__(256, 2) linear_scan_kernel(const ScanArgs A) {
 // takes SCAN_ROWS rows of up to 128 neighbouring columns, four a lane, so that every access is a whole row of them and all of a
 // thread's loads are in flight together; the warps' parts of a token's read-out meet in shared memory.  Nothing is staged: k
 // and q are the same for a warp's lanes.  At most 16 warps (d up to 256).
+// CHANNEL: a warp makes its rows' keeps itself, from the first thin product and its rows of the second (W: their type).
 #define STEP_COLUMNS 128
+template <bool CHANNEL, typename W>
 __global__ void __launch_bounds__(512) linear_step_kernel(const ScanArgs A) {
     __shared__ __align__(16) float parts[2][16][STEP_COLUMNS];
     pdl_launch_dependents();
@@ -450,7 +598,17 @@ __global__ void __launch_bounds__(512) linear_step_kernel(const ScanArgs A) {
         const size_t row = (size_t)t * A.stride;
         const float *k = A.k + row + head * A.d + row0, *q = A.q + row + head * A.d + row0, *v = A.v + row + head * A.e + col;
         float keep = 1.0f, take = 1.0f;
-        if (A.decay) keep = A.decay[head];
+        if (CHANNEL) {                                       // two lanes a row; lane 2 i ends with the keep of row i
+            const int mine_row = row0 + (lane >> 1);
+            float z = 0.0f;
+            if (mine_row < A.d) {
+                const W* up = (const W*)A.up + ((size_t)head * A.d + mine_row) * A.rank;
+                const float* low = A.low + row;
+                for (int r = lane & 1; r < A.rank; r += 2) z = fmaf(to_float(up[r]), low[r], z);
+            }
+            z += __shfl_xor_sync(0xffffffffu, z, 1);
+            if (mine_row < A.d) keep = channel_keep(z + A.keep_bias[head * A.d + mine_row], A.inverse_tau);
+        } else if (A.decay) keep = A.decay[head];
         else keep = A.coef[(size_t)t * A.coef_stride + head], take = A.coef[(size_t)t * A.coef_stride + A.heads + head];
         float4 tv = make_float4(0.0f, 0.0f, 0.0f, 0.0f), y = tv;
         if (is_norm) {
@@ -476,8 +634,9 @@ __global__ void __launch_bounds__(512) linear_step_kernel(const ScanArgs A) {
 #pragma unroll
             for (int u = 0; u < 4; ++u) {
                 float4& r = s[i + u];
-                r.x = fmaf(keep, r.x, kk[u] * tv.x), r.y = fmaf(keep, r.y, kk[u] * tv.y);
-                r.z = fmaf(keep, r.z, kk[u] * tv.z), r.w = fmaf(keep, r.w, kk[u] * tv.w);
+                const float held = CHANNEL ? __shfl_sync(0xffffffffu, keep, 2 * (i + u)) : keep;
+                r.x = fmaf(held, r.x, kk[u] * tv.x), r.y = fmaf(held, r.y, kk[u] * tv.y);
+                r.z = fmaf(held, r.z, kk[u] * tv.z), r.w = fmaf(held, r.w, kk[u] * tv.w);
                 y.x = fmaf(r.x, qq[u], y.x), y.y = fmaf(r.y, qq[u], y.y), y.z = fmaf(r.z, qq[u], y.z), y.w = fmaf(r.w, qq[u], y.w);
             }
         }
@@ -512,7 +671,7 @@ __global__ void __launch_bounds__(512) linear_step_kernel(const ScanArgs A) {
 // A thread takes one element (VEC: four neighbouring ones) of a (sequence, head)'s S (and n behind it): chunk c's entry goes from
 // the chunk's end state from zero to the state at its start, in[0] = the slot's state (zero at position 0), in[c + 1] =
 // product_c in[c] + end_c.  The end states of eight chunks are asked for together.
-template <bool VEC>
+template <bool VEC, bool CHANNEL>
 __global__ void scan_chunk_states_kernel(const ScanArgs A, int elements) {
     pdl_launch_dependents();
     pdl_wait();
@@ -523,10 +682,12 @@ __global__ void scan_chunk_states_kernel(const ScanArgs A, int elements) {
     if (slot < 0 || rows <= 0) return;
     const int i = (blockIdx.z * blockDim.x + threadIdx.x) * W;
     if (i >= elements) return;
-    const int chunks = (rows + A.chunk_len - 1) / A.chunk_len, matrix = A.d * A.e;
+    const int matrix = A.d * A.e;
+    const int chunks = CHANNEL ? (first + rows - 1) / A.chunk_len - first / A.chunk_len + 1 : (rows + A.chunk_len - 1) / A.chunk_len;
     const bool fresh = A.positions[first] == 0;
     float* local = A.chunk_state + ((size_t)seq * A.heads + head) * A.max_chunks * A.chunk_floats + i;
-    const float* product = A.chunk_decay + ((size_t)seq * A.heads + head) * A.max_chunks;
+    const int products = CHANNEL ? A.d : 1;                  // of a chunk
+    const float* product = A.chunk_decay + ((size_t)seq * A.heads + head) * A.max_chunks * products + (CHANNEL ? i / A.e : 0);
     float* slot_at = (i < matrix ? A.state + (size_t)head * matrix + i : A.norm_state + (size_t)head * A.d + (i - matrix)) +
                      (long long)slot * A.state_stride;
     float value[W];
@@ -538,7 +699,7 @@ __global__ void scan_chunk_states_kernel(const ScanArgs A, int elements) {
         for (int c = 0; c < AHEAD; ++c) {
             if (c0 + c >= chunks) continue;
             const float* from = local + (size_t)(c0 + c) * A.chunk_floats;
-            keep[c] = product[c0 + c];
+            keep[c] = product[(size_t)(c0 + c) * products];
             if (VEC) {
                 const float4 f = *reinterpret_cast<const float4*>(from);
                 end[c][0] = f.x;
@@ -604,6 +765,16 @@ MRS_EXPORT int mrs_memory_gates(const float* raw, int raw_stride, int i_offset, 
     MRS_RETURN_LAUNCH_STATUS();
 }
 
+// Tokens of a batch in shared memory; keeps a channel add one vector a batch.
+static int scan_batch(int parts, int cols, bool channel) {
+    const int budget = 40 * 1024 / (2 * (int)sizeof(float)) - (channel ? parts * SCAN_PITCH : 0);
+    int batch = budget / (2 * parts * SCAN_PITCH + cols);
+    if (batch > SCAN_BATCH) batch = SCAN_BATCH;
+    if (channel)
+        while (batch & (batch - 1)) --batch;                 // batches begin at multiples of their length, and so do chunks
+    return batch;
+}
+
 // How the recurrence is cut: lanes that share a column group, columns a block, slices of the columns.  Returns the slices.
 static int scan_shape(int d, int e, bool normaliser, int* parts_out, int* cols_out) {
     int parts = 1;
@@ -623,11 +794,57 @@ MRS_EXPORT int mrs_linear_scan_slices(int d, int e, int normaliser) {
     return scan_shape(d, e, normaliser != 0, &parts, &cols);
 }
 
-// Floats of scratch that a run in chunks needs.
-MRS_EXPORT long long mrs_linear_scan_scratch_floats(int tokens, int sequences, int heads, int d, int e, int normaliser, int chunk_len) {
+// Floats of scratch that a run in chunks needs.  `channel`: keeps a key channel.
+MRS_EXPORT long long mrs_linear_scan_scratch_floats(int tokens, int sequences, int heads, int d, int e, int normaliser, int chunk_len,
+                                                    int channel) {
     if (chunk_len <= 0) return 0;
     const long long chunks = (tokens + chunk_len - 1) / chunk_len;
-    return (long long)sequences * heads * chunks * (((long long)d * e + (normaliser ? d : 0) + 3) / 4 * 4 + 1);
+    return (long long)sequences * heads * chunks * (((long long)d * e + (normaliser ? d : 0) + 3) / 4 * 4 + (channel ? d : 1));
+}
+
+// Rows that a run in chunks of keeps a channel begins its chunks at multiples of (0: sizes that are not built).
+MRS_EXPORT int mrs_channel_scan_batch(int d, int e) {
+    int parts, cols;
+    if (d <= 0 || d > 512 || e <= 0) return 0;
+    scan_shape(d, e, false, &parts, &cols);
+    return scan_batch(parts, cols, true);
+}
+
+// The launches of a recurrence whose inputs and state stand in `A`.
+template <bool CHANNEL>
+static int scan_run(ScanArgs& A, int tokens, int sequences, int parts, float* scratch, void* s) {
+    const int d = A.d, e = A.e, heads = A.heads, chunk_len = A.chunk_len;
+    const int threads = A.cols / (4 * (32 / parts)) * 32;
+    const int token_floats = 2 * parts * SCAN_PITCH + A.cols;
+    const size_t smem = 2 * ((size_t)A.batch * token_floats + (CHANNEL ? parts * SCAN_PITCH : 0)) * sizeof(float);
+#define SCAN_LAUNCH(MODE, GRID)                                                                                  \
+    switch (parts) {                                                                                             \
+        case 1: MRS_LAUNCH((linear_scan_kernel<MODE, 1, CHANNEL>), GRID, threads, smem, s, A); break;             \
+        case 2: MRS_LAUNCH((linear_scan_kernel<MODE, 2, CHANNEL>), GRID, threads, smem, s, A); break;             \
+        case 4: MRS_LAUNCH((linear_scan_kernel<MODE, 4, CHANNEL>), GRID, threads, smem, s, A); break;             \
+        case 8: MRS_LAUNCH((linear_scan_kernel<MODE, 8, CHANNEL>), GRID, threads, smem, s, A); break;             \
+        case 16: MRS_LAUNCH((linear_scan_kernel<MODE, 16, CHANNEL>), GRID, threads, smem, s, A); break;           \
+        default: MRS_LAUNCH((linear_scan_kernel<MODE, 32, CHANNEL>), GRID, threads, smem, s, A); break;           \
+    }
+    if (chunk_len == 0) {
+        SCAN_LAUNCH(SCAN_WHOLE, dim3(sequences, heads * A.slices));
+        MRS_RETURN_LAUNCH_STATUS();
+    }
+    A.max_chunks = (tokens + chunk_len - 1) / chunk_len;
+    if (A.max_chunks > 65535) return MRS_BAD_ARGUMENT;
+    const int elements = d * e + (A.norm_state ? d : 0);
+    A.chunk_floats = (elements + 3) / 4 * 4;
+    A.chunk_state = scratch;
+    A.chunk_decay = scratch + (size_t)sequences * heads * A.max_chunks * A.chunk_floats;
+    A.vec_state = e % 4 == 0;
+    SCAN_LAUNCH(SCAN_LOCAL, dim3(sequences, heads * A.slices, A.max_chunks));
+    if (d * e % 4 == 0 && elements % 4 == 0 && A.vec_state)
+        MRS_LAUNCH((scan_chunk_states_kernel<true, CHANNEL>), dim3(sequences, heads, (elements / 4 + 127) / 128), 128, 0, s, A, elements);
+    else
+        MRS_LAUNCH((scan_chunk_states_kernel<false, CHANNEL>), dim3(sequences, heads, (elements + 127) / 128), 128, 0, s, A, elements);
+    SCAN_LAUNCH(SCAN_FINAL, dim3(sequences, heads * A.slices, A.max_chunks));
+#undef SCAN_LAUNCH
+    MRS_RETURN_LAUNCH_STATUS();
 }
 
 // q, k, v: pointers to the columns of the first head in float32 rows of `stride` floats.  `chunk_len` 0: in one go.
@@ -646,52 +863,66 @@ MRS_EXPORT int mrs_linear_scan(const float* q, const float* k, const float* v, i
     A.q = q, A.k = k, A.v = v, A.stride = stride, A.decay = decay, A.coef = decay ? nullptr : coef, A.coef_stride = coef_stride;
     A.state = state, A.norm_state = norm_state, A.state_stride = state_stride;
     A.positions = positions, A.q_start = q_start, A.state_slots = state_slots, A.out = out, A.norm_out = norm_out;
-    A.heads = heads, A.d = d, A.e = e, A.cols = cols, A.slices = slices, A.write_state = write_state;
+    A.heads = heads, A.d = d, A.e = e, A.cols = cols, A.slices = slices, A.write_state = write_state, A.chunk_len = chunk_len;
     A.vec_qk = d % 4 == 0 && stride % 4 == 0 && (((uintptr_t)q | (uintptr_t)k) & 15) == 0;
     A.vec_v = e % 4 == 0 && stride % 4 == 0 && ((uintptr_t)v & 15) == 0;
     A.vec_out = e % 4 == 0 && ((uintptr_t)out & 15) == 0;
-    const int token_floats = 2 * parts * SCAN_PITCH + cols;
-    int batch = (40 * 1024) / (2 * token_floats * (int)sizeof(float));
-    if (batch > SCAN_BATCH) batch = SCAN_BATCH;
+    A.vec_state = e % 4 == 0 && state_stride % 4 == 0 && ((uintptr_t)state & 15) == 0;
+    if (chunk_len == 0 && d <= 256 && tokens < 4LL * sequences) {
+        const int columns = norm_state ? (e + 3) / 4 * 4 + 4 : e;
+        MRS_LAUNCH((linear_step_kernel<false, float>), dim3(sequences, heads, (columns + STEP_COLUMNS - 1) / STEP_COLUMNS),
+                   (d + SCAN_ROWS - 1) / SCAN_ROWS * 32, 0, s, A);
+        MRS_RETURN_LAUNCH_STATUS();
+    }
+    int batch = scan_batch(parts, cols, false);
     if (tokens < SCAN_BATCH * sequences && batch > (tokens + sequences - 1) / sequences) batch = (tokens + sequences - 1) / sequences;
     if (batch < 1) return MRS_BAD_ARGUMENT;
     A.batch = batch;
-    const int threads = cols / (4 * (32 / parts)) * 32;
-    const size_t smem = 2 * (size_t)batch * token_floats * sizeof(float);
-#define SCAN_LAUNCH(MODE, GRID)                                                                          \
-    switch (parts) {                                                                                     \
-        case 1: MRS_LAUNCH((linear_scan_kernel<MODE, 1>), GRID, threads, smem, s, A); break;             \
-        case 2: MRS_LAUNCH((linear_scan_kernel<MODE, 2>), GRID, threads, smem, s, A); break;             \
-        case 4: MRS_LAUNCH((linear_scan_kernel<MODE, 4>), GRID, threads, smem, s, A); break;             \
-        case 8: MRS_LAUNCH((linear_scan_kernel<MODE, 8>), GRID, threads, smem, s, A); break;             \
-        case 16: MRS_LAUNCH((linear_scan_kernel<MODE, 16>), GRID, threads, smem, s, A); break;           \
-        default: MRS_LAUNCH((linear_scan_kernel<MODE, 32>), GRID, threads, smem, s, A); break;           \
-    }
-    if (chunk_len == 0) {
-        A.vec_state = e % 4 == 0 && state_stride % 4 == 0 && ((uintptr_t)state & 15) == 0;
-        if (d <= 256 && tokens < 4LL * sequences) {
-            const int columns = norm_state ? (e + 3) / 4 * 4 + 4 : e;
-            MRS_LAUNCH(linear_step_kernel, dim3(sequences, heads, (columns + STEP_COLUMNS - 1) / STEP_COLUMNS),
-                       (d + SCAN_ROWS - 1) / SCAN_ROWS * 32, 0, s, A);
-            MRS_RETURN_LAUNCH_STATUS();
-        }
-        SCAN_LAUNCH(SCAN_WHOLE, dim3(sequences, heads * slices));
+    return scan_run<false>(A, tokens, sequences, parts, scratch, s);
+}
+
+// The recurrence with keeps a key channel, made here: sigmoid(up low + bias)^(inverse_tau), `low` pointing to `rank` columns of the
+// rows that hold q, k and v, `up` [heads * d, rank] in float32 or bfloat16, `bias` [heads * d].  In portions q and k are changed in
+// place; `keeps` [tokens, heads * d] and `direct` [tokens, heads] are scratch.  A run in chunks wants chunks of a multiple of
+// mrs_channel_scan_batch rows.
+MRS_EXPORT int mrs_channel_scan(float* q, float* k, const float* v, int stride, const float* low, int rank, const void* up, int up_is_bf16,
+                                const float* bias, float inverse_tau, float* keeps, int* direct, float* state, long long state_stride,
+                                const int* positions, const int* seq_of_token, const int* q_start, const int* state_slots, float* out,
+                                int tokens, int sequences, int heads, int d, int e, int write_state, int chunk_len, float* scratch, void* s) {
+    if (tokens <= 0 || sequences <= 0) return 0;
+    if (heads <= 0 || d <= 0 || d > 512 || e <= 0 || rank <= 0 || rank > 1024 || chunk_len < 0 || (chunk_len > 0 && !scratch) || !up || !bias ||
+        !keeps || !direct || !(inverse_tau > 0.0f) || ((uintptr_t)scratch & 15))
+        return MRS_BAD_ARGUMENT;
+    ScanArgs A = {};
+    int parts, cols;
+    const int slices = scan_shape(d, e, false, &parts, &cols);
+    if ((long long)heads * slices > 65535) return MRS_BAD_ARGUMENT;
+    A.q = q, A.k = k, A.v = v, A.stride = stride, A.low = low, A.rank = rank, A.up = up, A.keep_bias = bias, A.inverse_tau = inverse_tau;
+    A.keeps = keeps, A.direct = direct, A.state = state, A.state_stride = state_stride;
+    A.positions = positions, A.q_start = q_start, A.state_slots = state_slots, A.out = out;
+    A.heads = heads, A.d = d, A.e = e, A.cols = cols, A.slices = slices, A.write_state = write_state, A.chunk_len = chunk_len;
+    A.vec_qk = d % 4 == 0 && stride % 4 == 0 && (((uintptr_t)q | (uintptr_t)k) & 15) == 0;
+    A.vec_v = e % 4 == 0 && stride % 4 == 0 && ((uintptr_t)v & 15) == 0;
+    A.vec_out = e % 4 == 0 && ((uintptr_t)out & 15) == 0;
+    A.vec_state = e % 4 == 0 && state_stride % 4 == 0 && ((uintptr_t)state & 15) == 0;
+    A.vec_keeps = d % 4 == 0 && ((uintptr_t)keeps & 15) == 0;
+    if (chunk_len == 0 && d <= 256 && tokens < 4LL * sequences) {
+        const dim3 grid(sequences, heads, (e + STEP_COLUMNS - 1) / STEP_COLUMNS);
+        const int threads = (d + SCAN_ROWS - 1) / SCAN_ROWS * 32;
+        if (up_is_bf16) MRS_LAUNCH((linear_step_kernel<true, bf16>), grid, threads, 0, s, A);
+        else MRS_LAUNCH((linear_step_kernel<true, float>), grid, threads, 0, s, A);
         MRS_RETURN_LAUNCH_STATUS();
     }
-    A.chunk_len = chunk_len;
-    A.max_chunks = (tokens + chunk_len - 1) / chunk_len;
-    if (A.max_chunks > 65535) return MRS_BAD_ARGUMENT;
-    const int elements = d * e + (norm_state ? d : 0);
-    A.chunk_floats = (elements + 3) / 4 * 4;
-    A.chunk_state = scratch;
-    A.chunk_decay = scratch + (size_t)sequences * heads * A.max_chunks * A.chunk_floats;
-    A.vec_state = e % 4 == 0;
-    SCAN_LAUNCH(SCAN_LOCAL, dim3(sequences, heads * slices, A.max_chunks));
-    if (d * e % 4 == 0 && elements % 4 == 0 && A.vec_state)
-        MRS_LAUNCH(scan_chunk_states_kernel<true>, dim3(sequences, heads, (elements / 4 + 127) / 128), 128, 0, s, A, elements);
-    else
-        MRS_LAUNCH(scan_chunk_states_kernel<false>, dim3(sequences, heads, (elements + 127) / 128), 128, 0, s, A, elements);
-    SCAN_LAUNCH(SCAN_FINAL, dim3(sequences, heads * slices, A.max_chunks));
-#undef SCAN_LAUNCH
-    MRS_RETURN_LAUNCH_STATUS();
+    A.batch = scan_batch(parts, cols, true);
+    if (A.batch < 1 || chunk_len % A.batch) return MRS_BAD_ARGUMENT;
+    int heads_a_block = 256 / d;
+    if (heads_a_block < 1) heads_a_block = 1;
+    if (heads_a_block > 32) heads_a_block = 32;
+    if (heads_a_block > heads) heads_a_block = heads;
+    const dim3 grid((tokens + A.batch - 1) / A.batch, (heads + heads_a_block - 1) / heads_a_block);
+    const int threads = (heads_a_block * d + 31) / 32 * 32;
+    const size_t smem = (size_t)A.batch * rank * sizeof(float);
+    if (up_is_bf16) MRS_LAUNCH(channel_fold_kernel<bf16>, grid, threads, smem, s, A, q, k, seq_of_token, tokens, heads_a_block);
+    else MRS_LAUNCH(channel_fold_kernel<float>, grid, threads, smem, s, A, q, k, seq_of_token, tokens, heads_a_block);
+    return scan_run<true>(A, tokens, sequences, parts, scratch, s);
 }

@@ -5,7 +5,8 @@
 //     pair (u, v) becomes (u cos a - v sin a, v cos a + u sin a), a = position * f_i; cosines and sines come from
 //     the step's table [tokens, rot / 2, 2] (float32); rot = 0: no rotation;
 //   * the norm x / sqrt(mean(x^2) + eps) over the whole head, with a weight of the head's size (one for all query
-//     heads, one for all key heads) or without one; before the rotation, after it, or not at all;
+//     heads, one for all key heads) or without one; before the rotation, after it, or not at all; or over the whole
+//     projection (all query heads at once, all key heads at once; weights of that size) before the rotation;
 //   * the values: columns of their own, or the key heads as they were projected (before norm and rotation).
 // Columns behind q, k and v (gates) are left to whoever reads them.  Key pages [pages, nkv, page, d], value pages
 // [pages, nkv, page, e]; slot < 0 writes nothing.  One warp a head; the head waits in shared memory as float32.  Heads of a
@@ -23,6 +24,16 @@ __device__ __forceinline__ void head_norm(float* x, int d, const float* w, float
     const float scale = 1.0f / sqrtf(warp_sum(sum) / (float)d + eps);
     for (int i = lane; i < d; i += 32) x[i] = w ? x[i] * scale * w[i] : x[i] * scale;
     __syncwarp();
+}
+
+// norm_mode: 0 none, 1 a head before the rotation, 2 a head after it, 3 the whole projection before it.
+// What the elements of q (and of k) are multiplied by when the norm is over all of them; the whole block takes part.
+__device__ __forceinline__ float2 projection_scales(const float* row, int qw, int kw, float eps, float* scratch) {
+    float q = 0.0f, k = 0.0f;
+    for (int i = threadIdx.x; i < qw; i += blockDim.x) q += row[i] * row[i];
+    for (int i = threadIdx.x; i < kw; i += blockDim.x) k += row[qw + i] * row[qw + i];
+    const float q_sum = block_sum(q, scratch), k_sum = block_sum(k, scratch);
+    return make_float2(1.0f / sqrtf(q_sum / (float)qw + eps), 1.0f / sqrtf(k_sum / (float)kw + eps));
 }
 
 template <typename T> __device__ __forceinline__ void put4(T* p, float4 v);
@@ -64,6 +75,8 @@ qkv_rotary_store_kernel(const float* __restrict__ proj, int proj_stride, const f
     const int half = rot / 2;
     const float* turn = rotations ? rotations + t * (size_t)half * 2 : nullptr;
     const int units = nq + nkv + (values_from_keys ? 0 : nkv);
+    __shared__ float scratch[33];
+    const float2 whole = norm_mode == 3 ? projection_scales(row, qw, kw, eps, scratch) : make_float2(1.0f, 1.0f);
     for (int unit = warp; unit < units; unit += ROTARY_WARPS) {
         if (unit >= nq + nkv) {                              // a value head with columns of its own
             if (!store || !v_cache) continue;
@@ -87,6 +100,11 @@ qkv_rotary_store_kernel(const float* __restrict__ proj, int proj_stride, const f
             copy_out<T, VEC>(v_cache + (((size_t)page * nkv + head) * page_size + in_page) * d, x, d, lane);
         const float* w = is_q ? q_norm : k_norm;
         if (norm_mode == 1) head_norm(x, d, w, eps, lane);
+        if (norm_mode == 3) {
+            const float scale = is_q ? whole.x : whole.y;
+            for (int i = lane; i < d; i += 32) x[i] = w ? x[i] * scale * w[head * d + i] : x[i] * scale;
+            __syncwarp();
+        }
         if (turn) {
             for (int i = lane; i < half; i += 32) {
                 const int a = interleaved ? 2 * i : i, b = interleaved ? 2 * i + 1 : i + half;
@@ -126,6 +144,8 @@ qkv_rotary_store_regs_kernel(const float* __restrict__ proj, int proj_stride, co
     const int units = nq + nkv + (values_from_keys ? 0 : nkv);
     const int at = 4 * lane;                                  // this lane's first element of a head
     const float4 zero = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    __shared__ float scratch[33];
+    const float2 whole = norm_mode == 3 ? projection_scales(row, qw, kw, eps, scratch) : make_float2(1.0f, 1.0f);
     for (int unit = warp; unit < units; unit += ROTARY_WARPS) {
         if (unit >= nq + nkv) {                              // a value head with columns of its own
             if (!store || !v_cache) continue;
@@ -142,9 +162,13 @@ qkv_rotary_store_regs_kernel(const float* __restrict__ proj, int proj_stride, co
         if (!is_q && values_from_keys && v_cache && mine)    // the value is the key as projected
             put4<T>(v_cache + (((size_t)page * nkv + head) * page_size + in_page) * d + at, x);
         const float* w = is_q ? q_norm : k_norm;
-        const float4 wv = (w && mine && norm_mode) ? *reinterpret_cast<const float4*>(w + at) : make_float4(1.0f, 1.0f, 1.0f, 1.0f);
+        const float4 wv = (w && mine && norm_mode) ? *reinterpret_cast<const float4*>(w + (norm_mode == 3 ? head * d : 0) + at) : make_float4(1.0f, 1.0f, 1.0f, 1.0f);
         if (norm_mode == 1) {
             const float scale = 1.0f / sqrtf(warp_sum(x.x * x.x + x.y * x.y + x.z * x.z + x.w * x.w) / (float)d + eps);
+            x = make_float4(x.x * scale * wv.x, x.y * scale * wv.y, x.z * scale * wv.z, x.w * scale * wv.w);
+        }
+        if (norm_mode == 3) {
+            const float scale = is_q ? whole.x : whole.y;
             x = make_float4(x.x * scale * wv.x, x.y * scale * wv.y, x.z * scale * wv.z, x.w * scale * wv.w);
         }
         if (turn) {
@@ -191,7 +215,7 @@ MRS_EXPORT int mrs_qkv_rotary_store(int is_bf16, const float* proj, int proj_str
                                     void* k_cache, void* v_cache, const int* slots, int tokens, int nq, int nkv, int d, int e,
                                     int page_size, int values_from_keys, void* s) {
     if (tokens <= 0) return 0;
-    if (nq <= 0 || nkv <= 0 || d <= 0 || d > ROTARY_MAX_D || e <= 0 || page_size <= 0 || norm_mode < 0 || norm_mode > 2 || rot < 0 ||
+    if (nq <= 0 || nkv <= 0 || d <= 0 || d > ROTARY_MAX_D || e <= 0 || page_size <= 0 || norm_mode < 0 || norm_mode > 3 || rot < 0 ||
         rot > d || rot % 2 || (rot > 0 && !rotations) || (values_from_keys && e != d) ||
         proj_stride < nq * d + nkv * d + (values_from_keys ? 0 : nkv * e))
         return MRS_BAD_ARGUMENT;

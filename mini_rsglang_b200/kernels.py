@@ -24,7 +24,7 @@ _SIGNATURES = {
     "mrs_rmsnorm": [_c_int, _c_vp, _c_vp, _c_float, _c_vp, _c_int, _c_int, _c_vp],
     "mrs_qk_norm_rope_store": [_c_int, _c_vp, _c_vp, _c_vp, _c_vp, _c_vp, _c_vp, _c_vp, _c_vp, _c_float, _c_vp, _c_vp,
                                _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_vp],
-    "mrs_rotation_table": [_c_vp, _c_vp, _c_int, _c_int, _c_vp, _c_vp],
+    "mrs_rotation_table": [_c_vp, _c_vp, _c_int, _c_int, _c_float, _c_vp, _c_vp],
     "mrs_silu_mul": [_c_int, _c_vp, _c_vp, _c_int, _c_int, _c_int, _c_vp],
     "mrs_attention_simt": [_c_int, _c_vp, _c_vp, _c_vp, _c_vp, _c_vp, _c_vp, _c_vp, _c_int, _c_int, _c_int, _c_int,
                            _c_int, _c_int, _c_float, _c_int, _c_vp],
@@ -175,15 +175,15 @@ def rmsnorm(x: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor
                                  x.numel() // width, width, _stream()), "rmsnorm")
 
 
-def rotation_table(positions: torch.Tensor, inv_freq: torch.Tensor) -> torch.Tensor:
-    """[tokens, d / 2, 2] float32: (cos, sin) of position * inv_freq, computed once a step for every layer that
-    rotates by the same frequencies."""
+def rotation_table(positions: torch.Tensor, inv_freq: torch.Tensor, magnitude: float = 1.0) -> torch.Tensor:
+    """[tokens, d / 2, 2] float32: (cos, sin) of position * inv_freq, both times `magnitude`, computed once a step for every
+    layer that rotates by the same frequencies."""
     tokens, half = positions.shape[0], inv_freq.shape[0]
     _need(positions, torch.int32, "positions", (tokens,))
     _need(inv_freq, torch.float32, "inv_freq", (half,))
     out = torch.empty((tokens, half, 2), dtype=torch.float32, device=positions.device)
-    _check(library().mrs_rotation_table(positions.data_ptr(), inv_freq.data_ptr(), tokens, half, out.data_ptr(), _stream()),
-           "rotation_table")
+    _check(library().mrs_rotation_table(positions.data_ptr(), inv_freq.data_ptr(), tokens, half, float(magnitude), out.data_ptr(),
+                                        _stream()), "rotation_table")
     return out
 
 
@@ -1370,7 +1370,8 @@ def attention_biased_mma_library(d: int, e: int, values_in_keys: bool = False) -
             defines["MRS_VALUES_IN_KEYS"] = 1
         lib = specialised_kernel_library("attention_biased_mma.cu", defines)
         lib.mrs_attention_biased_mma.argtypes = [_c_int] + [_c_vp] * 5 + [_c_int, _c_vp, _c_int, _c_vp, _c_vp, _c_int, _c_vp, _c_int,
-                                                 _c_int, _c_int, _c_float, _c_float, _c_int, _c_int, _c_int, _c_int, _c_vp, _c_vp, _c_int, _c_vp]
+                                                 _c_int, _c_int, _c_float, _c_float, _c_int, _c_int, _c_int, _c_int, _c_vp, _c_vp, _c_int, _c_int,
+                                                 _c_vp]
         lib.mrs_attention_biased_mma.restype = _c_int
         lib.mrs_attention_biased_mma_scratch_floats.argtypes = [_c_int, _c_int, _c_int]
         lib.mrs_attention_biased_mma_scratch_floats.restype = ctypes.c_longlong
@@ -1385,7 +1386,8 @@ def attention_biased_mma(q, k_cache, v_cache, positions, block_table, tiles, out
     """`attention_biased_simt`'s formulas on the tensor cores, bfloat16, over a list of tiles (sequence, first row, tokens, 0):
     `narrow` tiles hold up to 16 // (nq // nkv) tokens (decoded tokens, short portions), the others up to 64 // (nq // nkv).
     `splits` > 1 (narrow tiles): that many CTAs share a tile's key blocks and a second kernel merges them.
-    `v_cache` None: the values are the first `e` elements of the key rows."""
+    `v_cache` None: the values are the first `e` elements of the key rows.  `sink_logits` may have a multiple m of nq elements
+    where a token's m * nq heads come as m rows, row t's heads then being (t mod m) * nq and on."""
     global launch_count
     tokens = q.shape[0]
     _need(q, torch.bfloat16, "q", (tokens, nq * d))
@@ -1408,7 +1410,9 @@ def attention_biased_mma(q, k_cache, v_cache, positions, block_table, tiles, out
     if gate is not None:
         _need(gate, torch.float32, "attention gate", (tokens, nq))
     if sink_logits is not None:
-        _need(sink_logits, torch.float32, "sink logits", (nq,))
+        _need(sink_logits, torch.float32, "sink logits")
+        if sink_logits.dim() != 1 or sink_logits.shape[0] % nq or not sink_logits.shape[0]:
+            raise InvalidRequest("attention: one sink logit a query head")
     lib = attention_biased_mma_library(d, e, values_in_keys=v_cache is None)
     scratch = None
     if splits > 1:
@@ -1420,7 +1424,8 @@ def attention_biased_mma(q, k_cache, v_cache, positions, block_table, tiles, out
                                         block_table.data_ptr(), block_table.shape[1], tiles.data_ptr(), tiles.shape[0], out.data_ptr(),
                                         _ptr(bias), bias.shape[0] if bias is not None else 0, _ptr(gate), nq, nkv, page_size,
                                         float(scale), float(cap), int(window), int(keep_first), int(sink or sink_logits is not None),
-                                        int(splits), _ptr(scratch), _ptr(sink_logits), int(chunk), _stream()),
+                                        int(splits), _ptr(scratch), _ptr(sink_logits), sink_logits.shape[0] if sink_logits is not None else 0,
+                                        int(chunk), _stream()),
            "attention_biased_mma")
 
 
@@ -1428,15 +1433,16 @@ def attention_biased_mma(q, k_cache, v_cache, positions, block_table, tiles, out
 # layer norms with bias, latent attention, routed experts
 # ------------------------------------------------------------------------------------------------
 _LATENT_SIGNATURES = {
-    "mrs_add_layernorm": [_c_int, _c_vp, _c_vp, _c_vp, _c_vp, _c_float, _c_vp, _c_vp, _c_int, _c_int, _c_int, _c_vp],
+    "mrs_add_layernorm": [_c_int, _c_vp, _c_vp, _c_int, _c_float, _c_vp, _c_vp, _c_vp, _c_vp, _c_float, _c_vp, _c_vp, _c_int, _c_int, _c_int,
+                          _c_vp],
     "mrs_latent_prepare": [_c_int, _c_vp, _c_int, _c_vp, _c_float, _c_vp, _c_float, _c_vp, _c_vp, _c_vp, _c_vp, _c_vp, _c_vp] +
-                          [_c_int] * 8 + [_c_vp],
+                          [_c_int] * 9 + [_c_vp],
     "mrs_latent_norms": [_c_int, _c_vp, _c_int, _c_vp, _c_vp, _c_float, _c_vp, _c_vp, _c_vp, _c_int, _c_int, _c_int, _c_vp],
     "mrs_sigmoid_gate_mul": [_c_int, _c_vp, _c_vp, _c_int, _c_int, _c_int, _c_vp],
     "mrs_scale": [_c_vp, ctypes.c_longlong, _c_float, _c_vp],
 }
 _EXPERT_SIGNATURES = {
-    "mrs_moe_route": [_c_vp, _c_int, _c_vp, _c_vp, _c_vp, _c_vp, _c_int, _c_int, _c_int, _c_float, _c_int, _c_int, _c_int, _c_vp],
+    "mrs_moe_route": [_c_vp, _c_int, _c_vp, _c_vp, _c_vp, _c_vp, _c_vp, _c_int, _c_int, _c_int, _c_float, _c_int, _c_int, _c_int, _c_vp],
     "mrs_moe_align": [_c_vp, _c_int, _c_int, _c_int, _c_vp, _c_vp, _c_int, _c_vp],
     "mrs_moe_product_simt": [_c_int, _c_int, _c_vp, _c_vp, _c_vp, _c_vp, _c_vp, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_vp],
     "mrs_moe_product_rows": [_c_int, _c_int, _c_vp, _c_vp, _c_vp, _c_vp, _c_vp, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_vp],
@@ -1486,9 +1492,11 @@ def expert_library() -> ctypes.CDLL:
 
 
 def add_layernorm(residual: torch.Tensor, delta: torch.Tensor | None, weight: torch.Tensor, bias: torch.Tensor, eps: float,
-                  out: torch.Tensor, rows: torch.Tensor | None = None, write_back: bool = True) -> None:
-    """v = residual (+ delta); residual = v when write_back; out = (v - mean) / sqrt(var + eps) * weight + bias.
-    With `rows`, out[i] comes from source row rows[i]."""
+                  out: torch.Tensor, rows: torch.Tensor | None = None, write_back: bool = True, factor: float = 1.0,
+                  extra: torch.Tensor | None = None, row: torch.Tensor | None = None) -> None:
+    """v = residual (+ factor * delta) (+ extra) (+ row); residual = v when write_back; out = (v - mean) / sqrt(var + eps) *
+    weight + bias.  delta has out's dtype or is float32, extra is float32, both of the residual's shape; row float32 [width]
+    goes to every row.  With `rows`, out[i] comes from source row rows[i]."""
     n_rows, width = out.shape
     _need(residual, torch.float32, "add_layernorm residual")
     _need(weight, torch.float32, "add_layernorm weight", (width,))
@@ -1497,13 +1505,18 @@ def add_layernorm(residual: torch.Tensor, delta: torch.Tensor | None, weight: to
     if residual.shape[1] != width:
         raise InvalidRequest("add_layernorm: width mismatch")
     if delta is not None:
-        _need(delta, out.dtype, "add_layernorm delta", tuple(residual.shape))
+        _need(delta, out.dtype if delta.dtype is not torch.float32 else torch.float32, "add_layernorm delta", tuple(residual.shape))
+    if extra is not None:
+        _need(extra, torch.float32, "add_layernorm second branch", tuple(residual.shape))
+    if row is not None:
+        _need(row, torch.float32, "add_layernorm row", (width,))
     if rows is not None:
         _need(rows, torch.int32, "add_layernorm rows", (n_rows,))
     elif residual.shape[0] != n_rows:
         raise InvalidRequest("add_layernorm: row count mismatch")
-    _check(latent_library().mrs_add_layernorm(_is_bf16(out.dtype), residual.data_ptr(), _ptr(delta), weight.data_ptr(), bias.data_ptr(),
-                                              float(eps), out.data_ptr(), _ptr(rows), n_rows, width, int(write_back), _stream()),
+    _check(latent_library().mrs_add_layernorm(_is_bf16(out.dtype), residual.data_ptr(), _ptr(delta),
+                                              int(delta is not None and delta.dtype is torch.float32), float(factor), _ptr(extra), _ptr(row),
+                                              weight.data_ptr(), bias.data_ptr(), float(eps), out.data_ptr(), _ptr(rows), n_rows, width, int(write_back), _stream()),
            "add_layernorm")
 
 
@@ -1516,13 +1529,16 @@ def scale_(x: torch.Tensor, factor: float) -> None:
 def latent_prepare(proj: torch.Tensor, latent_weight: torch.Tensor | None, eps: float, inv_freq: torch.Tensor | None, magnitude: float,
                    positions: torch.Tensor, slots: torch.Tensor | None, q_plain: torch.Tensor, q_rows: torch.Tensor,
                    cache: torch.Tensor | None, gate: torch.Tensor | None, heads: int, plain: int, rotated: int, latent: int,
-                   rotary: int, has_latent: bool) -> None:
+                   rotary: int, has_latent: bool, pairing: str = "split_half") -> None:
     """After the fused float32 projection q | (latent, rotated key part) | (one gate a head) of a latent attention:
     `q_plain` [heads, tokens, plain] gets the unrotated query parts, the last `rotated` columns of `q_rows`
     [tokens, heads, latent + rotated] the rotated ones; with `has_latent`, the latent over its root mean square times
     `latent_weight` and the rotated key part go into `cache` [pages, 1, page, latent + rotated] at `slots` (None, or a
     slot of -1: nowhere); `gate` [tokens, heads] float32 gets the sigmoids.  Of a rotated part the first `rotary`
-    elements turn, element i with i + rotary / 2, by position * inv_freq[i], cosines and sines times `magnitude`."""
+    elements turn, element i with i + rotary / 2 ("split_half") or 2 i with 2 i + 1 ("interleaved"), by position * inv_freq[i],
+    cosines and sines times `magnitude`."""
+    if pairing not in ("split_half", "interleaved"):
+        raise InvalidRequest(f"latent_prepare: unknown pairing {pairing!r}")
     tokens, width = proj.shape
     _need(proj, torch.float32, "latent projection")
     _need(q_plain, None, "q_plain", (heads, tokens, plain))
@@ -1542,7 +1558,7 @@ def latent_prepare(proj: torch.Tensor, latent_weight: torch.Tensor | None, eps: 
     _check(latent_library().mrs_latent_prepare(
         _is_bf16(q_plain.dtype), proj.data_ptr(), width, _ptr(latent_weight), float(eps), _ptr(inv_freq), float(magnitude),
         positions.data_ptr(), _ptr(slots) if cache is not None else None, q_plain.data_ptr(), q_rows.data_ptr(), _ptr(cache), _ptr(gate),
-        tokens, heads, plain, rotated, latent, rotary, int(has_latent), int(gate is not None), _stream()), "latent_prepare")
+        tokens, heads, plain, rotated, latent, rotary, int(pairing == "interleaved"), int(has_latent), int(gate is not None), _stream()), "latent_prepare")
 
 
 def latent_norms(proj: torch.Tensor, q_weight: torch.Tensor, latent_weight: torch.Tensor, eps: float, slots: torch.Tensor | None,
@@ -1581,22 +1597,25 @@ def sigmoid_gate_mul(x: torch.Tensor, gate: torch.Tensor) -> None:
 
 def moe_route(logits: torch.Tensor, correction: torch.Tensor | None, chosen: torch.Tensor, weights: torch.Tensor,
               shared_gate: torch.Tensor | None, experts: int, top: int, scale: float, sigmoid_scores: bool = False,
-              normalize: bool = True) -> None:
+              normalize: bool = True, bias: torch.Tensor | None = None) -> None:
     """Router logits float32 [tokens, experts (+ 1) or more] -> `chosen` [tokens, top] int32, the `top` experts with the
     largest score + correction, and `weights` [tokens, top] float32, score / (sum of the chosen + 1e-20) * scale; scores
     are the softmax (or the sigmoids) of the first `experts` columns.  With `shared_gate` [tokens] the column after them
-    is one more gate, whose sigmoid it gets.  Further columns are not read.  `normalize` False: the weights are score * scale."""
+    is one more gate, whose sigmoid it gets.  Further columns are not read.  `normalize` False: the weights are score * scale.
+    `bias` [experts] float32: added to the logits before anything else."""
     tokens = logits.shape[0]
     _need(logits, torch.float32, "router logits")
     if logits.dim() != 2 or logits.shape[1] < experts + (1 if shared_gate is not None else 0):
         raise InvalidRequest("moe_route: fewer logits a token than experts")
+    if bias is not None:
+        _need(bias, torch.float32, "router bias", (experts,))
     if correction is not None:
         _need(correction, torch.float32, "router correction", (experts,))
     _need(chosen, torch.int32, "chosen experts", (tokens, top))
     _need(weights, torch.float32, "expert weights", (tokens, top))
     if shared_gate is not None:
         _need(shared_gate, torch.float32, "shared gate", (tokens,))
-    _check(expert_library().mrs_moe_route(logits.data_ptr(), logits.shape[1], _ptr(correction), chosen.data_ptr(), weights.data_ptr(),
+    _check(expert_library().mrs_moe_route(logits.data_ptr(), logits.shape[1], _ptr(bias), _ptr(correction), chosen.data_ptr(), weights.data_ptr(),
                                           _ptr(shared_gate), tokens, experts, top, float(scale), int(sigmoid_scores),
                                           int(shared_gate is not None), int(normalize), _stream()), "moe_route")
 
@@ -2103,11 +2122,15 @@ _LINEAR_SCAN_SIGNATURES = {
     "mrs_memory_gates": [_c_vp, _c_int, _c_int, _c_int, _c_vp, _c_vp, _c_float, _c_vp, _c_ll, _c_vp, _c_vp, _c_vp, _c_vp, _c_int, _c_int,
                          _c_int, _c_int, _c_vp],
     "mrs_linear_scan_slices": [_c_int, _c_int, _c_int],
+    "mrs_channel_scan_batch": [_c_int, _c_int],
+    "mrs_channel_scan": [_c_vp, _c_vp, _c_vp, _c_int, _c_vp, _c_int, _c_vp, _c_int, _c_vp, _c_float, _c_vp, _c_vp, _c_vp, _c_ll, _c_vp, _c_vp,
+                         _c_vp, _c_vp, _c_vp, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_vp, _c_vp],
     "mrs_linear_scan": [_c_vp, _c_vp, _c_vp, _c_int, _c_vp, _c_vp, _c_int, _c_vp, _c_vp, _c_ll, _c_vp, _c_vp, _c_vp, _c_vp, _c_vp, _c_int,
                         _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_vp, _c_vp],
 }
 _linear_scan_lib = None
 LINEAR_SCAN_MAX_DIM = 512
+CHANNEL_SCAN_MAX_RANK = 1024
 
 
 def linear_scan_library() -> ctypes.CDLL:
@@ -2118,7 +2141,7 @@ def linear_scan_library() -> ctypes.CDLL:
         from .csrc.build import linear_scan_kernel_library
 
         lib = _typed(linear_scan_kernel_library(), _LINEAR_SCAN_SIGNATURES)
-        lib.mrs_linear_scan_scratch_floats.argtypes = [_c_int] * 7
+        lib.mrs_linear_scan_scratch_floats.argtypes = [_c_int] * 8
         lib.mrs_linear_scan_scratch_floats.restype = ctypes.c_longlong
         _linear_scan_lib = lib
     return _linear_scan_lib
@@ -2221,7 +2244,7 @@ def linear_scan(rows: torch.Tensor, q_offset: int, k_offset: int, v_offset: int,
         chunk_len = linear_scan_chunk_length(tokens, sequences, heads, d, e, lib.mrs_linear_scan_slices(d, e, int(norm_state is not None)), sm_count(rows.device))
     scratch = None
     if chunk_len:
-        need = lib.mrs_linear_scan_scratch_floats(tokens, sequences, heads, d, e, int(norm_state is not None), int(chunk_len))
+        need = lib.mrs_linear_scan_scratch_floats(tokens, sequences, heads, d, e, int(norm_state is not None), int(chunk_len), 0)
         scratch = attention_scratch(rows.device, need, lane=2)
         launch_count += 2
     base = rows.data_ptr()
@@ -2229,6 +2252,48 @@ def linear_scan(rows: torch.Tensor, q_offset: int, k_offset: int, v_offset: int,
                                coef.shape[1] if coef is not None else 0, state.data_ptr(), _ptr(norm_state), state.stride(0),
                                positions.data_ptr(), q_start.data_ptr(), state_slots.data_ptr(), out.data_ptr(), _ptr(norm_out), tokens,
                                sequences, heads, d, e, int(write_state), int(chunk_len), _ptr(scratch), _stream()), "linear_scan")
+
+
+def channel_scan(rows: torch.Tensor, q_offset: int, k_offset: int, v_offset: int, low_offset: int, up: torch.Tensor, bias: torch.Tensor,
+                 tau: float, state: torch.Tensor, positions, seq_of_token, q_start, state_slots, out: torch.Tensor, heads: int, d: int,
+                 e: int, write_state: bool = True, chunk_len: int | None = None) -> None:
+    """S_t = diag(a_t) S_(t-1) + k_t v_t^T, o_t = S_t^T q_t per (sequence, head), float32, with one decay a key channel,
+    a_t = sigmoid(up low_t + bias)^(1 / tau): q, k [heads * d], v [heads * e] and low [rank] are columns of the float32 `rows`
+    (q and k are changed in place), `up` [heads * d, rank] float32 or bfloat16, `bias` [heads * d] float32.  `state`
+    [slots, heads, d, e] float32 (a view: dense within a slot), zero where a sequence starts at position 0; `out`
+    [tokens, heads * e].  `chunk_len` as in `linear_scan` (rounded up to whole batches)."""
+    global launch_count
+    tokens, rank = rows.shape[0], up.shape[1]
+    _need(rows, torch.float32, "projection")
+    _need(up, None, "second thin product", (heads * d, rank))
+    _need(bias, torch.float32, "decay bias", (heads * d,))
+    if min(q_offset, k_offset, v_offset, low_offset) < 0 or max(q_offset, k_offset) + heads * d > rows.shape[1] or \
+            v_offset + heads * e > rows.shape[1] or low_offset + rank > rows.shape[1]:
+        raise InvalidRequest("channel_scan: q, k, v or the thin product lie outside the rows")
+    if not 0 < d <= LINEAR_SCAN_MAX_DIM or not 0 < rank <= CHANNEL_SCAN_MAX_RANK or not tau > 0:
+        raise InvalidRequest(f"channel_scan: query/key heads of up to {LINEAR_SCAN_MAX_DIM} elements, thin products of up to "
+                             f"{CHANNEL_SCAN_MAX_RANK} and a positive tau are built")
+    _check_matrix_state(state, heads, d, e, "channel_scan")
+    _need(out, torch.float32, "recurrence output", (tokens, heads * e))
+    _need(seq_of_token, torch.int32, "seq_of_token", (tokens,))
+    sequences = state_slots.shape[0]
+    lib = linear_scan_library()
+    if chunk_len is None:
+        chunk_len = linear_scan_chunk_length(tokens, sequences, heads, d, e, lib.mrs_linear_scan_slices(d, e, 0), sm_count(rows.device))
+    scratch = None
+    if chunk_len:
+        batch = lib.mrs_channel_scan_batch(d, e)
+        chunk_len = -(-int(chunk_len) // batch) * batch
+        scratch = attention_scratch(rows.device, lib.mrs_linear_scan_scratch_floats(tokens, sequences, heads, d, e, 0, chunk_len, 1), lane=2)
+    launch_count += 3 if chunk_len else int(tokens >= 4 * sequences or d > 256)
+    keeps = torch.empty((tokens, heads * d), dtype=torch.float32, device=rows.device)
+    direct = torch.empty((tokens, heads), dtype=torch.int32, device=rows.device)
+    base = rows.data_ptr()
+    _check(lib.mrs_channel_scan(base + 4 * q_offset, base + 4 * k_offset, base + 4 * v_offset, rows.shape[1], base + 4 * low_offset, rank,
+                                up.data_ptr(), _is_bf16(up.dtype), bias.data_ptr(), 1.0 / float(tau), keeps.data_ptr(), direct.data_ptr(),
+                                state.data_ptr(), state.stride(0), positions.data_ptr(), seq_of_token.data_ptr(), q_start.data_ptr(),
+                                state_slots.data_ptr(), out.data_ptr(), tokens, sequences, heads, d, e, int(write_state), int(chunk_len),
+                                _ptr(scratch), _stream()), "channel_scan")
 
 
 # ------------------------------------------------------------------------------------------------
@@ -2243,7 +2308,7 @@ _ROTARY_SIGNATURES = {
     "mrs_concat_rows": [_c_int, _c_vp, _c_vp, _c_vp, _c_int, _c_int, _c_vp],
 }
 _rotary_lib = None
-HEAD_NORM_PLACES = {None: 0, "before_rotation": 1, "after_rotation": 2}
+HEAD_NORM_PLACES = {None: 0, "before_rotation": 1, "after_rotation": 2, "whole_before_rotation": 3}
 ROTARY_MAX_HEAD = 256
 
 
@@ -2266,7 +2331,8 @@ def qkv_rotary_store(proj: torch.Tensor, q_out: torch.Tensor, k_cache: torch.Ten
     key head turn by the token's position (`rotations` [tokens, rotary_dim / 2, 2] float32 cosines and sines; `pairing`
     "split_half": element i with i + rotary_dim / 2, "interleaved": 2 i with 2 i + 1), the heads pass an RMS norm over all
     their elements `norm_place` the rotation ("before_rotation", "after_rotation", None: no norm) with `q_norm` / `k_norm`
-    [d] float32 or, where one is None, without a weight; q goes to `q_out`, k into the key pages [pages, nkv, page, d], v
+    [d] float32 or, where one is None, without a weight, or ("whole_before_rotation") one RMS norm over all of q and one over
+    all of k with weights of those sizes; q goes to `q_out`, k into the key pages [pages, nkv, page, d], v
     into the value pages [pages, nkv, page, e] at `slots`.  `values_from_keys`: the rows have no value columns, a value is
     its key head as projected (e = d).  Columns behind these are not read."""
     tokens = proj.shape[0]
@@ -2291,9 +2357,9 @@ def qkv_rotary_store(proj: torch.Tensor, q_out: torch.Tensor, k_cache: torch.Ten
         _need(slots, torch.int32, "slots", (tokens,))
     if rotary_dim:
         _need(rotations, torch.float32, "rotations", (tokens, rotary_dim // 2, 2))
-    for w in (q_norm, k_norm):
+    for w, heads in ((q_norm, nq), (k_norm, nkv)):
         if w is not None:
-            _need(w, torch.float32, "head norm weight", (d,))
+            _need(w, torch.float32, "head norm weight", (heads * d if norm_place == "whole_before_rotation" else d,))
     _check(rotary_library().mrs_qkv_rotary_store(
         _is_bf16(q_out.dtype), proj.data_ptr(), proj.shape[1], _ptr(q_norm), _ptr(k_norm), HEAD_NORM_PLACES[norm_place], float(norm_eps),
         _ptr(rotations) if rotary_dim else None, int(rotary_dim), int(pairing == "interleaved"), q_out.data_ptr(), _ptr(k_cache),

@@ -4,14 +4,12 @@ from __future__ import annotations
 
 import torch
 
-from ..parts.base import Runtime
+from ..parts.base import BranchSum, Normed, Prenormed, Runtime
 from .spec import ModelSpec
 
 
 def plain_or_none(pending):
     """A branch output that the stream does not hold yet, or None when it does (`Prenormed`) or there is none."""
-    from ..parts.base import Normed, Prenormed
-
     return None if isinstance(pending, (Prenormed, Normed)) else pending
 
 
@@ -83,15 +81,21 @@ class Model:
         pending = None
         order = self.spec.run_order
         # a stream entry reads the embedding's output; the stream itself is updated in place, so a copy is kept
-        origin = stream.clone() if any(e.enter is not None for e in order) else None
+        origin = stream.clone() if any(e.enter is not None and self.stream_entries[e.enter].reads_origin for e in order) else None
         for index, entry in enumerate(order):
             block = self.blocks[entry.layer]
             ctx.label = f"layer{index}"
             if entry.enter is not None:
                 delta = plain_or_none(pending)          # the block before was told of no following norm: the stream holds its sum
-                if delta is not None:
-                    stream.add_(delta.float())
-                stream, pending = self.stream_entries[entry.enter].forward(stream, origin, ctx), None
+                part = self.stream_entries[entry.enter]
+                if part.adds_only:                      # its terms join what the layer's first norm adds
+                    pending = part.join(delta, origin)
+                else:
+                    if isinstance(delta, BranchSum):
+                        stream = delta.add_to(stream)
+                    elif delta is not None:
+                        stream.add_(delta.float())
+                    stream, pending = part.forward(stream, origin, ctx), None
             extra = {}
             if block.links_norms:        # the norm that reads the stream after this block; none when something stands between
                 if index + 1 < len(order):

@@ -8,8 +8,9 @@ import os
 from dataclasses import dataclass
 from typing import Callable
 
-from ..config.model_config import MigenexConfig, ModelConfig, NiduvikConfig, NubipelConfig, PisatarConfig, Qwen3Config, SatedraConfig
+from ..config.model_config import BilipelConfig, MigenexConfig, ModelConfig, NiduvikConfig, NubipelConfig, PisatarConfig, Qwen3Config, SatedraConfig
 from ..errors import InvalidRequest
+from .bilipel import bilipel_spec
 from .migenex import migenex_spec
 from .niduvik import niduvik_spec
 from .nubipel import nubipel_spec
@@ -41,6 +42,7 @@ register_architecture("satedra", SatedraConfig, satedra_spec)
 register_architecture("nubipel", NubipelConfig, nubipel_spec)
 register_architecture("migenex", MigenexConfig, migenex_spec)
 register_architecture("pisatar", PisatarConfig, pisatar_spec)
+register_architecture("bilipel", BilipelConfig, bilipel_spec)
 
 
 def config_from_dict(raw: dict) -> ModelConfig:

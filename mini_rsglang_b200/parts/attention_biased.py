@@ -8,7 +8,8 @@
   * a sliding window that also keeps the first `keep_first` positions in sight (at their true distances); or sight in
     chunks: position i sees j <= i only where floor(i / chunk) = floor(j / chunk), chunks counted from position 0;
   * an RMS norm over every query and key head (one weight of the head's size for all query heads, one for all key heads,
-    or no weight);
+    or no weight), or over the whole query and the whole key projection before they are split into heads (a weight for every
+    row);
   * a rotation of query and key heads by their positions (any registered position encoding: all or part of a head, split
     halves or interleaved pairs), with the head norm before or after it;
   * values that are the key heads as projected (before norm and rotation): no value projection;
@@ -67,7 +68,7 @@ class BiasedWindowAttention(Mixer):
                  position: PartSpec | None = None, head_norm_place: str = "before_rotation", head_norm_weights: bool = True,
                  values_from_keys: bool = False, names: dict | None = None):
         """`position`: a position encoding that rotates query and key heads (None: none); `head_norm_place`: the head norm
-        stands "before_rotation" or "after_rotation"; `head_norm_weights` False: it has no weights.  `values_from_keys`: no
+        stands "before_rotation" or "after_rotation", or is one norm over the whole projection, "whole_before_rotation"; `head_norm_weights` False: it has no weights.  `values_from_keys`: no
         value projection, a value head is its key head as projected (`value_dim` = `head_dim`).  `output_gate`: True or
         "heads": one gate a (token, head); "elements": one a value element of every head.
         `chunk` > 0 (no window then): sight within the query's chunk of positions.  `sink_logits`: the sink's logit is a
@@ -104,13 +105,14 @@ class BiasedWindowAttention(Mixer):
         self.position = POSITION_ENCODINGS.build(position, prefix) if position is not None else None
         self.head_norm_place, self.head_norm_weights = head_norm_place, bool(head_norm_weights)
         self.values_from_keys = bool(values_from_keys)
-        if head_norm_place not in ("before_rotation", "after_rotation"):
-            raise InvalidRequest(f"{prefix}: a head norm stands before_rotation or after_rotation")
+        if head_norm_place not in ("before_rotation", "after_rotation", "whole_before_rotation"):
+            raise InvalidRequest(f"{prefix}: a head norm stands before_rotation, after_rotation or whole_before_rotation")
+        self.whole_norm = head_norm_place == "whole_before_rotation"
         if self.values_from_keys and self.e != self.d:
             raise InvalidRequest(f"{prefix}: values taken from the keys have the keys' size")
         # what only the kernel with rotations does, and what only the one with biases and blending does
         self.rotary_store = (self.position is not None or self.values_from_keys or not self.head_norm_weights
-                             or head_norm_place == "after_rotation" or self.output_gate == "elements")
+                             or head_norm_place != "before_rotation" or self.output_gate == "elements")
         if self.rotary_store and (projection_bias or value_mix or self.output_gate == "heads"):
             raise InvalidRequest(f"{prefix}: rotation, values from keys, weightless or late head norms and gates a value element "
                                  "are not built together with projection biases, blended values or gates a head")
@@ -148,7 +150,8 @@ class BiasedWindowAttention(Mixer):
         if self.output_gate:
             specs.append(WeightSpec(self.name(n["gate"]), (self.nq * (self.e if self.output_gate == "elements" else 1), self.width)))
         if self.head_norm_eps is not None and self.head_norm_weights:
-            specs += [WeightSpec(self.name(n["q_norm"]), (self.d,), "vector"), WeightSpec(self.name(n["k_norm"]), (self.d,), "vector")]
+            specs += [WeightSpec(self.name(n[key]), (heads * self.d if self.whole_norm else self.d,), "vector")
+                      for key, heads in (("q_norm", self.nq), ("k_norm", self.nkv))]
         if self.sink_logits:
             specs.append(WeightSpec(self.name(n["sink"]), (self.nq,), "bias"))
         return specs
@@ -207,8 +210,6 @@ class BiasedWindowAttention(Mixer):
             rotation = self.position.rotation() if self.position is not None else None
             if rotation is not None and rotation.rotary_dim == 0:
                 rotation = None
-            if rotation is not None and rotation.magnitude != 1.0:
-                raise InvalidRequest(f"{self.prefix}: stretched cosines and sines are not built for this attention")
             kernels.qkv_rotary_store(proj, q, cache.k if write_cache else None, cache.v if write_cache else None,
                                      ctx.slots[cache.group] if write_cache else None, self.nq, self.nkv, self.d, self.e,
                                      rotations=self.position.rotations(ctx) if rotation is not None else None,

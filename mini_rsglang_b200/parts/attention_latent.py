@@ -9,7 +9,8 @@ and a latent of R elements:
   k_head = W_uk[head] c  [d],  v_head = W_uv[head] c  [e]
   score(i, j) = (q_plain_i . k_head_j + q_rot_i . k_r_j) * scale,  softmax over the keys in sight (all earlier
   ones, or a sliding window), out_head = sum_j p_j v_head_j, times sigmoid(W_g h)_head where the layer gates,
-  then W_o over the concatenated heads.
+  then W_o over the concatenated heads.  With sinks the softmax has one more term in its denominator, exp of a learned
+  number a head (not scaled), which has no key and no value.
 
 The cache holds one row a token, [c | k_r] (`KVNeed.values = False`: no value pages), and the attention runs in the
 latent space, where every head reads the same rows: since q_plain . (W_uk c) = (W_uk^T q_plain) . c and
@@ -44,7 +45,7 @@ class LatentAttention(Mixer):
     def __init__(self, prefix: str, width: int, num_heads: int, head_dim: int, rotary_head_dim: int, value_dim: int,
                  latent_dim: int, scale: float, eps: float, position: PartSpec | None = None, window: int = 0,
                  cache_window: int | None = None, shares_cache: bool = False, output_gate: bool | str = False,
-                 query_latent_dim: int = 0, float32_out: bool = False,
+                 query_latent_dim: int = 0, float32_out: bool = False, sink_logits: bool = False,
                  names: dict | None = None):
         """`position`: the encoding of the rotated part (None: nothing turns).  `window` 0: every earlier key is seen.
         `cache_window`: the window that the cache is kept for, where other layers read this layer's cache with wider
@@ -52,7 +53,7 @@ class LatentAttention(Mixer):
         `output_gate`: False, True or "heads" (one gate a head), or "elements" (one a value element of every head).
         `query_latent_dim` > 0: the queries are made from a normed latent of that size.
         `float32_out`: the output projection hands on its float32 sums (for a residual sum that reads them).
-        `names`: leaves of the tensors below the part's root."""
+        `sink_logits`: a learned sink a head in the softmax.  `names`: leaves of the tensors below the part's root."""
         super().__init__(prefix)
         self.width, self.heads, self.d, self.r = int(width), int(num_heads), int(head_dim), int(rotary_head_dim)
         self.e, self.latent = int(value_dim), int(latent_dim)
@@ -68,7 +69,7 @@ class LatentAttention(Mixer):
             raise InvalidRequest(f"{prefix}: output_gate must be False, True, \"heads\" or \"elements\"")
         self.shares_cache, self.output_gate = bool(shares_cache), bool(output_gate)
         self.gate_elements = output_gate == "elements"
-        self.float32_out = bool(float32_out)
+        self.float32_out, self.sink_logits, self.sinks = bool(float32_out), bool(sink_logits), None
         self.query_latent = int(query_latent_dim)
         if self.query_latent < 0 or (self.query_latent and (self.r or self.shares_cache or position is not None)):
             raise InvalidRequest(f"{prefix}: queries from a latent together with a rotated part or a borrowed cache are not built")
@@ -77,7 +78,7 @@ class LatentAttention(Mixer):
         self.position = POSITION_ENCODINGS.build(position, prefix) if position is not None else None
         self.leaf = {"q": "q_proj.weight", "down": "kv_down_proj.weight", "latent_norm": "kv_norm.weight", "up_k": "k_up_proj.weight",
                      "up_v": "v_up_proj.weight", "gate": "gate_proj.weight", "o": "o_proj.weight", "q_down": "q_down_proj.weight",
-                     "q_norm": "q_norm.weight", "q_up": "q_up_proj.weight"}
+                     "q_norm": "q_norm.weight", "q_up": "q_up_proj.weight", "sink": "sinks"}
         self.leaf.update(names or {})
         self.fused = self.latent_weight = self.up_k = self.up_v = self.o = self.q_up = self.q_latent_weight = None
         self.rotation = None
@@ -103,6 +104,8 @@ class LatentAttention(Mixer):
                   WeightSpec(self.name(n["up_v"]), (self.heads * self.e, self.latent))]
         if self.output_gate:
             specs.append(WeightSpec(self.name(n["gate"]), (self.heads * self.e if self.gate_elements else self.heads, self.width)))
+        if self.sink_logits:
+            specs.append(WeightSpec(self.name(n["sink"]), (self.heads,), "bias"))
         specs.append(WeightSpec(self.name(n["o"]), (self.width, self.heads * self.e)))
         return specs
 
@@ -126,13 +129,14 @@ class LatentAttention(Mixer):
         self.up_k = tensors[self.name(n["up_k"])].contiguous().view(self.heads, self.d, self.latent)
         self.up_v = tensors[self.name(n["up_v"])].contiguous().view(self.heads, self.e, self.latent).transpose(1, 2)
         self.o = tensors[self.name(n["o"])].contiguous()
+        if self.sink_logits:
+            self.sinks = tensors[self.name(n["sink"])].float().contiguous()
         if self.position is not None:
             self.position.bind(tensors, runtime)
             self.rotation = self.position.rotation()
         if self.rotation is not None:
-            if self.rotation.pairing != "split_half" or self.rotation.rotary_dim > self.r or self.rotation.rotary_dim % 2:
-                raise InvalidRequest(f"{self.prefix}: the kernel turns an even number of the rotated part's first elements, "
-                                     "element i with i + half of them")
+            if self.rotation.rotary_dim > self.r or self.rotation.rotary_dim % 2:
+                raise InvalidRequest(f"{self.prefix}: the kernel turns an even number of the rotated part's first elements")
 
     def forward(self, h, ctx, cache, write_cache=True):
         tokens = h.shape[0]
@@ -155,7 +159,8 @@ class LatentAttention(Mixer):
             kernels.latent_prepare(proj, self.latent_weight, self.eps, rotation.inv_freq if rotation else None,
                                    rotation.magnitude if rotation else 1.0, ctx.positions, ctx.slots[cache.group] if keeps else None,
                                    q_plain, q_rows, cache.k if keeps else None, gate, H, self.d, self.r, R,
-                                   rotation.rotary_dim if rotation else 0, not self.shares_cache)
+                                   rotation.rotary_dim if rotation else 0, not self.shares_cache,
+                                   pairing=rotation.pairing if rotation else "split_half")
         # the queries in the latent space: q_rows[:, head, :R] = q_plain[head] . W_uk[head]
         torch.bmm(q_plain, self.up_k, out=q_rows[:, :, :R].transpose(0, 1))
         q_rows = q_rows.view(tokens, H * row)
@@ -165,7 +170,7 @@ class LatentAttention(Mixer):
         if not arguments:
             # the 32-bit path and sizes that the tensor-core kernel does not take: one warp a (token, head)
             kernels.attention_biased_simt(q_rows, cache.k, None, ctx.positions, ctx.seq_of_token, table, mixed, H, 1, row, R,
-                                          self.scale, window=self.window, gate=gate)
+                                          self.scale, window=self.window, gate=gate, sink_logits=self.sinks)
         else:
             narrow, wide, longest, _ = plan_attention_tiles(ctx, *arguments)
             few = kernels.MMA_ROWS_NARROW
@@ -179,7 +184,8 @@ class LatentAttention(Mixer):
                 splits = min(choose_splits(tiles.shape[0], 1, reach, arguments[5]), 16)
                 kernels.attention_biased_mma(q_rows.view(tokens * m, few * row), cache.k, None, positions, table, tiles,
                                              mixed.view(tokens * m, few * R), few, 1, row, R, self.scale, window=self.window,
-                                             gate=gate.view(tokens * m, few) if gate is not None else None, narrow=True, splits=splits)
+                                             gate=gate.view(tokens * m, few) if gate is not None else None, narrow=True, splits=splits,
+                                             sink_logits=self.sinks)
                 wide = None
             for tiles, is_narrow in ((narrow, True), (wide, False)):
                 if tiles is not None:
@@ -188,7 +194,7 @@ class LatentAttention(Mixer):
                         reach = min(longest, self.window) if self.window else longest
                         splits = min(choose_splits(tiles.shape[0], 1, reach, arguments[5]), 16)
                     kernels.attention_biased_mma(q_rows, cache.k, None, ctx.positions, table, tiles, mixed, H, 1, row, R, self.scale,
-                                                 window=self.window, gate=gate, narrow=is_narrow, splits=splits)
+                                                 window=self.window, gate=gate, narrow=is_narrow, splits=splits, sink_logits=self.sinks)
         # back to the heads' values: out[:, head] = mixed[:, head] . W_uv[head]^T
         out = torch.empty((tokens, H, self.e), dtype=dtype, device=device)
         torch.bmm(mixed.view(tokens, H, R).transpose(0, 1), self.up_v, out=out.transpose(0, 1))

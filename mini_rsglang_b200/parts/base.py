@@ -12,11 +12,11 @@ something new.
 Interfaces (all tensors on the device; `ctx` is an `engine.context.StepContext`):
   Norm.forward(x) -> y                             x, y [rows, width] of the engine's dtype
   Norm.add_norm(residual, delta, rows, write_back) -> y
-      residual float32 [T, width] (+ delta of the engine's dtype), normalised; the sum is
+      residual float32 [T, width] (+ delta of the engine's dtype, or a `BranchSum`), normalised; the sum is
       written back unless told otherwise; `rows` picks source rows
   Embedding.forward(ctx) -> stream                 float32 [T, width] from `ctx.token_ids`
   StreamEntry.forward(stream, origin, ctx) -> stream   before a run of a layer: the stream it reads, from the stream so far
-      and the embedding's output
+      and the embedding's output (an entry that only adds hands its terms to the norm that follows: `StreamEntry.join`)
   Head.forward(hidden) -> logits                   float32 [rows, vocab]; `hidden` may be a `Prenormed`
   PositionEncoding.rotation() -> Rotation | None   how the mixer's kernel rotates: frequencies, how many of the
       head's elements turn, which elements pair, a factor on cosines and sines; None: no rotation
@@ -179,10 +179,19 @@ class Normed:
 
 @dataclass
 class BranchSum:
-    """A mixer's output as a sum that nobody has formed yet: the terms [(float32 [T, width], factor)].  A block whose kernel adds
-    several branches to the stream takes it as it is (`Mixer.gives_terms`)."""
+    """A branch's output as a sum that nobody has formed yet: the terms [(float32 [T, width], factor)] and, if there is one, a
+    vector [width] for every row.  A block whose kernel adds several branches to the stream takes it as it is
+    (`Mixer.gives_terms`); every norm takes it as what is still to be added (`Norm.add_norm`)."""
 
     terms: list
+    row: torch.Tensor | None = None
+
+    def add_to(self, stream: torch.Tensor) -> torch.Tensor:
+        """The stream with the sum in it, as a tensor of its own (for whoever wants it without the norm that adds it)."""
+        out = stream.clone()
+        for x, factor in self.terms:
+            out.add_(x.float(), alpha=factor)
+        return out if self.row is None else out.add_(self.row)
 
 
 def observing(ctx) -> bool:
@@ -248,7 +257,15 @@ class Embedding(Part):
 
 class StreamEntry(Part):
     """What stands before a run of a layer and acts on the whole residual stream: `forward(stream, origin, ctx)` returns the
-    stream that the layer reads (float32 [T, width]); `origin` is the stream as the embedding left it."""
+    stream that the layer reads (float32 [T, width]); `origin` is the stream as the embedding left it (None where no entry of the
+    model says `reads_origin`).  An entry that only adds to the stream (`adds_only`) has `join(pending, origin)` instead: what is
+    still to be added, with its own terms, as the `BranchSum` that the layer's first norm adds."""
+
+    reads_origin = True
+    adds_only = False
+
+    def join(self, pending, origin: torch.Tensor | None) -> "BranchSum":
+        raise NotImplementedError
 
     def forward(self, stream: torch.Tensor, origin: torch.Tensor, ctx) -> torch.Tensor:
         raise NotImplementedError

@@ -1,5 +1,5 @@
 """How a layer's parts are arranged.  "pre_norm": x + mixer(norm1(x)), then
-+ feed_forward(norm2(.)) (reference: crates/models/src/qwen3.rs:176-225).  "sandwich_norm": a norm before and after
++ feed_forward(norm2(.)) (reference: crates/models/src/qwen3.rs:176-225), both branches times a constant if the layer says so.  "sandwich_norm": a norm before and after
 each branch.  "parallel": both branches read one norm's output, x + (mixer(norm1(x)) + feed_forward(norm1(x))).
 "parallel_two_norms": each branch reads a norm of its own, x + (mixer(norm1(x)) + feed_forward(norm2(x))).
 
@@ -13,7 +13,7 @@ import torch
 
 from .. import kernels
 from ..errors import InvalidRequest
-from .base import BLOCKS, FEED_FORWARDS, MIXERS, NORMS, Block, Normed, Prenormed, ResidualLink, observing, plain
+from .base import BLOCKS, FEED_FORWARDS, MIXERS, NORMS, Block, BranchSum, Normed, Prenormed, ResidualLink, observing, plain
 from .norm import NormPair
 
 
@@ -33,15 +33,25 @@ class PreNormBlock(Block):
     optional_roles = ("norm2", "feed_forward")       # a layer may be a mixer alone (both are left out together)
     entry_role = "norm1"
 
-    def __init__(self, prefix: str, **parts):
+    def __init__(self, prefix: str, branch_scale: float = 1.0, **parts):
+        """`branch_scale`: what both branches are multiplied by when they join the stream; the norm that adds them does it."""
         super().__init__(prefix, **parts)
+        self.branch_scale = float(branch_scale)
         if (self.norm2 is None) != (self.feed_forward is None):
             raise InvalidRequest(f"block at {prefix!r}: a feed-forward comes with the norm before it")
+
+    def _scaled(self, branch):
+        return BranchSum([(branch, self.branch_scale)])
 
     def forward(self, stream, pending, ctx, cache, write_cache=True, next_norm=None):
         if observing(ctx):
             return self.forward_observed(stream, pending, ctx, cache, write_cache)
         h = self.norm1.add_norm(stream, pending)
+        if self.branch_scale != 1.0:
+            a = self._scaled(self.mixer.forward(plain(h), ctx, cache, write_cache))
+            if self.feed_forward is None:
+                return a
+            return self._scaled(self.feed_forward.forward(plain(self.norm2.add_norm(stream, a)), ctx))
         if self.feed_forward is None:
             return _branch(self.mixer, h, stream, next_norm, ctx, cache, write_cache)
         a = _branch(self.mixer, h, stream, self.norm2, ctx, cache, write_cache)
@@ -53,13 +63,13 @@ class PreNormBlock(Block):
         (crates/models/src/qwen3.rs:177-226): input_norm here, the mixer's and feed-forward's inside them, output."""
         h = plain(self.norm1.add_norm(stream, pending))
         ctx.observe(f"{ctx.label}-input_norm", h)
-        a = self.mixer.forward(h, ctx, cache, write_cache)
+        a = self._scaled(self.mixer.forward(h, ctx, cache, write_cache))
         if self.feed_forward is None:
-            ctx.observe(f"{ctx.label}-output", stream + a.float())
+            ctx.observe(f"{ctx.label}-output", a.add_to(stream))
             return a
         h = plain(self.norm2.add_norm(stream, a))
-        f = self.feed_forward.forward(h, ctx)
-        ctx.observe(f"{ctx.label}-output", stream + f.float())
+        f = self._scaled(self.feed_forward.forward(h, ctx))
+        ctx.observe(f"{ctx.label}-output", f.add_to(stream))
         return f
 
 

@@ -6,7 +6,8 @@ their outputs (no biases anywhere).
   weight_e = s_e / (sum of the chosen s + 1e-20) * scale
   out = sum over the chosen of weight_e * expert_e(h),   expert_e(h) = W_down silu(W_gate h) * (W_up h)
 
-Variations, all parameters: `normalize` False leaves the weights as the chosen scores (times scale); `form` "plain" makes
+Variations, all parameters: `router_bias` adds a number an expert to the logits z (float32; normalised softmax scores are then the
+softmax over the chosen logits alone); `normalize` False leaves the weights as the chosen scores (times scale); `form` "plain" makes
 an expert W_down act(W_up h) without a gate, `activation` one of `kernels.ACTIVATIONS`; `weight_on` "input" multiplies what
 a chosen expert reads by its weight instead of what it returns: out = sum over the chosen of expert_e(weight_e * h).
 
@@ -33,7 +34,7 @@ class RoutedExperts(FeedForward):
     def __init__(self, prefix: str, width: int, experts: int, top: int, inner: int, identity: int = 0, scale: float = 1.0,
                  score: str = "softmax", correction: bool = False, shared: PartSpec | None = None, shared_gate: bool = False,
                  normalize: bool = True, form: str = "gated", activation: str = "silu", weight_on: str = "output",
-                 float32_out: bool = False, names: dict | None = None):
+                 float32_out: bool = False, router_bias: bool = False, names: dict | None = None):
         """`experts` with tensors, then `identity` without; `shared`: the feed-forward that every token passes as well
         (its root is the leaf "shared" below this part's), `shared_gate`: behind a sigmoid gate of one number a token.
         `names`: leaves below the part's root; "expert" is a pattern with `{}` for the expert's number."""
@@ -46,7 +47,7 @@ class RoutedExperts(FeedForward):
             raise InvalidRequest(f"{prefix}: sizes must be positive")
         if score not in ("softmax", "sigmoid"):
             raise InvalidRequest(f"{prefix}: router scores {score!r} are not built; softmax or sigmoid")
-        self.score, self.correction = score, bool(correction)
+        self.score, self.correction, self.router_bias = score, bool(correction), bool(router_bias)
         self.normalize, self.form, self.activation, self.weight_on = bool(normalize), form, activation, weight_on
         self.float32_out = bool(float32_out)       # the summed outputs leave as float32 (a float32 norm or sum reads them)
         if form not in ("gated", "plain") or weight_on not in ("output", "input"):
@@ -57,12 +58,12 @@ class RoutedExperts(FeedForward):
             raise InvalidRequest(f"{prefix}: activation {activation!r} is not built; known: {sorted(kernels.ACTIVATIONS)}")
         if weight_on == "input" and (form != "plain" or self.identity):
             raise InvalidRequest(f"{prefix}: weights on the experts' input are built for plain experts without identity experts")
-        self.leaf = {"router": "router.weight", "correction": "router.correction", "expert": "experts.{}", "gate": "gate_proj.weight",
+        self.leaf = {"router": "router.weight", "router_bias": "router.bias", "correction": "router.correction", "expert": "experts.{}", "gate": "gate_proj.weight",
                      "up": "up_proj.weight", "down": "down_proj.weight", "shared": "shared", "shared_gate": "shared_gate.weight"}
         self.leaf.update(names or {})
         self.shared = FEED_FORWARDS.build(shared, self.name(self.leaf["shared"])) if shared is not None else None
         self.shared_gate = bool(shared_gate) and self.shared is not None
-        self.router = self.correction_values = self.gate_up = self.down = None
+        self.router = self.router_bias_values = self.correction_values = self.gate_up = self.down = None
         self.block = 0
 
     @property
@@ -81,6 +82,8 @@ class RoutedExperts(FeedForward):
             specs += [WeightSpec(self._expert(number, "up"), (self.inner, self.width)),
                       WeightSpec(self._expert(number, "down"), (self.width, self.inner))]
         specs.append(WeightSpec(self.name(n["router"]), (self.all_experts, self.width)))
+        if self.router_bias:
+            specs.append(WeightSpec(self.name(n["router_bias"]), (self.all_experts,), "bias"))
         if self.correction:
             specs.append(WeightSpec(self.name(n["correction"]), (self.all_experts,), "bias"))
         if self.shared is not None:
@@ -117,6 +120,7 @@ class RoutedExperts(FeedForward):
         if count % 8:
             rows.append(torch.zeros((8 - count % 8, self.width), dtype=rows[0].dtype, device=rows[0].device))
         self.router = torch.cat(rows, dim=0).contiguous()
+        self.router_bias_values = tensors[self.name(n["router_bias"])] if self.router_bias else None
         self.correction_values = tensors[self.name(n["correction"])] if self.correction else None
         if self.shared is not None:
             self.shared.bind(tensors, runtime)
@@ -130,7 +134,7 @@ class RoutedExperts(FeedForward):
         weights = torch.empty((tokens, self.top), dtype=torch.float32, device=device)
         shared_gate = torch.empty((tokens,), dtype=torch.float32, device=device) if self.shared_gate else None
         kernels.moe_route(logits, self.correction_values, chosen, weights, shared_gate, self.all_experts, self.top, self.scale,
-                          sigmoid_scores=self.score == "sigmoid", normalize=self.normalize)
+                          sigmoid_scores=self.score == "sigmoid", normalize=self.normalize, bias=self.router_bias_values)
         on_input = self.weight_on == "input"
         y = None
         if self.experts:

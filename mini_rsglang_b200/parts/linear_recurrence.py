@@ -15,6 +15,12 @@ of d query/key and e value elements:
   o = S^T q / (max(|n . q|, exp(-m)) + floor_eps)
   out = W_o (o / rms(o) * w_norm * sigmoid(W_g h))                        rms over a head, w_norm of all heads' size
 
+"gated_linear_attention": one decay a key channel and token, which acts on the rows of S, from two thin products:
+
+  q = W_q h d^(-1/2), k = W_k h  [H, d];  v = W_v h  [H, e];  a = sigmoid(W_a2 (W_a1 h) + b)^(1 / tau)  [H, d]
+  S <- diag(a) S + k v^T;  o = S^T q
+  out = W_o (o / rms(o) * w_norm * silu(W_g h))                           rms over a head, w_norm of a head's size
+
 A request's state lives in its state slot as one float32 vector (S of every head, then n, then m) and counts as zero where a
 sequence starts at position 0.  One projection gives everything that is read of h as float32 sums; rotation, gates, maxima,
 recurrence and head norm are float32 (`kernels.linear_scan`; the factors d^(-1/2) are applied to the read-out, which is linear
@@ -156,4 +162,50 @@ class MatrixMemory(LinearRecurrence):
         normed = torch.empty((tokens, H * e), dtype=self.runtime.dtype, device=device)
         kernels.head_norm_gate(o, proj[:, g_at:i_at], self.norm_w, self.eps, normed, H, gate_kind="sigmoid", factor=d ** -0.5,
                                normaliser=(c, coef[:, 2 * H:], self.floor_eps))
+        return linear(normed, self.w_o, out_dtype=torch.float32)
+
+
+@MIXERS.register("gated_linear_attention")
+class GatedLinearAttention(LinearRecurrence):
+    PROJECTED = ("q", "k", "v", "gate", "a_down")
+
+    def __init__(self, prefix: str, width: int, heads: int, head_dim: int, value_dim: int, tau: float, eps: float, decay_rank: int = -1,
+                 names: dict | None = None):
+        """`tau`: the root that is taken of the sigmoid; `decay_rank`: inner size of the two thin products (-1: as the checkpoint
+        has it)."""
+        super().__init__(prefix, width, heads, head_dim, value_dim, eps, dict({"a_down": "a_down.weight", "a_up": "a_up.weight",
+                                                                               "a_bias": "a_up.bias", "norm": "norm.weight"}, **(names or {})))
+        self.tau, self.rank = float(tau), int(decay_rank)
+        if not self.tau > 0:
+            raise InvalidRequest(f"{prefix}: tau must be positive")
+
+    def weight_specs(self):
+        n, qk = self.leaf, self.heads * self.d
+        return super().weight_specs() + [
+            WeightSpec(self.name(n["norm"]), (self.e,), "vector"), WeightSpec(self.name(n["a_down"]), (self.rank, self.width)),
+            WeightSpec(self.name(n["a_up"]), (qk, self.rank)), WeightSpec(self.name(n["a_bias"]), (qk,), "bias")]
+
+    def state_need(self):
+        return StateNeed((self.heads * self.d * self.e,), torch.float32)
+
+    def bind(self, tensors, runtime):
+        super().bind(tensors, runtime)
+        n = self.leaf
+        self.norm_w = tensors[self.name(n["norm"])].float().contiguous()
+        self.a_up = tensors[self.name(n["a_up"])].contiguous()
+        self.a_bias = tensors[self.name(n["a_bias"])].float().contiguous()
+        self.rank = self.a_up.shape[1]
+        if tensors[self.name(n["a_down"])].shape[0] != self.rank or self.rank > kernels.CHANNEL_SCAN_MAX_RANK:
+            raise InvalidRequest(f"{self.prefix}: the thin products' inner sizes differ, or are above {kernels.CHANNEL_SCAN_MAX_RANK}")
+
+    def forward_projected(self, proj, offset, ctx, cache, write_cache=True):
+        tokens, device = proj.shape[0], proj.device
+        H, d, e = self.heads, self.d, self.e
+        k_at, v_at = offset + H * d, offset + 2 * H * d
+        g_at, low_at = v_at + H * e, v_at + 2 * H * e
+        o = torch.empty((tokens, H * e), dtype=torch.float32, device=device)
+        kernels.channel_scan(proj, offset, k_at, v_at, low_at, self.a_up, self.a_bias, self.tau, self.matrix_state(cache), ctx.positions,
+                             ctx.seq_of_token, ctx.q_start, ctx.state_slots, o, H, d, e, write_state=write_cache)
+        normed = torch.empty((tokens, H * e), dtype=self.runtime.dtype, device=device)
+        kernels.head_norm_gate(o, proj[:, g_at:low_at], self.norm_w, self.eps, normed, H, factor=d ** -0.5)
         return linear(normed, self.w_o, out_dtype=torch.float32)

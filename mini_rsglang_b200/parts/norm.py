@@ -9,7 +9,18 @@ import torch
 from .. import kernels
 from ..errors import InvalidRequest
 from ..weights.spec import WeightSpec
-from .base import NORMS, Norm, Normed, Prenormed
+from .base import NORMS, BranchSum, Norm, Normed, Prenormed
+
+
+def _settle(residual: torch.Tensor, delta: BranchSum, write_back: bool) -> torch.Tensor:
+    """The stream with the sum's terms added (in place when `write_back`), for norms whose own kernel adds one branch."""
+    residual = residual if write_back else residual.clone()
+    terms = [(x if x.dtype is torch.float32 else x.float(), factor) for x, factor in delta.terms]
+    for at in range(0, len(terms), kernels.MAX_BRANCHES):
+        kernels.add_scaled_branches_norms(residual, terms[at:at + kernels.MAX_BRANCHES], [], 0.0)
+    if delta.row is not None:
+        residual.add_(delta.row)
+    return residual
 
 
 @NORMS.register("rmsnorm")
@@ -46,6 +57,9 @@ class RMSNorm(Norm):
             if delta.norm is self and rows is None:
                 return delta.rows
             delta = None
+        if isinstance(delta, BranchSum):
+            residual = _settle(residual, delta, write_back)
+            delta = None
         n = residual.shape[0] if rows is None else rows.shape[0]
         out = torch.empty((n, self.width), dtype=self.runtime.dtype, device=residual.device)
         kernels.add_rmsnorm(residual, delta, self.weight, self.eps, out, rows, write_back)
@@ -76,6 +90,8 @@ class NormPair(Norm):
         if rows is not None or not write_back:
             raise InvalidRequest("a pair of norms reads whole streams")
         outs = self.outputs(residual, self.first.runtime.dtype)
+        if isinstance(delta, BranchSum):
+            residual, delta = _settle(residual, delta, True), None
         kernels.add_scaled_branches_norms(residual, [(delta.float(), 1.0)] if delta is not None else [], outs, self.eps)
         return tuple(out for _, out in outs)
 
@@ -108,7 +124,17 @@ class LayerNorm(Norm):
     def add_norm(self, residual, delta, rows=None, write_back=True):
         if isinstance(delta, (Prenormed, Normed)):       # the stream holds the sum already
             delta = None
+        factor, extra, row = 1.0, None, None
+        if isinstance(delta, BranchSum):
+            # the kernel adds a branch times a factor, a second branch as it is and a vector; anything beyond is added before
+            terms, row = list(delta.terms), delta.row
+            plain_one = next((i for i in reversed(range(len(terms))) if terms[i][1] == 1.0 and terms[i][0].dtype is torch.float32), None)
+            if len(terms) > 1 and plain_one is not None:
+                extra = terms.pop(plain_one)[0]
+            if len(terms) > 1:
+                residual = _settle(residual, BranchSum(terms[1:]), write_back)
+            delta, factor = terms[0] if terms else (None, 1.0)
         n = residual.shape[0] if rows is None else rows.shape[0]
         out = torch.empty((n, self.width), dtype=self.runtime.dtype, device=residual.device)
-        kernels.add_layernorm(residual, delta, self.weight, self.bias, self.eps, out, rows, write_back)
+        kernels.add_layernorm(residual, delta, self.weight, self.bias, self.eps, out, rows, write_back, factor=factor, extra=extra, row=row)
         return out

@@ -16,6 +16,17 @@ from ..errors import InvalidRequest
 from .base import POSITION_ENCODINGS, PositionEncoding, Rotation
 
 
+def step_table(ctx, key, inv_freq: torch.Tensor, magnitude: float = 1.0) -> torch.Tensor:
+    """The cosines and sines of the step's positions, made at the first layer that asks and kept for the others."""
+    shared = getattr(ctx, "shared", None)
+    if shared is not None and key in shared:
+        return shared[key]
+    table = kernels.rotation_table(ctx.positions, inv_freq, magnitude)
+    if shared is not None:
+        shared[key] = table
+    return table
+
+
 @POSITION_ENCODINGS.register("rope")
 class RotaryPosition(PositionEncoding):
     def __init__(self, prefix: str, head_dim: int, theta: float, rotary_dim: int | None = None, pairing: str = "split_half"):
@@ -53,13 +64,7 @@ class RotaryPosition(PositionEncoding):
     def rotations(self, ctx):
         """[tokens, rotary_dim / 2, 2] float32 (cos, sin) for the step's positions; kept in `ctx.shared` for the
         step's other layers (the model empties it when a step begins)."""
-        shared = getattr(ctx, "shared", None)
-        if shared is not None and self.shared_key in shared:
-            return shared[self.shared_key]
-        table = kernels.rotation_table(ctx.positions, self.inv_freq)
-        if shared is not None:
-            shared[self.shared_key] = table
-        return table
+        return step_table(ctx, self.shared_key, self.inv_freq)
 
 
 @POSITION_ENCODINGS.register("banded_rope")
@@ -113,6 +118,7 @@ class YarnRotaryPosition(PositionEncoding):
         if self.scaled and (self.factor <= 0.0 or self.original <= 0.0 or self.fast <= 0.0 or self.slow <= 0.0):
             raise InvalidRequest("stretched rotary positions need a positive factor, original length and turn counts")
         self.inv_freq: torch.Tensor | None = None
+        self.shared_key = None
 
     def frequencies(self) -> torch.Tensor:
         dims, half = self.rotary_dim, self.rotary_dim // 2
@@ -137,10 +143,16 @@ class YarnRotaryPosition(PositionEncoding):
 
     def bind(self, tensors, runtime):
         super().bind(tensors, runtime)
-        self.inv_freq = self.frequencies().to(torch.float32).to(runtime.device)
+        frequencies = self.frequencies().to(torch.float32)
+        self.inv_freq = frequencies.to(runtime.device)
+        self.shared_key = ("rotations", frequencies.numpy().tobytes(), self.magnitude)
 
     def rotation(self):
         return Rotation(self.inv_freq, self.rotary_dim, "split_half", self.magnitude)
+
+    def rotations(self, ctx):
+        """As `RotaryPosition.rotations`, cosines and sines times `magnitude`."""
+        return step_table(ctx, self.shared_key, self.inv_freq, self.magnitude)
 
 
 @POSITION_ENCODINGS.register("none")
