@@ -323,13 +323,37 @@ def recurrent_configs(size: dict, vocab: int = 32768):
     return pisatar, parallel_configs(size, vocab)[0]
 
 
+def passed_configs(size: dict, vocab: int = 32768):
+    """Bilipel at these layer sizes: six layers of which the first two are passed twice (eight layer runs), gated linear attention
+    (width / 128 heads of 128 query/key and 256 value elements, thin products of 16; in layers 0, 3 and 4), attention (heads of
+    128, half of each rotated, sinks; layers 1 and 5) and latent attention (heads of 64 unrotated and 32 rotated query/key and 64
+    value elements, a latent of 256, a window of 1,024, sinks; layer 2); the first layer's feed-forward dense, the others 32
+    experts of ff / 8 with 4 chosen.  Beside it Satedra, the engine's other model of layer norms, latent attention and routed
+    experts, at equal width, heads, experts and depth."""
+    w, ff = size["width"], size["ff"]
+    dense = {"kind": "dense", "ff": ff}
+    routed = {"kind": "moe", "expert": {"ff": ff // 8}, "router": {"experts": 32, "top": 4}}
+    recurrent = {"type": "gla", "mixer": {"heads": w // 128, "dim": 128, "vdim": 256, "tau": 16.0, "decay_rank": 16}}
+    attention = {"type": "attention", "mixer": {
+        "heads": size["heads"], "kv_heads": size["kv_heads"], "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
+        "rot": {"base": 1000000.0, "dims": 64, "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}}
+    latent = {"type": "latent_attention", "mixer": {"heads": size["heads"], "dim": 64, "rot_dim": 32, "vdim": 64, "kv_rank": 256, "scale": 96 ** -0.5,
+                                                    "mask": {"size": 1024}, "rot": {"base": 1000000.0, "dims": 32}}}
+    layers = [dict(recurrent, mlp=dense), dict(attention, mlp=routed), dict(latent, mlp=routed), dict(recurrent, mlp=routed),
+              dict(recurrent, mlp=routed), dict(attention, mlp=routed)]
+    bilipel = {"architecture": "Bilipel", "vocab": vocab, "width": w, "norm": {"eps": 1e-5}, "residual_mult": 0.5,
+               "loop": {"start": 0, "stop": 2, "times": 2}, "layers": layers}
+    return bilipel, latent_configs(size, vocab)[0]
+
+
 # design: (title, what stands beside it, the key of that model in the output, the two configurations)
 DESIGNS = {"niduvik": ("Niduvik", "Qwen3 of equal width, heads, feed-forward and depth", "qwen3", hybrid_configs),
            "satedra": ("Satedra", "Qwen3 of equal width, heads and depth, its feed-forward as wide as the experts a token passes", "qwen3",
                        latent_configs),
            "nubipel": ("Nubipel", "Niduvik of equal width, heads, feed-forward and depth", "niduvik", parallel_configs),
            "migenex": ("Migenex", "Satedra of equal width, heads, experts and depth", "satedra", looped_configs),
-           "pisatar": ("Pisatar", "Nubipel of equal width, heads, feed-forward and depth", "nubipel", recurrent_configs)}
+           "pisatar": ("Pisatar", "Nubipel of equal width, heads, feed-forward and depth", "nubipel", recurrent_configs),
+           "bilipel": ("Bilipel", "Satedra of equal width, heads, experts and depth", "satedra", passed_configs)}
 
 
 def hybrid_run(args, torch, peak: dict) -> dict:

@@ -17,7 +17,8 @@
 // stores its slice, in the order of the shares.  Nothing of the merge goes through global memory,
 // whose dependent trips (result out, fence, counter, results in) cost microseconds each at the
 // end of a kernel.  Other split counts leave their results in scratch memory, and the CTA that
-// finishes a (tile, head) last merges them in order.
+// finishes a (tile, head) last merges them in order.  A learned sink a query head (one more term exp(sink) in the denominator,
+// without key and value) joins a row's sum in the last merge.
 #include "tma.cuh"
 
 #ifndef MRS_HEAD_DIM
@@ -98,6 +99,11 @@ __device__ __forceinline__ void cluster_sync_all() {
 }
 constexpr int MAX_CLUSTER = 16;
 
+// The sink's term of a row whose sum is scaled by 2^-base (beyond the range of a float the row's weights are 0 anyway).
+__device__ __forceinline__ float sink_term(const float* sinks, int head, float base) {
+    return sinks ? exp2f(sinks[head] * 1.4426950408889634f - base) : 0.0f;
+}
+
 __device__ __forceinline__ void consumer_sync() { asm volatile("bar.sync 1, %0;" ::"n"(32 * CONSUMER_WARPS) : "memory"); }
 
 __global__ void __launch_bounds__(THREADS) attention_decode_kernel(
@@ -105,7 +111,7 @@ __global__ void __launch_bounds__(THREADS) attention_decode_kernel(
     const bf16* __restrict__ q, const int* __restrict__ positions, const int* __restrict__ block_table, int table_width,
     const Tile* __restrict__ tiles, bf16* __restrict__ out, float* __restrict__ part_o, float* __restrict__ part_ml,
     int* __restrict__ counters, int nq, int nkv, int page_size, int page_shift, float scale_log2, float scale, float cap, int window, int splits,
-    int in_cluster) {
+    int in_cluster, const float* __restrict__ sinks) {
     extern __shared__ unsigned char smem_raw[];
     __shared__ int is_last;
     const Tile tile = tiles[blockIdx.x];
@@ -369,6 +375,7 @@ __global__ void __launch_bounds__(THREADS) attention_decode_kernel(
                 sum += incoming_ml[(s * ROWS + row) * 2 + 1] * f;
                 acc.x += v.x * f, acc.y += v.y * f, acc.z += v.z * f, acc.w += v.w * f;
             }
+            sum += sink_term(sinks, kv_head * group + row % group, base);
             const float inv = sum > 0.0f ? 1.0f / sum : 0.0f;
             bf16* dst = out + ((size_t)(tile.first_token + row / group) * nq + kv_head * group + row % group) * D + split * cols + col;
             *reinterpret_cast<__nv_bfloat162*>(dst) = __floats2bfloat162_rn(acc.x * inv, acc.y * inv);
@@ -394,6 +401,7 @@ __global__ void __launch_bounds__(THREADS) attention_decode_kernel(
             acc += merge_o[(w * ROWS + row) * D + col] * f;
         }
         if (splits == 1) {
+            sum += sink_term(sinks, kv_head * group + row % group, base);
             out[((size_t)(tile.first_token + row / group) * nq + kv_head * group + row % group) * D + col] =
                 __float2bfloat16_rn(sum > 0.0f ? acc / sum : 0.0f);
         } else {
@@ -446,6 +454,7 @@ __global__ void __launch_bounds__(THREADS) attention_decode_kernel(
                     acc.x += v[u].x * f, acc.y += v[u].y * f, acc.z += v[u].z * f, acc.w += v[u].w * f;
                 }
         }
+        sum += sink_term(sinks, kv_head * group + row % group, base);
         const float inv = sum > 0.0f ? 1.0f / sum : 0.0f;
         bf16* dst = out + ((size_t)(tile.first_token + row / group) * nq + kv_head * group + row % group) * D + col;
         *reinterpret_cast<__nv_bfloat162*>(dst) = __floats2bfloat162_rn(acc.x * inv, acc.y * inv);
@@ -486,7 +495,7 @@ MRS_EXPORT long long mrs_attention_decode_tma_scratch_floats(int tiles, int nkv,
 MRS_EXPORT int mrs_attention_decode_tma(const void* k_map, const void* v_map, const void* q, const int* positions,
                                         const int* block_table, int table_width, const int* tiles, int num_tiles,
                                         void* out, float* scratch, int* counters, int nq, int nkv, int page_size,
-                                        float scale, int window, int splits, float cap, void* stream) {
+                                        float scale, int window, int splits, float cap, const float* sinks, void* stream) {
     if (num_tiles <= 0) return 0;
     if (cap < 0.0f) return MRS_BAD_ARGUMENT;
     const int shift = page_shift_of(page_size);
@@ -536,12 +545,12 @@ MRS_EXPORT int mrs_attention_decode_tma(const void* k_map, const void* v_map, co
         return (int)cudaLaunchKernelEx(&config, attention_decode_kernel, *reinterpret_cast<const CUtensorMap*>(k_map),
                                        *reinterpret_cast<const CUtensorMap*>(v_map), (const bf16*)q, positions, block_table, table_width,
                                        (const Tile*)tiles, (bf16*)out, part_o, part_ml, counters, nq, nkv, page_size, shift, scale_log2,
-                                       scale, cap, window, splits, 1);
+                                       scale, cap, window, splits, 1, sinks);
     }
     MRS_LAUNCH(attention_decode_kernel, dim3(num_tiles, nkv, splits), THREADS, SMEM_BYTES, stream,
         *reinterpret_cast<const CUtensorMap*>(k_map), *reinterpret_cast<const CUtensorMap*>(v_map), (const bf16*)q,
         positions, block_table, table_width, (const Tile*)tiles, (bf16*)out, part_o, part_ml, counters, nq, nkv, page_size,
-        shift, scale_log2, scale, cap, window, splits, 0);
+        shift, scale_log2, scale, cap, window, splits, 0, sinks);
     MRS_RETURN_LAUNCH_STATUS();
 }
 

@@ -26,7 +26,8 @@
 // memory carries only Q, K and V: with P there too its bandwidth (128 bytes a clock) was the bound.
 // The accumulators stay in tensor memory; one is rescaled only when a row's maximum grew by more
 // than 2^8 since the last rescale (the sum uses the same reference, so the quotient is exact), and
-// is normalised and stored at the end.
+// is normalised and stored at the end.  A learned sink a query head (one more term exp(sink) in the denominator, without key
+// and value) joins a row's sum there.
 // Every wait is bounded (tma.cuh).
 #include "tcgen05.cuh"
 
@@ -109,13 +110,18 @@ struct Barriers {
 
 constexpr size_t SMEM_BYTES = 1024 + TILES * Q_TILE_BYTES + 2 * STAGES * KV_TILE_BYTES + sizeof(Barriers) + 16;
 
+// The sink's term of a row whose sum is scaled by 2^-reference (beyond the range of a float the row's weights are 0 anyway).
+__device__ __forceinline__ float sink_term(const float* sinks, int head, float reference) {
+    return sinks ? exp2f(sinks[head] * 1.4426950408889634f - reference) : 0.0f;
+}
+
 // CAPPED: the scores pass the soft cap (a variant of its own, so that the plain one keeps its registers)
 template <bool CAPPED>
 __global__ void __launch_bounds__(THREADS, 1) attention_prefill_kernel(
     const __grid_constant__ CUtensorMap q_map, const __grid_constant__ CUtensorMap k_map,
     const __grid_constant__ CUtensorMap v_map, const int* __restrict__ positions, const int* __restrict__ block_table,
     int table_width, const Tile* __restrict__ tiles, bf16* __restrict__ out, int nq, int nkv, int page_size,
-    int page_shift, float scale_log2, int window, float* __restrict__ partials, float cap_in, float cap_out) {
+    int page_shift, float scale_log2, int window, float* __restrict__ partials, float cap_in, float cap_out, const float* __restrict__ sinks) {
     extern __shared__ unsigned char smem_raw[];
     // the grid runs over the key/value heads first: with the entries sorted by their work, all heavy CTAs start first
     const Tile work = tiles[blockIdx.y];
@@ -429,6 +435,7 @@ __global__ void __launch_bounds__(THREADS, 1) attention_prefill_kernel(
                 for (int c = 0; c < D; c += 4) dst[c / 4] = make_float4(o[c], o[c + 1], o[c + 2], o[c + 3]);
                 dst[D / 4] = make_float4(reference, sum, 0.0f, 0.0f);
             } else if (row < rows) {
+                sum += sink_term(sinks, kv_head * group + row % group, reference);
                 const float inv = sum > 0.0f ? 1.0f / sum : 0.0f;
                 bf16* dst = out + ((size_t)(tile_first[i] + row / group) * nq + kv_head * group + row % group) * D;
 #pragma unroll
@@ -455,7 +462,7 @@ __global__ void __launch_bounds__(THREADS, 1) attention_prefill_kernel(
 // Puts the shares of an entry together: out = sum_s O_s 2^(m_s - M) / sum_s l_s 2^(m_s - M), M the largest maximum.
 // A warp per query row (grid: key/value heads x entries x 32 groups of 8 rows); only the CTAs of an entry's first share work.
 __global__ void __launch_bounds__(256) attention_prefill_merge_kernel(const Tile* __restrict__ tiles, const float* __restrict__ partials,
-                                                                    bf16* __restrict__ out, int nq, int nkv) {
+                                                                    bf16* __restrict__ out, int nq, int nkv, const float* __restrict__ sinks) {
     pdl_launch_dependents();
     pdl_wait();
     const Tile work = tiles[blockIdx.y];
@@ -486,6 +493,7 @@ __global__ void __launch_bounds__(256) attention_prefill_merge_kernel(const Tile
 #pragma unroll
         for (int e = 0; e < PER_LANE; ++e) acc[e] += p[lane * PER_LANE + e] * w;
     }
+    total += sink_term(sinks, kv_head * group + row % group, best);
     const float inv = total > 0.0f ? 1.0f / total : 0.0f;
     bf16* dst = out + ((size_t)(work.first_token + i * tokens_per_tile + row / group) * nq + kv_head * group + row % group) * D +
                 lane * PER_LANE;
@@ -538,7 +546,7 @@ MRS_EXPORT long long mrs_attention_prefill_tc_partial_floats(int num_tiles, int 
 MRS_EXPORT int mrs_attention_prefill_tc(const void* q_map, const void* k_map, const void* v_map, const int* positions,
                                         const int* block_table, int table_width, const int* tiles, int num_tiles,
                                         void* out, int nq, int nkv, int page_size, float scale, int window,
-                                        float* partials, int with_shares, float cap, void* stream) {
+                                        float* partials, int with_shares, float cap, const float* sinks, void* stream) {
     if (num_tiles <= 0) return 0;
     if (with_shares && (!partials || num_tiles > 65535)) return MRS_BAD_ARGUMENT;
     if (cap < 0.0f || !(scale > 0.0f)) return MRS_BAD_ARGUMENT;
@@ -559,16 +567,16 @@ MRS_EXPORT int mrs_attention_prefill_tc(const void* q_map, const void* k_map, co
             MRS_LAUNCH(attention_prefill_kernel<true>, dim3(nkv, now), THREADS, SMEM_BYTES, stream,
                    *reinterpret_cast<const CUtensorMap*>(q_map), *reinterpret_cast<const CUtensorMap*>(k_map),
                    *reinterpret_cast<const CUtensorMap*>(v_map), positions, block_table, table_width, (const Tile*)tiles + done,
-                   (bf16*)out, nq, nkv, page_size, shift, scale * 1.4426950408889634f, window, with_shares ? partials : nullptr, cap_in, cap_out);
+                   (bf16*)out, nq, nkv, page_size, shift, scale * 1.4426950408889634f, window, with_shares ? partials : nullptr, cap_in, cap_out, sinks);
         else
             MRS_LAUNCH(attention_prefill_kernel<false>, dim3(nkv, now), THREADS, SMEM_BYTES, stream,
                    *reinterpret_cast<const CUtensorMap*>(q_map), *reinterpret_cast<const CUtensorMap*>(k_map),
                    *reinterpret_cast<const CUtensorMap*>(v_map), positions, block_table, table_width, (const Tile*)tiles + done,
-                   (bf16*)out, nq, nkv, page_size, shift, scale * 1.4426950408889634f, window, with_shares ? partials : nullptr, cap_in, cap_out);
+                   (bf16*)out, nq, nkv, page_size, shift, scale * 1.4426950408889634f, window, with_shares ? partials : nullptr, cap_in, cap_out, sinks);
     }
     if (with_shares)
         MRS_LAUNCH(attention_prefill_merge_kernel, dim3(nkv, num_tiles, TILES * BM / 8), 256, 0, stream, (const Tile*)tiles, (const float*)partials,
-                   (bf16*)out, nq, nkv);
+                   (bf16*)out, nq, nkv, sinks);
     MRS_RETURN_LAUNCH_STATUS();
 }
 

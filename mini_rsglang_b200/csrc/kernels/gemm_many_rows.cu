@@ -1,6 +1,6 @@
 // The feed-forward's first product for many rows (prompt portions) on the tcgen05 tensor cores, bfloat16 in, float32
 // accumulation, with the activation in its epilogue:
-//   out[T, N / 2] = silu(x . gate^T) * (x . up^T)          (gated feed-forwards)
+//   out[T, N / 2] = act(x . gate^T) * (x . up^T)           (gated feed-forwards: silu, relu, gelu with tanh)
 //   out[T, N]     = act(x . w^T)                            (plain ones: gelu with the error function or with tanh, silu)
 //
 // The library's product for these sizes runs near the tensor cores' peak, but it leaves its result in
@@ -39,7 +39,10 @@ __device__ __forceinline__ float activate(float z, int kind) {
     return z / (1.0f + expf(-z));
 }
 
-// ACT < 0: the gated product (-1: silu(gate) * up, -2: relu(gate) * up); 0 to 4: the plain product with gelu (error
+// 0.5 z (1 + tanh(u)) = z / (1 + exp(-2 u)) with u = sqrt(2 / pi) (z + 0.044715 z^3)
+__device__ __forceinline__ float gelu_tanh_gate(float z) { return z / (1.0f + __expf(-1.5957691216057308f * (z + 0.044715f * z * z * z))); }
+
+// ACT < 0: the gated product (-1: silu(gate) * up, -2: relu(gate) * up, -3: gelu with tanh); 0 to 4: the plain product with gelu (error
 // function), gelu (tanh), silu, relu or the square of relu on every sum.
 template <int ACT>
 __global__ void __launch_bounds__(THREADS, 1) gemm_many_rows_kernel(
@@ -187,6 +190,8 @@ __global__ void __launch_bounds__(THREADS, 1) gemm_many_rows_kernel(
                                 const float g0 = g[e + 2 * p], g1 = g[e + 2 * p + 1];
                                 __nv_bfloat162 pair = ACT == -2
                                     ? __floats2bfloat162_rn(fmaxf(g0, 0.0f) * u[e + 2 * p], fmaxf(g1, 0.0f) * u[e + 2 * p + 1])
+                                    : ACT == -3
+                                    ? __floats2bfloat162_rn(gelu_tanh_gate(g0) * u[e + 2 * p], gelu_tanh_gate(g1) * u[e + 2 * p + 1])
                                     : __floats2bfloat162_rn(g0 / (1.0f + __expf(-g0)) * u[e + 2 * p],
                                                             g1 / (1.0f + __expf(-g1)) * u[e + 2 * p + 1]);
                                 w[p] = *reinterpret_cast<uint32_t*>(&pair);
@@ -236,14 +241,15 @@ MRS_EXPORT int mrs_gemm_many_rows_map(const void* base, long long rows, long lon
     return mrs_make_tensor_map_bf16(reinterpret_cast<CUtensorMap*>(map_out), base, 2, dims, strides, box, CU_TENSOR_MAP_SWIZZLE_128B);
 }
 
-// out[T, N / 2] = act(x . gate^T) * (x . up^T), bfloat16, act silu (gate_act 2) or relu (3); w [N, K] holds in every block of 128 rows 64 gate rows and
+// out[T, N / 2] = act(x . gate^T) * (x . up^T), bfloat16, act gelu with tanh (gate_act 1), silu (2) or relu (3); w [N, K] holds in every block of 128 rows 64 gate rows and
 // then the 64 matching up rows (N a multiple of 128).  `x_map`: map of x [T, K] with boxes of 128 rows; `w_map`: map
 // of w with boxes of 256 rows.  `ctas`: the GPU's SMs.
 MRS_EXPORT int mrs_gemm_gated_rows(const void* x_map, const void* w_map, void* out, int T, int N, int K, int gate_act, int ctas,
                                    void* stream) {
     if (T <= 0 || N <= 0) return 0;
-    if (K <= 0 || K % 8 || N % 128 || ctas < 1 || !x_map || !w_map || !out || ((uintptr_t)out & 15) || (gate_act != 2 && gate_act != 3))
+    if (K <= 0 || K % 8 || N % 128 || ctas < 1 || !x_map || !w_map || !out || ((uintptr_t)out & 15) || gate_act < 1 || gate_act > 3)
         return MRS_BAD_ARGUMENT;
+    if (gate_act == 1) return launch<-3>(x_map, w_map, out, T, N, K, ctas, stream);
     if (gate_act == 3) return launch<-2>(x_map, w_map, out, T, N, K, ctas, stream);
     return launch<-1>(x_map, w_map, out, T, N, K, ctas, stream);
 }

@@ -97,6 +97,7 @@ struct NormLink {
     float* stream;                   // [M, N] float32 (EPI_RESIDUAL)
     const float* next_weight;        // [N]
     float* out_square_sums;          // [tiles of N][MPAD]
+    int gelu;                        // EPI_GATED: the gate passes gelu (tanh form) instead of silu
 };
 
 // What the head epilogue needs beside the product: where q goes, the cache pages of k and v, the
@@ -398,7 +399,9 @@ __global__ void __launch_bounds__(THREADS, 1) gemm_small_m_kernel(
                         for (int m = 0; m < MPAD; ++m)
                             if (m < M) {
                                 const float g = acc[m], u = exchange[m * 64 + row];
-                                out[(size_t)m * (N >> 1) + tile * 64 + row] = from_float<OutT>(g / (1.0f + __expf(-g)) * u);
+                                // gelu with tanh: g / (1 + exp(-2 sqrt(2 / pi) (g + 0.044715 g^3)))
+                                const float z = link.gelu ? 1.5957691216057308f * (g + 0.044715f * g * g * g) : g;
+                                out[(size_t)m * (N >> 1) + tile * 64 + row] = from_float<OutT>(g / (1.0f + __expf(-z)) * u);
                             }
                     }
                 } else if (EPI == EPI_HEADS) {
@@ -547,7 +550,7 @@ MRS_EXPORT int mrs_gemm_tc_counters(int N) { return (N + TILE_N - 1) / TILE_N; }
 // out[M, N] = x . w^T.  `w_map`: mrs_gemm_tc_map(w, N, K, 128); `x_map`: mrs_gemm_tc_map(x, M, K, mpad) with
 // mpad = 16, 32, 64 or 128 >= M.  `out` is bfloat16 or float32 [M, N].  `ctas`: CTAs to launch (the GPU's SMs).
 // With `gated`, w holds in every block of 128 rows 64 gate rows followed by the 64 matching up rows (N a
-// multiple of 128), and out[M, N / 2] = silu(x . gate^T) * (x . up^T), bfloat16.
+// multiple of 128), and out[M, N / 2] = act(x . gate^T) * (x . up^T), bfloat16, act silu (1) or gelu with tanh (2).
 // `link` (or null): a NormLink.  With `in_square_sums` the sums are multiplied by their rows' norm factors; with
 // `stream` (up to 32 rows, bfloat16 out, not gated) the result is added to the stream and `out` gets the stream
 // times `next_weight`, with the parts of the rows' sums of squares in `out_square_sums` [ceil(N / 128)][mpad].
@@ -557,6 +560,7 @@ MRS_EXPORT int mrs_gemm_tc_small_m(const void* w_map, const void* x_map, void* o
     if (M <= 0 || N <= 0) return 0;
     NormLink link{};
     if (link_in) link = *reinterpret_cast<const NormLink*>(link_in);
+    link.gelu = gated == 2;
     if (link.in_square_sums && (link.in_parts <= 0 || link.in_stride < M)) return MRS_BAD_ARGUMENT;
     if (link.stream && (gated || out_is_f32 || mpad > 32 || !link.next_weight || !link.out_square_sums)) return MRS_BAD_ARGUMENT;
     if (K <= 0 || K % 8 || M > mpad || !ranges_fit(splits, N, K) || ctas < 1) return MRS_BAD_ARGUMENT;

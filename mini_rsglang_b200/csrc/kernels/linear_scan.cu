@@ -187,7 +187,7 @@ __device__ __forceinline__ float channel_keep(float z, float inverse_tau) { retu
 // S_t = diag(P_t) U_t with U_t = U_(t-1) + (k_t / P_t) v_t^T and o_t = U_t^T (P_t q_t): k and q are divided and multiplied in place,
 // P goes to `keeps`, and the recurrence multiplies S by P once a batch.  Where some P of a (batch, head) falls below FOLD_LEAST
 // nothing is folded there: `keeps` gets the keeps themselves and `direct` says so.
-// A thread takes a channel and the rows of a batch; a block whole heads.  Dynamic shared memory: batch * rank floats.
+// A thread takes a channel and the rows of a batch; a block whole heads.  Dynamic shared memory: SCAN_BATCH * rank floats.
 // ---------------------------------------------------------------------------------------------
 #define FOLD_LEAST 1e-15f
 template <typename W>
@@ -200,22 +200,40 @@ __global__ void channel_fold_kernel(const ScanArgs A, float* __restrict__ q, flo
     const int t0 = blockIdx.x * A.batch, n = min(A.batch, tokens - t0);
     const int head0 = blockIdx.y * heads_a_block, own = threadIdx.x / A.d;
     const bool live = own < heads_a_block && head0 + own < A.heads;
-    for (int i = threadIdx.x; i < n * A.rank; i += blockDim.x)
-        low_rows[i] = A.low[(size_t)(t0 + i / A.rank) * A.stride + i % A.rank];
+    const int channel = head0 * A.d + threadIdx.x;
+    float a[SCAN_BATCH], P[SCAN_BATCH], qs[SCAN_BATCH], ks[SCAN_BATCH];
+#pragma unroll
+    for (int j = 0; j < SCAN_BATCH; ++j) {                   // asked for ahead of their use
+        const bool here = live && j < n;
+        qs[j] = here ? q[(size_t)(t0 + j) * A.stride + channel] : 0.0f;
+        ks[j] = here ? k[(size_t)(t0 + j) * A.stride + channel] : 0.0f;
+    }
+    for (int i = threadIdx.x; i < SCAN_BATCH * A.rank; i += blockDim.x) {        // [rank][SCAN_BATCH]
+        const int j = i / A.rank, r = i % A.rank;
+        low_rows[r * SCAN_BATCH + j] = j < n ? A.low[(size_t)(t0 + j) * A.stride + r] : 0.0f;
+    }
     if (threadIdx.x < 32) small[threadIdx.x] = 0;
     __syncthreads();
-    const int channel = head0 * A.d + threadIdx.x;
-    float a[SCAN_BATCH], P[SCAN_BATCH];
     if (live) {
         const float b = A.keep_bias[channel];
 #pragma unroll
         for (int j = 0; j < SCAN_BATCH; ++j) a[j] = b;
         const W* up = (const W*)A.up + (size_t)channel * A.rank;
-        for (int r = 0; r < A.rank; ++r) {
-            const float w = to_float(up[r]);
+        auto add = [&](float w, int r) {
+            const float4 lo = *reinterpret_cast<const float4*>(low_rows + r * SCAN_BATCH), hi = *reinterpret_cast<const float4*>(low_rows + r * SCAN_BATCH + 4);
+            a[0] = fmaf(w, lo.x, a[0]), a[1] = fmaf(w, lo.y, a[1]), a[2] = fmaf(w, lo.z, a[2]), a[3] = fmaf(w, lo.w, a[3]);
+            a[4] = fmaf(w, hi.x, a[4]), a[5] = fmaf(w, hi.y, a[5]), a[6] = fmaf(w, hi.z, a[6]), a[7] = fmaf(w, hi.w, a[7]);
+        };
+        constexpr int PIECE = 16 / sizeof(W);                // matrix elements of a 16-byte load
+        if (A.rank % PIECE == 0 && ((uintptr_t)A.up & 15) == 0) {
+            for (int r = 0; r < A.rank; r += PIECE) {
+                const uint4 raw = *reinterpret_cast<const uint4*>(up + r);
+                const W* w = reinterpret_cast<const W*>(&raw);
 #pragma unroll
-            for (int j = 0; j < SCAN_BATCH; ++j)
-                if (j < n) a[j] = fmaf(w, low_rows[j * A.rank + r], a[j]);
+                for (int u = 0; u < PIECE; ++u) add(to_float(w[u]), r + u);
+            }
+        } else {
+            for (int r = 0; r < A.rank; ++r) add(to_float(up[r]), r);
         }
         float p = 1.0f;
         bool tiny = false;
@@ -242,8 +260,8 @@ __global__ void channel_fold_kernel(const ScanArgs A, float* __restrict__ q, flo
         const size_t t = t0 + j;
         A.keeps[t * A.heads * A.d + channel] = direct ? a[j] : P[j];
         if (!direct) {
-            k[t * A.stride + channel] /= P[j];
-            q[t * A.stride + channel] *= P[j];
+            k[t * A.stride + channel] = ks[j] / P[j];
+            q[t * A.stride + channel] = qs[j] * P[j];
         }
     }
     if (threadIdx.x % A.d == 0) A.direct[(size_t)blockIdx.x * A.heads + head0 + own] = direct;
@@ -921,7 +939,7 @@ MRS_EXPORT int mrs_channel_scan(float* q, float* k, const float* v, int stride, 
     if (heads_a_block > heads) heads_a_block = heads;
     const dim3 grid((tokens + A.batch - 1) / A.batch, (heads + heads_a_block - 1) / heads_a_block);
     const int threads = (heads_a_block * d + 31) / 32 * 32;
-    const size_t smem = (size_t)A.batch * rank * sizeof(float);
+    const size_t smem = (size_t)SCAN_BATCH * rank * sizeof(float);
     if (up_is_bf16) MRS_LAUNCH(channel_fold_kernel<bf16>, grid, threads, smem, s, A, q, k, seq_of_token, tokens, heads_a_block);
     else MRS_LAUNCH(channel_fold_kernel<float>, grid, threads, smem, s, A, q, k, seq_of_token, tokens, heads_a_block);
     return scan_run<true>(A, tokens, sequences, parts, scratch, s);

@@ -28,10 +28,21 @@ __device__ __forceinline__ void head_norm(float* x, int d, const float* w, float
 
 // norm_mode: 0 none, 1 a head before the rotation, 2 a head after it, 3 the whole projection before it.
 // What the elements of q (and of k) are multiplied by when the norm is over all of them; the whole block takes part.
+template <bool VEC>
 __device__ __forceinline__ float2 projection_scales(const float* row, int qw, int kw, float eps, float* scratch) {
     float q = 0.0f, k = 0.0f;
-    for (int i = threadIdx.x; i < qw; i += blockDim.x) q += row[i] * row[i];
-    for (int i = threadIdx.x; i < kw; i += blockDim.x) k += row[qw + i] * row[qw + i];
+    if (VEC) {
+#pragma unroll 4
+        for (int i = 4 * threadIdx.x; i < qw + kw; i += 4 * blockDim.x) {
+            const float4 x = *reinterpret_cast<const float4*>(row + i);
+            const float part = (x.x * x.x + x.y * x.y) + (x.z * x.z + x.w * x.w);
+            if (i < qw) q += part;
+            else k += part;
+        }
+    } else {
+        for (int i = threadIdx.x; i < qw; i += blockDim.x) q += row[i] * row[i];
+        for (int i = threadIdx.x; i < kw; i += blockDim.x) k += row[qw + i] * row[qw + i];
+    }
     const float q_sum = block_sum(q, scratch), k_sum = block_sum(k, scratch);
     return make_float2(1.0f / sqrtf(q_sum / (float)qw + eps), 1.0f / sqrtf(k_sum / (float)kw + eps));
 }
@@ -76,7 +87,7 @@ qkv_rotary_store_kernel(const float* __restrict__ proj, int proj_stride, const f
     const float* turn = rotations ? rotations + t * (size_t)half * 2 : nullptr;
     const int units = nq + nkv + (values_from_keys ? 0 : nkv);
     __shared__ float scratch[33];
-    const float2 whole = norm_mode == 3 ? projection_scales(row, qw, kw, eps, scratch) : make_float2(1.0f, 1.0f);
+    const float2 whole = norm_mode == 3 ? projection_scales<VEC>(row, qw, kw, eps, scratch) : make_float2(1.0f, 1.0f);
     for (int unit = warp; unit < units; unit += ROTARY_WARPS) {
         if (unit >= nq + nkv) {                              // a value head with columns of its own
             if (!store || !v_cache) continue;
@@ -145,7 +156,7 @@ qkv_rotary_store_regs_kernel(const float* __restrict__ proj, int proj_stride, co
     const int at = 4 * lane;                                  // this lane's first element of a head
     const float4 zero = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
     __shared__ float scratch[33];
-    const float2 whole = norm_mode == 3 ? projection_scales(row, qw, kw, eps, scratch) : make_float2(1.0f, 1.0f);
+    const float2 whole = norm_mode == 3 ? projection_scales<true>(row, qw, kw, eps, scratch) : make_float2(1.0f, 1.0f);
     for (int unit = warp; unit < units; unit += ROTARY_WARPS) {
         if (unit >= nq + nkv) {                              // a value head with columns of its own
             if (!store || !v_cache) continue;

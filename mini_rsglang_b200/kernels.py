@@ -434,7 +434,7 @@ def attention_decode_tma_library(d: int) -> ctypes.CDLL:
         lib.mrs_attention_decode_tma_map.argtypes = [_c_vp, ctypes.c_longlong, _c_int, _c_int, _c_vp]
         lib.mrs_attention_decode_tma_map.restype = _c_int
         lib.mrs_attention_decode_tma.argtypes = [_c_vp] * 5 + [_c_int, _c_vp, _c_int, _c_vp, _c_vp, _c_vp, _c_int, _c_int,
-                                                 _c_int, _c_float, _c_int, _c_int, _c_float, _c_vp]
+                                                 _c_int, _c_float, _c_int, _c_int, _c_float, _c_vp, _c_vp]
         lib.mrs_attention_decode_tma.restype = _c_int
         lib.mrs_attention_decode_tma_scratch_floats.argtypes = [_c_int, _c_int, _c_int]
         lib.mrs_attention_decode_tma_scratch_floats.restype = ctypes.c_longlong
@@ -487,11 +487,14 @@ def kv_tensor_map(cache: torch.Tensor) -> int:
 
 def attention_decode_tma(q, k_cache, v_cache, positions, block_table, tiles, out, nq: int, nkv: int, d: int,
                          window: int = 0, splits: int = 1, scale: float | None = None,
-                         scratch: torch.Tensor | None = None, cap: float = 0.0) -> None:
+                         scratch: torch.Tensor | None = None, cap: float = 0.0, sink_logits: torch.Tensor | None = None) -> None:
     """Tiles of up to 16 // (nq // nkv) tokens each; keys and values come through bulk tensor copies.  `scale`: of the
-    scores (None: 1 / sqrt(d)); `cap` > 0: the scaled scores are bent into (-cap, cap), cap * tanh(score / cap)."""
+    scores (None: 1 / sqrt(d)); `cap` > 0: the scaled scores are bent into (-cap, cap), cap * tanh(score / cap); `sink_logits`
+    [nq] float32: the softmax's denominator also has exp(sink_logits[head])."""
     global launch_count
     _attention_mma_checks(q, k_cache, v_cache, positions, block_table, tiles, out, nq, nkv, d)
+    if sink_logits is not None:
+        _need(sink_logits, torch.float32, "sink logits", (nq,))
     lib = attention_decode_tma_library(d)
     counters = None
     if splits > 1:
@@ -507,7 +510,7 @@ def attention_decode_tma(q, k_cache, v_cache, positions, block_table, tiles, out
                                         out.data_ptr(), _ptr(scratch) if splits > 1 else None, _ptr(counters), nq, nkv,
                                         k_cache.shape[2],
                                         float(scale if scale is not None else 1.0 / math.sqrt(d)), int(window),
-                                        int(splits), float(cap), _stream())
+                                        int(splits), float(cap), _ptr(sink_logits), _stream())
     launch_count += 1
     if code != 0:
         raise BackendError(f"attention_decode_tma: {lib.mrs_attention_decode_tma_error_string(code).decode()} (code {code})")
@@ -542,7 +545,7 @@ def attention_prefill_tc_library(d: int) -> ctypes.CDLL:
         lib.mrs_attention_prefill_tc_kv_map.argtypes = [_c_vp, ctypes.c_longlong, _c_int, _c_int, _c_vp]
         lib.mrs_attention_prefill_tc_q_map.argtypes = [_c_vp, ctypes.c_longlong, _c_int, _c_int, _c_vp]
         lib.mrs_attention_prefill_tc.argtypes = [_c_vp] * 5 + [_c_int, _c_vp, _c_int, _c_vp, _c_int, _c_int, _c_int, _c_float,
-                                                 _c_int, _c_vp, _c_int, _c_float, _c_vp]
+                                                 _c_int, _c_vp, _c_int, _c_float, _c_vp, _c_vp]
         lib.mrs_attention_prefill_tc_partial_floats.argtypes = [_c_int, _c_int]
         lib.mrs_attention_prefill_tc_partial_floats.restype = ctypes.c_longlong
         for name in ("mrs_attention_prefill_tc_kv_map", "mrs_attention_prefill_tc_q_map", "mrs_attention_prefill_tc"):
@@ -560,15 +563,19 @@ def attention_prefill_tc_library(d: int) -> ctypes.CDLL:
 
 
 def attention_prefill_tc(q, k_cache, v_cache, positions, block_table, tiles, out, nq: int, nkv: int, d: int,
-                         window: int = 0, scale: float | None = None, shares: bool = False, cap: float = 0.0) -> None:
+                         window: int = 0, scale: float | None = None, shares: bool = False, cap: float = 0.0,
+                         sink_logits: torch.Tensor | None = None) -> None:
     """Work entries of up to 256 // (nq // nkv) tokens of one request each, on the tcgen05 tensor cores; `scale` of the
     scores (None: 1 / sqrt(d)), `cap` > 0: the scaled scores are bent into (-cap, cap), cap * tanh(score / cap).  The
     fourth number of an entry is 0, or index | count << 8 when `count` entries (one after the other in the list)
     walk one share of the keys each (`shares` says that the list has such entries, whose sums a second kernel
     merges), or gap << 16 when the entry's second tile of 128 // (nq // nkv) tokens starts `gap` tokens behind
-    the end of its first (the entry's token count is that of both tiles)."""
+    the end of its first (the entry's token count is that of both tiles).  `sink_logits` [nq] float32: the softmax's
+    denominator also has exp(sink_logits[head])."""
     global launch_count
     _attention_mma_checks(q, k_cache, v_cache, positions, block_table, tiles, out, nq, nkv, d)
+    if sink_logits is not None:
+        _need(sink_logits, torch.float32, "sink logits", (nq,))
     lib = attention_prefill_tc_library(d)
 
     def fail(code, what):
@@ -595,7 +602,7 @@ def attention_prefill_tc(q, k_cache, v_cache, positions, block_table, tiles, out
     code = lib.mrs_attention_prefill_tc(q_map, maps[0], maps[1], positions.data_ptr(), block_table.data_ptr(),
                                         block_table.shape[1], tiles.data_ptr(), tiles.shape[0], out.data_ptr(), nq, nkv,
                                         k_cache.shape[2], float(scale if scale is not None else 1.0 / math.sqrt(d)),
-                                        int(window), _ptr(partials), int(shares), float(cap), _stream())
+                                        int(window), _ptr(partials), int(shares), float(cap), _ptr(sink_logits), _stream())
     if code != 0:
         fail(code, "attention_prefill_tc")
 
@@ -607,6 +614,7 @@ _gemm_lib = None
 _weight_maps: dict[tuple, tuple] = {}
 _gemm_state: dict[torch.device, dict] = {}
 GEMM_TC_MAX_ROWS = 128          # what the kernel takes
+GEMM_TC_GATES = {"silu": 1, "gelu_tanh": 2}      # what its gated form applies to the gate
 # Measured in the engine (decode steps at a context of 4,096, with the norms riding on the products), this kernel against
 # the library's products: batch 8 9% faster; batch 16 5.13 against 5.22 ms a step at the 8B shape, 8.83 against 8.94 ms
 # at the 14B shape (context 8,192), 2.36 against 2.46 ms at the 0.6B shape; batch 32 8.15 against 6.65 ms.  Its epilogue
@@ -665,7 +673,8 @@ class _NormLink(ctypes.Structure):
     """The product's ties to the norms around it (`NormLink` of csrc/kernels/gemm_tc.cu)."""
 
     _fields_ = [("in_square_sums", _c_vp), ("in_parts", _c_int), ("in_stride", _c_int), ("in_inv_width", _c_float),
-                ("in_eps", _c_float), ("stream", _c_vp), ("next_weight", _c_vp), ("out_square_sums", _c_vp)]
+                ("in_eps", _c_float), ("stream", _c_vp), ("next_weight", _c_vp), ("out_square_sums", _c_vp),
+                ("gelu", _c_int)]           # set by the launcher
 
 
 def _gemm_tc_prepare(x: torch.Tensor, weight: torch.Tensor, splits: int | None, max_mpad: int = 128):
@@ -725,10 +734,11 @@ def _norm_link(m: int, row_sums, stream=None, next_weight=None, out_sums=None):
 
 
 def gemm_tc(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, gated: bool = False,
-            splits: int | None = None, row_sums: tuple | None = None, residual: tuple | None = None) -> torch.Tensor | None:
+            splits: int | None = None, row_sums: tuple | None = None, residual: tuple | None = None,
+            gate: str = "silu") -> torch.Tensor | None:
     """out[M, N] = x[M, K] . weight[N, K]^T for M <= 128; bfloat16 in, float32 sums, `out` bfloat16 or float32.
     With `gated`, `weight` holds, in every block of 128 rows, 64 gate rows and then the 64 matching up rows, and
-    out[M, N / 2] = silu(x . gate^T) * (x . up^T) in bfloat16.
+    out[M, N / 2] = act(x . gate^T) * (x . up^T) in bfloat16, act (`gate`) one of GEMM_TC_GATES.
 
     The RMSNorms around a product can ride on it.  `row_sums` = (parts [P, >= M] float32, width, eps): x holds
     rows that were multiplied by a norm's weights but not yet divided by their root mean square; the product
@@ -740,6 +750,8 @@ def gemm_tc(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, gated: boo
     _need(x, torch.bfloat16, "gemm input")
     _need(weight, torch.bfloat16, "gemm weight", (n, k))
     if gated:
+        if gate not in GEMM_TC_GATES:
+            raise InvalidRequest(f"the gated product for few rows applies one of {sorted(GEMM_TC_GATES)} to the gate, not {gate!r}")
         if n % 128:
             raise InvalidRequest("a gated product needs whole blocks of 64 gate and 64 up rows")
         _need(out, torch.bfloat16, "gemm out", (m, n // 2))
@@ -763,7 +775,7 @@ def gemm_tc(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, gated: boo
         link = _norm_link(m, row_sums)
     global launch_count
     launch_count += 1
-    code = lib.mrs_gemm_tc_small_m(w_map, x_map, out.data_ptr(), int(out.dtype is torch.float32), int(gated),
+    code = lib.mrs_gemm_tc_small_m(w_map, x_map, out.data_ptr(), int(out.dtype is torch.float32), GEMM_TC_GATES[gate] if gated else 0,
                                    state["partials"].data_ptr(), state["counters"].data_ptr(), m, n, k, splits, mpad,
                                    state["sms"], ctypes.byref(link) if link is not None else None, _stream())
     if code != 0:
@@ -934,11 +946,11 @@ def gemm_gated_rows_supported(x: torch.Tensor, weight: torch.Tensor) -> bool:
             and x.data_ptr() % 16 == 0 and weight.data_ptr() % 16 == 0)
 
 
-GATE_ACTIVATIONS = ("silu", "relu")       # what the tcgen05 gate/up product applies to the gate in its epilogue
+GATE_ACTIVATIONS = ("silu", "relu", "gelu_tanh")       # what the tcgen05 gate/up product applies to the gate in its epilogue
 
 
 def gemm_gated_rows(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, gate: str = "silu") -> None:
-    """out[T, N / 2] = act(x . gate^T) * (x . up^T) in bfloat16 for any number of rows, act "silu" or "relu"; `weight`
+    """out[T, N / 2] = act(x . gate^T) * (x . up^T) in bfloat16 for any number of rows, act one of GATE_ACTIVATIONS; `weight`
     [N, K] holds, in every block of 128 rows, 64 gate rows and then the 64 matching up rows (as the gated `gemm_tc`)."""
     if gate not in GATE_ACTIVATIONS:
         raise InvalidRequest(f"the gated product applies one of {GATE_ACTIVATIONS} to the gate, not {gate!r}")

@@ -242,8 +242,8 @@ class BiasedWindowAttention(Mixer):
         table = ctx.block_tables[cache.group]
         arguments = self._tile_plan()
         if self._plain_scores():
-            # nothing but scale, cap and window around the scores: the kernels that are fed by bulk tensor copies take them
-            paged_attention(q, cache, ctx, out, self.nq, self.nkv, self.d, self.window, scale=self.scale, cap=self.softcap)
+            # nothing but scale, cap, window and learned sinks around the scores: the kernels that are fed by bulk tensor copies take them
+            paged_attention(q, cache, ctx, out, self.nq, self.nkv, self.d, self.window, scale=self.scale, cap=self.softcap, sinks=self.sinks)
         elif not arguments:
             # the 32-bit path and head sizes that the tensor-core kernel does not take: one warp a (token, head)
             kernels.attention_biased_simt(q, cache.k, cache.v, ctx.positions, ctx.seq_of_token, table, out, self.nq, self.nkv,
@@ -266,10 +266,10 @@ class BiasedWindowAttention(Mixer):
         return linear(out, self.o, out_dtype=torch.float32)
 
     def _plain_scores(self) -> bool:
-        """Whether this attention, as it is served, is scale, cap, window and softmax and nothing else (no bias table, no
-        sink, no kept first positions, no chunks, no gate a head, values of the keys' size), at sizes that the kernels fed by
-        bulk tensor copies take."""
-        return (self.runtime.dtype is torch.bfloat16 and self.e == self.d and not self.bias_rows and not self.sink
+        """Whether this attention, as it is served, is scale, cap, window and softmax, with a learned sink or without, and nothing
+        else (no bias table, no kept first positions, no chunks, no gate a head, values of the keys' size), at sizes that the
+        kernels fed by bulk tensor copies take."""
+        return (self.runtime.dtype is torch.bfloat16 and self.e == self.d and not self.bias_rows and self.sink == self.sink_logits
                 and not self.keep_first and not self.chunk and self.output_gate != "heads"
                 and fast_kernels_take(self.d, self.nq // self.nkv, self.runtime.page_size))
 

@@ -142,8 +142,8 @@ class GatedMLP(FeedForward):
     arithmetic) whose result keeps the down product's float32 sums (the norm or residual sum that follows reads them).  Gate
     and up are one projection; when serving in bfloat16 with an inner size of a multiple of 64, blocks of 64 gate rows
     alternate with the 64 matching up rows, so that from 2,048 rows on the tcgen05 product may apply the activation in its
-    epilogue (silu and relu gates; where it was timed ahead of the library's product and the activation kernel); the product for few
-    rows applies a silu gate itself."""
+    epilogue (silu, relu and gelu gates; where it was timed ahead of the library's product and the activation kernel); the product for
+    few rows applies a silu or gelu gate itself."""
 
     BLOCK = 64
 
@@ -179,8 +179,8 @@ class GatedMLP(FeedForward):
     def forward(self, h, ctx):
         h = plain(h)
         act = torch.empty((h.shape[0], self.inner), dtype=self.runtime.dtype, device=self.down.device)
-        if self.block and self.activation == "silu" and few_rows(h, self.gate_up) and not observing(ctx):
-            kernels.gemm_tc(h, self.gate_up, act, gated=True)          # few rows: the product's tiles hold both halves
+        if self.block and self.activation in kernels.GEMM_TC_GATES and few_rows(h, self.gate_up) and not observing(ctx):
+            kernels.gemm_tc(h, self.gate_up, act, gated=True, gate=self.activation)          # few rows: the product's tiles hold both halves
         elif self.block and self.activation in kernels.GATE_ACTIVATIONS and not observing(ctx) \
                 and kernels.gemm_gated_rows_wins(h, self.gate_up, self.activation):
             kernels.gemm_gated_rows(h, self.gate_up, act, self.activation)
