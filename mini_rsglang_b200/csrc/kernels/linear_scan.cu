@@ -281,10 +281,14 @@ __global__ void __launch_bounds__(256, 2) linear_scan_kernel(const ScanArgs A) {
     constexpr int GROUPS = 32 / PARTS;                       // groups of four columns a warp covers
     constexpr int VECTOR = PARTS * SCAN_PITCH;               // floats of a k (or q) in shared memory
     constexpr int PAIRS = SCAN_ROWS / 2;
+    constexpr bool PRODUCTS = CHANNEL && MODE == SCAN_LOCAL;
+    __shared__ float products[PRODUCTS ? PARTS * SCAN_ROWS : 1];     // of the chunk's keeps, a channel each; one warp's alone
     pdl_launch_dependents();
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
     const int token_floats = 2 * VECTOR + A.cols, stage_floats = A.batch * token_floats + (CHANNEL ? VECTOR : 0);
     for (int i = threadIdx.x; i < 2 * stage_floats; i += blockDim.x) stage[i] = 0.0f;      // rows beyond d, columns beyond e
+    if (PRODUCTS)
+        for (int i = threadIdx.x; i < PARTS * SCAN_ROWS; i += blockDim.x) products[i] = 1.0f;
     __syncthreads();
     pdl_wait();
     const int seq = blockIdx.x, head = blockIdx.y / A.slices, slice = blockIdx.y % A.slices, chunk = blockIdx.z;
@@ -470,6 +474,18 @@ __global__ void __launch_bounds__(256, 2) linear_scan_kernel(const ScanArgs A) {
         __syncthreads();
         const float* token = stage + (b & 1) * stage_floats;
         if constexpr (CHANNEL) {
+            if (PRODUCTS && slice == 0 && warp == warps - 1) {
+                const float* ends = token + A.batch * token_floats;
+                for (int i = lane; i < A.d; i += 32) {
+                    float p = products[i];
+                    if (direct) {
+                        for (int j = 0; j < n; ++j) p *= A.keeps[(size_t)(t0 + j) * A.heads * A.d + q_at + i];
+                    } else {
+                        p *= ends[(i / SCAN_ROWS) * SCAN_PITCH + i % SCAN_ROWS];
+                    }
+                    products[i] = p;
+                }
+            }
             if (!idle && direct) {
                 for (int j = 0; j < n; ++j, token += token_floats) {
                     const float* keep = A.keeps + (size_t)(t0 + j) * A.heads * A.d + q_at;
@@ -532,21 +548,8 @@ __global__ void __launch_bounds__(256, 2) linear_scan_kernel(const ScanArgs A) {
         __syncthreads();                                     // the stage is copied into again two batches on
     }
     if (MODE == SCAN_LOCAL && !CHANNEL && threadIdx.x == 0 && slice == 0) A.chunk_decay[chunk_at] = product;
-    if (MODE == SCAN_LOCAL && CHANNEL && slice == 0) {
-        for (int i = threadIdx.x; i < A.d; i += blockDim.x) {
-            float p = 1.0f;
-            for (int t0 = first; t0 < last;) {
-                const int n = rows_at(t0);
-                if (direct_at(t0)) {
-                    for (int j = 0; j < n; ++j) p *= A.keeps[(size_t)(t0 + j) * A.heads * A.d + q_at + i];
-                } else {
-                    p *= A.keeps[(size_t)(t0 + n - 1) * A.heads * A.d + q_at + i];
-                }
-                t0 += n;
-            }
-            A.chunk_decay[chunk_at * A.d + i] = p;
-        }
-    }
+    if (PRODUCTS && slice == 0 && warp == warps - 1)
+        for (int i = lane; i < A.d; i += 32) A.chunk_decay[chunk_at * A.d + i] = products[i];
     if (MODE == SCAN_LOCAL || (MODE == SCAN_WHOLE && A.write_state)) {
         rescale(P);
 #pragma unroll
